@@ -5,6 +5,7 @@ from .bidinex import BidinexConfig
 from .loduzen import LoduzenConfig
 from .birepel import BirepelConfig
 from .ludazen import LudazenConfig
+from .zisesun import ZisesunConfig
 from .presets import PRESETS, preset
 
 

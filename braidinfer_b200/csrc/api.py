@@ -10,7 +10,7 @@ from __future__ import annotations
 import ctypes
 import os
 from ctypes import c_int, c_longlong, c_float, c_void_p, c_char_p
-from typing import List, Optional
+from typing import List, Optional, Tuple
 
 import torch
 
@@ -144,6 +144,8 @@ class Kernels:
                                     c_void_p]
         L.braid_head_prep_kv.argtypes = [c_void_p, c_longlong, c_int] + [c_void_p] * 5 + [c_int] * 10 + \
                                         [c_float, c_float, c_int, c_void_p, c_void_p]
+        L.braid_proj_prep_kv.argtypes = [c_void_p, c_longlong, c_int] + [c_void_p] * 10 + [c_int] * 10 + \
+                                        [c_float, c_void_p, c_void_p]
         L.braid_head_gate.argtypes = [c_void_p, c_longlong, c_void_p, c_longlong, c_void_p] + [c_int] * 5 + [c_void_p]
         L.braid_glu_clamp.argtypes = [c_void_p, c_void_p, c_int, c_int, c_int, c_float, c_float, c_void_p]
         L.braid_silu_mul.argtypes = [c_void_p, c_void_p, c_int, c_int, c_int, c_void_p]
@@ -163,7 +165,7 @@ class Kernels:
         L.braid_attn_simple.argtypes = [c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p,
                                         c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
                                         c_float, c_int, c_float, c_float, c_void_p, c_void_p, c_longlong, c_int, c_void_p,
-                                        c_int, c_void_p, c_void_p]
+                                        c_int, c_void_p, c_void_p, c_void_p, c_void_p]
         L.braid_head_mix.argtypes = [c_void_p, c_longlong, c_void_p, c_int, c_void_p, c_longlong, c_int, c_void_p] + \
                                     [c_int] * 5 + [c_void_p]
         L.braid_bias_xielu.argtypes = [c_void_p, c_longlong, c_void_p, c_void_p, c_int, c_void_p, c_longlong] + [c_int] * 4 + \
@@ -196,7 +198,7 @@ class Kernels:
         L.braid_concat2.argtypes = [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p]
         for name in ("braid_dyt", "braid_softcap", "braid_concat2", "braid_head_mix", "braid_bias_xielu"):
             getattr(L, name).restype = c_int
-        for name in ("braid_embed", "braid_embed_pos", "braid_head_prep_kv", "braid_head_gate", "braid_glu_clamp", "braid_rmsnorm", "braid_silu_mul", "braid_act_mul", "braid_head_norm_rope_kv",
+        for name in ("braid_embed", "braid_embed_pos", "braid_head_prep_kv", "braid_proj_prep_kv", "braid_head_gate", "braid_glu_clamp", "braid_rmsnorm", "braid_silu_mul", "braid_act_mul", "braid_head_norm_rope_kv",
                      "braid_act_mul_gather", "braid_rmsnorm_add", "braid_residual_add",
                      "braid_rope_kv_write", "braid_cast", "braid_attn_simple", "braid_gemm_simt",
                      "braid_gemm_tc", "braid_gemm_tc2", "braid_argmax", "braid_sample", "braid_streamk_reduce",
@@ -350,6 +352,31 @@ class Kernels:
             cache.shape[0] if cache is not None else 0, float(eps), float(temp_coef), int(temp_every),
             self._error_flag.data_ptr(), self._stream()), "head_prep_kv")
 
+    def proj_prep_kv(self, src: torch.Tensor, q_out: torch.Tensor, positions: torch.Tensor, token_seq: torch.Tensor,
+                     page_table: Optional[torch.Tensor], cache: Optional[torch.Tensor], nqh: int, nkh: int, dk: int, dv: int,
+                     hd: int, eps: float, q_w: Optional[torch.Tensor] = None, k_w: Optional[torch.Tensor] = None,
+                     biases: Optional[Tuple[torch.Tensor, torch.Tensor, torch.Tensor]] = None, v_unit: bool = False) -> None:
+        """The rows of `head_prep_kv` (nqh query heads of dk, nkh key heads of dk, nkh value heads of dv) with another
+        preparation: `biases` (q, k, v; one number a column) are added first; q_w [nqh * dk] and k_w [nkh * dk] RMS-norm all
+        query heads of a row together and all its key heads together; with `v_unit` every value head is divided by its own
+        root mean square.  Queries go to q_out [rows, nqh * hd], keys and values into the cache, padded with zeros up to hd."""
+        if src.stride(1) != 1 or src.shape[1] < nqh * dk + nkh * (dk + dv) or q_out.dtype != src.dtype \
+                or tuple(q_out.shape) != (src.shape[0], nqh * hd) or not q_out.is_contiguous():
+            raise KernelError("proj_prep_kv: the rows do not hold the heads, or q_out is not [rows, heads * padded size]")
+        if cache is not None and (cache.dtype != src.dtype or cache.shape[-1] != hd or cache.shape[1] != 2 or cache.shape[2] != nkh):
+            raise KernelError("proj_prep_kv: the cache is [pages, 2, kv_heads, page, padded size] of the rows' element type")
+        b = biases or (None, None, None)
+        for t, n in ((q_w, nqh * dk), (k_w, nkh * dk), (b[0], nqh * dk), (b[1], nkh * dk), (b[2], nkh * dv)):
+            if t is not None and (t.dtype != src.dtype or t.numel() != n or not t.is_contiguous()):
+                raise KernelError("proj_prep_kv: a norm's weights and a bias hold one number a column, in the rows' element type")
+        self.launches += 1
+        self._check(self.lib.braid_proj_prep_kv(
+            src.data_ptr(), src.stride(0), dtype_code(src.dtype), _ptr(b[0]), _ptr(b[1]), _ptr(b[2]), _ptr(q_w), _ptr(k_w),
+            q_out.data_ptr(), positions.data_ptr(), token_seq.data_ptr(), _ptr(page_table), _ptr(cache), src.shape[0], nqh, nkh,
+            dk, dv, hd, int(v_unit), cache.shape[3] if cache is not None else build.page_size(),
+            page_table.shape[1] if page_table is not None else 0, cache.shape[0] if cache is not None else 0, float(eps),
+            self._error_flag.data_ptr(), self._stream()), "proj_prep_kv")
+
     def head_gate(self, x: torch.Tensor, gate: Optional[torch.Tensor], out: torch.Tensor, heads: int, hd: int, dv: int) -> None:
         """out[r, h * dv + c] = x[r, h * hd + c] * sigmoid(gate[r, h]), c < dv (gate None: the copy alone)."""
         rows = out.shape[0]
@@ -402,16 +429,18 @@ class Kernels:
                     page_size: int, window: Optional[int], scale: float, sink: Optional[float] = None,
                     out_scale: float = 1.0, head_sinks: Optional[torch.Tensor] = None,
                     head_gate: Optional[torch.Tensor] = None, keep_first: int = 0,
-                    head_scale: Optional[torch.Tensor] = None, value_heads: int = 1) -> None:
+                    head_scale: Optional[torch.Tensor] = None, value_heads: int = 1,
+                    distance_bias: Optional[Tuple[torch.Tensor, torch.Tensor]] = None) -> None:
         """q: [rows, >= nqh*hd] (a view of the qkv rows is fine), out: [rows, nqh*hd].  `keep_first`: with a window,
         a sequence's first positions stay visible; `head_scale` (float32 [nqh]): a factor a head on the scores;
         `value_heads` = nkh: every query head reads the values of every kv head, out is [rows, nqh*nkh*hd] with
         the result of (head h, value head c) at virtual head h*nkh + c (see `head_mix`).  `sink`: the score of an
         attention sink, one more term of the softmax's denominator that has no value (None: no sink);
         `head_sinks` (float32 [nqh]): a sink score a head instead; `out_scale`: a constant factor on the result;
+        `distance_bias` (r1, r2; float32 [nqh] each): r1 ln(1 + r2 (p - j)) comes off the score of key j at position p;
         `head_gate` ([rows, >= nqh] of the rows' type, a view is fine): head h's result times sigmoid(head_gate[row, h])."""
         rows = out.shape[0]
-        self._check_head_extras(head_sinks, head_gate, nqh, out.dtype, head_scale)
+        self._check_head_extras(head_sinks, head_gate, nqh, out.dtype, head_scale, distance_bias)
         if out.shape[1] < nqh * value_heads * hd:
             raise KernelError("attn_simple: the result's rows do not hold the heads")
         self.launches += 1
@@ -421,7 +450,7 @@ class Kernels:
             page_size, page_table.shape[1], cache.shape[0], int(window or 0), float(scale),
             int(sink is not None), float(sink or 0.0), float(out_scale), _ptr(head_sinks), _ptr(head_gate),
             head_gate.stride(0) if head_gate is not None else 0, int(keep_first or 0), _ptr(head_scale), int(value_heads),
-            self._error_flag.data_ptr() + 16, self._stream()),
+            *self._bias_args(distance_bias), self._error_flag.data_ptr() + 16, self._stream()),
             "attn_simple")
 
     def head_mix(self, src: torch.Tensor, talk: torch.Tensor, out: torch.Tensor, token_seq: Optional[torch.Tensor],
@@ -450,7 +479,14 @@ class Kernels:
                                               self._stream()), "bias_xielu")
 
     @staticmethod
-    def _check_head_extras(head_sinks, head_gate, nqh: int, dtype, head_scale=None) -> None:
+    def _bias_args(distance_bias):
+        return (None, None) if distance_bias is None else (distance_bias[0].data_ptr(), distance_bias[1].data_ptr())
+
+    @staticmethod
+    def _check_head_extras(head_sinks, head_gate, nqh: int, dtype, head_scale=None, distance_bias=None) -> None:
+        for t in distance_bias or ():
+            if t.dtype != torch.float32 or t.numel() != nqh or not t.is_contiguous():
+                raise KernelError(f"a distance bias is two float32 tensors of {nqh} numbers, one a head")
         if head_scale is not None and (head_scale.dtype != torch.float32 or head_scale.numel() != nqh or not head_scale.is_contiguous()):
             raise KernelError(f"attention: a factor a head is a contiguous float32 tensor of {nqh} numbers")
         if head_sinks is not None and (head_sinks.dtype != torch.float32 or head_sinks.numel() != nqh or not head_sinks.is_contiguous()):
@@ -480,7 +516,7 @@ class Kernels:
             lib.braid_last_error.restype = c_char_p
             lib.braid_attn_mma.restype = c_int
             lib.braid_attn_mma.argtypes = [c_void_p] * 9 + [c_int] * 13 + [c_float, c_int, c_float, c_float, c_void_p, c_void_p,
-                                           c_longlong, c_int, c_void_p, c_int, c_int, c_void_p, c_void_p]
+                                           c_longlong, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p]
             lib.braid_attn_mma_partial_floats.restype = c_longlong
             lib.braid_attn_mma_partial_floats.argtypes = [c_int, c_int, c_int]
             if lib.braid_attn_mma_value_heads() != value_heads:
@@ -492,7 +528,8 @@ class Kernels:
             if lib.has_tc:
                 lib.braid_attn_tc.restype = c_int
                 lib.braid_attn_tc.argtypes = [c_void_p, c_void_p, c_void_p, c_longlong] + [c_void_p] * 4 + [c_int] * 10 + \
-                                             [c_float, c_int, c_float, c_float, c_void_p, c_void_p, c_longlong, c_void_p, c_void_p]
+                                             [c_float, c_int, c_float, c_float, c_void_p, c_void_p, c_longlong, c_void_p, c_void_p,
+                                              c_void_p, c_void_p]
             lib.braid_attn_mma_decode_slots.restype = c_int
             lib.braid_attn_mma_decode_slots.argtypes = [c_int]
             lib.decode_slots = lib.braid_attn_mma_decode_slots(1)     # CTAs of the few-token kernel held at once
@@ -514,11 +551,12 @@ class Kernels:
                 q_start: torch.Tensor, q_len: torch.Tensor, kv_before: torch.Tensor, n_seqs: int, max_q_len: int,
                 nqh: int, nkh: int, hd: int, window: Optional[int], scale: float, sink: Optional[float] = None,
                 out_scale: float = 1.0, head_sinks: Optional[torch.Tensor] = None,
-                head_gate: Optional[torch.Tensor] = None) -> None:
+                head_gate: Optional[torch.Tensor] = None,
+                distance_bias: Optional[Tuple[torch.Tensor, torch.Tensor]] = None) -> None:
         """bfloat16 attention of prompts over the cache on tcgen05 (head sizes 64 and 128); `sink`, `head_sinks`,
-        `out_scale` and `head_gate` as in `attn_simple`."""
+        `out_scale`, `head_gate` and `distance_bias` as in `attn_simple`."""
         lib = self.attn_mma_library(hd)
-        self._check_head_extras(head_sinks, head_gate, nqh, out.dtype)
+        self._check_head_extras(head_sinks, head_gate, nqh, out.dtype, distance_bias=distance_bias)
         self._check_pages(cache)
         if not lib.has_tc:
             raise KernelError(f"the tcgen05 attention is built for head sizes 64 and 128, not {hd}")
@@ -529,7 +567,7 @@ class Kernels:
                                out.shape[0], n_seqs, max_q_len, nqh, nkh, hd, page_table.shape[1], int(window or 0),
                                float(scale), int(sink is not None), float(sink or 0.0), float(out_scale),
                                _ptr(head_sinks), _ptr(head_gate), head_gate.stride(0) if head_gate is not None else 0,
-                               self._error_flag.data_ptr() + 12, self._stream())
+                               *self._bias_args(distance_bias), self._error_flag.data_ptr() + 12, self._stream())
         if rc != 0:
             raise KernelError(f"attn_tc: {lib.braid_last_error().decode(errors='replace')} (code {rc})")
 
@@ -543,15 +581,16 @@ class Kernels:
                  n_splits: int = 1, few_tokens: bool = False, sink: Optional[float] = None,
                  out_scale: float = 1.0, head_sinks: Optional[torch.Tensor] = None,
                  head_gate: Optional[torch.Tensor] = None, keep_first: int = 0,
-                 head_scale: Optional[torch.Tensor] = None, value_heads: int = 1) -> None:
+                 head_scale: Optional[torch.Tensor] = None, value_heads: int = 1,
+                 distance_bias: Optional[Tuple[torch.Tensor, torch.Tensor]] = None) -> None:
         """bfloat16 attention over the cache on the tensor cores; `n_splits` > 1 slices the
         context (for steps of few tokens) and merges the slices in a second kernel.  `sink`, `head_sinks`,
-        `out_scale`, `head_gate`, `keep_first`, `head_scale` and `value_heads` as in `attn_simple` (the sink is counted
+        `out_scale`, `head_gate`, `keep_first`, `head_scale`, `distance_bias` and `value_heads` as in `attn_simple` (the sink is counted
         once, where the slices merge; where the accumulators do not hold the values of all kv heads, groups of them
         go to CTAs of their own)."""
         vh = self.attn_value_heads_a_launch(hd, value_heads) if value_heads > 1 else 1
         lib = self.attn_mma_library(hd, vh)
-        self._check_head_extras(head_sinks, head_gate, nqh, out.dtype, head_scale)
+        self._check_head_extras(head_sinks, head_gate, nqh, out.dtype, head_scale, distance_bias)
         self._check_pages(cache)
         rows = out.shape[0]
         if value_heads > 1 and (value_heads != nkh or out.shape[1] < nqh * nkh * hd):
@@ -573,7 +612,7 @@ class Kernels:
                                     1 if few_tokens else 0, float(scale), int(sink is not None), float(sink or 0.0),
                                     float(out_scale), _ptr(head_sinks), _ptr(head_gate),
                                     head_gate.stride(0) if head_gate is not None else 0, int(keep_first or 0),
-                                    _ptr(head_scale), vh0, value_heads if value_heads > 1 else 0,
+                                    _ptr(head_scale), *self._bias_args(distance_bias), vh0, value_heads if value_heads > 1 else 0,
                                     self._error_flag.data_ptr() + 16, self._stream())
             if rc != 0:
                 raise KernelError(f"attn_mma: {lib.braid_last_error().decode(errors='replace')} (code {rc})")
@@ -630,7 +669,7 @@ class Kernels:
                 lib.braid_linear_scan.argtypes = [c_void_p, c_longlong] * 4 + [c_void_p] * 3 + [c_void_p, c_longlong] + \
                                                  [c_void_p, c_longlong, c_longlong] + [c_void_p] * 3 + [c_int] * 7 + \
                                                  [c_float, c_float, c_int, c_int, c_void_p, c_longlong, c_int, c_void_p, c_int,
-                                                  c_void_p]
+                                                  c_int, c_void_p]
                 lib.braid_mlstm_gates.argtypes = [c_void_p, c_longlong, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_longlong,
                                                   c_longlong, c_void_p, c_void_p, c_void_p, c_int, c_int, c_float, c_void_p]
                 lib.braid_mlstm_out.argtypes = [c_void_p, c_void_p, c_longlong, c_void_p, c_longlong, c_void_p, c_void_p,
@@ -639,11 +678,11 @@ class Kernels:
                 lib.braid_linear_scan_work_floats.argtypes = [c_int] * 7
                 lib.braid_linear_scan_work_floats.restype = c_longlong
                 lib.braid_gated_norm.argtypes = [c_void_p, c_void_p, c_longlong, c_void_p, c_int, c_void_p, c_longlong,
-                                                 c_void_p] + [c_int] * 5 + [c_float, c_float, c_void_p]
+                                                 c_void_p] + [c_int] * 6 + [c_float, c_float, c_void_p]
                 names = ("braid_causal_conv", "braid_linear_scan", "braid_gated_norm", "braid_scan_decay", "braid_mlstm_gates",
                          "braid_mlstm_out")
             elif name == "moe":
-                lib.braid_moe_route.argtypes = [c_void_p] * 3 + [c_int] * 5 + [c_float, c_int, c_void_p]
+                lib.braid_moe_route.argtypes = [c_void_p] * 3 + [c_int] * 5 + [c_float, c_int, c_int, c_void_p, c_void_p]
                 lib.braid_moe_plan.argtypes = [c_void_p] * 6 + [c_int] * 5 + [c_void_p]
                 lib.braid_moe_gemm_simt.argtypes = [c_void_p] * 7 + [c_int, c_int, c_longlong, c_longlong] + [c_int] * 5 + \
                                                    [c_void_p, c_void_p]
@@ -653,6 +692,11 @@ class Kernels:
                                                   [c_void_p, c_void_p]
                 lib.braid_moe_gemm_mma.restype = c_int
                 names = ("braid_moe_route", "braid_moe_plan", "braid_moe_gemm_simt", "braid_moe_combine")
+            elif name == "streams":
+                lib.braid_streams.argtypes = [c_void_p, c_void_p] + [c_int] * 4 + [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int,
+                                              c_longlong, c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_int,
+                                              c_void_p, c_int, c_float, c_int, c_void_p]
+                names = ("braid_streams", "braid_streams_max")
             else:
                 names = ()
             for n in names:
@@ -744,19 +788,25 @@ class Kernels:
 
     # ------------------------------------------------------------------ mixture of experts
     def moe_route(self, logits: torch.Tensor, idx: torch.Tensor, wgt: torch.Tensor, groups: int, keep: int,
-                  mult: float = 1.0, sigmoid: bool = False) -> None:
+                  mult: float = 1.0, sigmoid: bool = False, renorm: Optional[bool] = None,
+                  correction: Optional[torch.Tensor] = None) -> None:
         """Router logits [rows, experts] (float32) -> for each row its `top` experts idx [rows, top] (int32, by falling
         score) and their weights wgt [rows, top] (float32): softmax scores of the chosen, over their sum, times mult;
-        with `sigmoid` the scores are sigmoids of the logits and the weights the chosen scores as they are, times mult."""
+        with `sigmoid` the scores are sigmoids of the logits and the weights the chosen scores as they are, times mult.
+        `renorm` (default: not with `sigmoid`) says whether the weights are divided by their sum.  `correction` (float32
+        [experts], experts in one group): the choice is made on score + correction, the weights are the scores without it."""
         lib = self.part_library("moe")
         rows, experts = logits.shape
         top = idx.shape[1]
         if logits.dtype != torch.float32 or not logits.is_contiguous() or idx.dtype != torch.int32 or wgt.dtype != torch.float32 \
                 or tuple(idx.shape) != (rows, top) or tuple(wgt.shape) != (rows, top) or not idx.is_contiguous() or not wgt.is_contiguous():
             raise KernelError("moe_route: logits float32 [rows, experts], idx int32 and wgt float32 [rows, top], contiguous")
+        if correction is not None and (correction.dtype != torch.float32 or correction.numel() != experts or not correction.is_contiguous()):
+            raise KernelError("moe_route: the correction is float32, one number an expert")
         self.launches += 1
         self._check_lib(lib, lib.braid_moe_route(logits.data_ptr(), idx.data_ptr(), wgt.data_ptr(), rows, experts, top,
-                                                 groups, keep, float(mult), int(sigmoid), self._stream()), "moe_route")
+                                                 groups, keep, float(mult), int(sigmoid), int(not sigmoid if renorm is None else renorm),
+                                                 _ptr(correction), self._stream()), "moe_route")
 
     @staticmethod
     def moe_max_tiles(rows: int, top: int, experts: int, tile: int) -> int:
@@ -917,6 +967,63 @@ class Kernels:
                                                    y.stride(0), self._stream()),
                         "moe_combine")
 
+    # ------------------------------------------------------------------ residual streams mixed at every sublayer
+    @staticmethod
+    def streams_cluster(rows: int, width: int) -> int:
+        """CTAs that share a row: more where a step has few rows, as long as each keeps a few hundred columns."""
+        c = 1
+        while c < 8 and rows * c * 2 <= 148 and width >= 512 * c:
+            c *= 2
+        return c
+
+    def streams(self, x: torch.Tensor, x_out: Optional[torch.Tensor], n: int, *, y=None, mix: Optional[torch.Tensor] = None,
+                back: Optional[torch.Tensor] = None, read: Optional[torch.Tensor] = None, w: Optional[torch.Tensor] = None,
+                eps: float = 0.0, out: Optional[torch.Tensor] = None, row_index: Optional[torch.Tensor] = None,
+                cluster: Optional[int] = None) -> None:
+        """x float32 [rows, n or 1, width] (1: all n streams are that row).  With y, a sublayer's result:
+        X_t <- sum_s mix[s, t] X_s + back[t] y, mix [n, n] and back [n] float32; y is float32 rows [rows, width], a
+        `PartialProduct` (its sum is added here), or (outputs [slots, width], plan, weights | None, top) as a mixture of experts
+        leaves them.  The new streams go to x_out [rows, n, width] (it may be x; None: not kept).  With `out`:
+        u = sum_s read[s] X_s (`read` None: ones), out = u / sqrt(mean(u^2) + eps) * w (w None: u itself), one row a row of
+        x or, with `row_index`, the rows it names (the streams are then not kept)."""
+        lib = self.part_library("streams")
+        rows_x, n_in, width = x.shape
+        if x.dtype != torch.float32 or not x.is_contiguous() or n_in not in (1, n):
+            raise KernelError("streams: x is contiguous float32 [rows, streams or 1, width]")
+        if x_out is not None and (x_out.dtype != torch.float32 or not x_out.is_contiguous() or tuple(x_out.shape) != (rows_x, n, width)):
+            raise KernelError("streams: the new streams are contiguous float32 [rows, streams, width]")
+        for t, k in ((mix, n * n), (back, n), (read, n)):
+            if t is not None and (t.dtype != torch.float32 or t.numel() != k or not t.is_contiguous()):
+                raise KernelError("streams: mix, back and read are float32, [n, n], [n] and [n]")
+        if out is not None and (not out.is_contiguous() or out.shape[1] != width
+                                or out.shape[0] != (row_index.numel() if row_index is not None else rows_x)):
+            raise KernelError("streams: out holds one contiguous row a row read")
+        if w is not None and (w.numel() != width or not w.is_contiguous()):
+            raise KernelError("streams: the norm has one weight a column")
+        kind, y_t, ldy, pair_slot, wgt, top, plan, prows = 0, None, 0, None, None, 0, None, 0
+        if isinstance(y, PartialProduct):
+            if y.w_rows != width or y.n_rows != rows_x or y.rs_rows is not None:
+                raise KernelError("streams: the partial product does not fit the streams")
+            self._close_partial(y)
+            kind, y_t, plan, prows = 2, y.workspace, y.plan, y.n_rows
+        elif isinstance(y, tuple):
+            y_t, p, wgt, top = y
+            if y_t.shape[1] != width or y_t.stride(1) != 1 or p[1].numel() != rows_x * top \
+                    or (wgt is not None and (wgt.dtype != torch.float32 or tuple(wgt.shape) != (rows_x, top) or not wgt.is_contiguous())):
+                raise KernelError("streams: the experts' outputs, their plan and weights do not fit the rows")
+            kind, ldy, pair_slot = 3, y_t.stride(0), p[1]
+        elif y is not None:
+            if y.dtype != torch.float32 or tuple(y.shape) != (rows_x, width) or y.stride(1) != 1:
+                raise KernelError("streams: a sublayer's finished rows are float32 [rows, width]")
+            kind, y_t, ldy = 1, y, y.stride(0)
+        rows = out.shape[0] if row_index is not None else rows_x
+        self.launches += 1
+        self._check_lib(lib, lib.braid_streams(
+            x.data_ptr(), _ptr(x_out), n, n_in, width, rows, _ptr(row_index), kind, _ptr(mix), _ptr(back), _ptr(y_t),
+            dtype_code(y_t.dtype) if y_t is not None else F32, ldy, _ptr(pair_slot), _ptr(wgt), top, plan, prows, _ptr(read),
+            _ptr(w), dtype_code(w.dtype) if w is not None else F32, _ptr(out), dtype_code(out.dtype) if out is not None else F32,
+            float(eps), cluster or self.streams_cluster(rows, width), self._stream()), "streams")
+
     # ------------------------------------------------------------------ mixers with a recurrent state
     @staticmethod
     def _state_args(state: torch.Tensor, offset: int):
@@ -946,7 +1053,7 @@ class Kernels:
                     out: torch.Tensor, state: torch.Tensor, state_offset: int, ctx, heads: int, groups: int, dk: int,
                     dv: int, mode: str, q_scale: float = 1.0, inv_tau: float = 1.0, a_log: Optional[torch.Tensor] = None,
                     skip: Optional[torch.Tensor] = None, chunk: Optional[int] = None, gate_is_decay: bool = False,
-                    kappa: Optional[torch.Tensor] = None, v_cols: Optional[int] = None) -> None:
+                    kappa: Optional[torch.Tensor] = None, v_cols: Optional[int] = None, act_silu: bool = False) -> None:
         """The recurrence S <- diag(a) S + (kappa k) v^T, o = S^T (q_scale q) + skip v, token by token along each
         sequence of the step, S float32 [heads, dk, dv] at `state_offset` bytes of each slot.  mode "channel":
         a = sigmoid(gate + gate_bias)^inv_tau per key channel (gate float32 [rows, heads * dk]); mode "head":
@@ -957,12 +1064,15 @@ class Kernels:
         before (`mlstm_gates`); with `v_cols` < dv, v holds v_cols columns a head and the state's other columns take
         a value of 1 (a normaliser: S[:, v_cols] sums the decayed keys, out[:, v_cols] is its product with the query).
         `gate_bias` is then unused (pass any tensor of the rows' type).
+        mode "constant": a = gate[head], float32 [heads], the same for every token, kappa = 1 (`gate_bias` is unused);
+        with `act_silu` q, k and v are silu of what is given, computed in float32.
         A step whose longest sequence brings at least two chunks of `chunk` tokens (default: see SCAN_CHUNK; 0: never)
         walks its chunks side by side in three passes (see csrc/scan.cu); the results differ from the walk
         token by token by rounding only."""
         lib = self.part_library("scan")
-        if not (q.dtype == k.dtype == v.dtype == gate_bias.dtype) or out.dtype != torch.float32 \
-                or any(t.stride(1) != 1 for t in (q, k, v, gate, out)):
+        if not (q.dtype == k.dtype == v.dtype) or (gate_bias is not None and gate_bias.dtype != q.dtype) \
+                or (gate_bias is None and mode in ("channel", "head")) or out.dtype != torch.float32 \
+                or any(t.stride(-1) != 1 for t in (q, k, v, gate, out)):
             raise KernelError("linear_scan: q, k, v and the gate's bias of one element type, out float32, rows contiguous")
         if mode == "channel":
             if gate.dtype != torch.float32 or gate.shape[1] != heads * dk or gate_bias.numel() != heads * dk:
@@ -976,6 +1086,9 @@ class Kernels:
             if gate.dtype != torch.float32 or kappa is None or kappa.dtype != torch.float32 or kappa.stride(0) != gate.stride(0) \
                     or kappa.stride(1) != 1 or gate.shape[1] < heads or kappa.shape[1] < heads:
                 raise KernelError("linear_scan: given decays and key factors are float32 [rows, heads] views of one row stride")
+        elif mode == "constant":
+            if gate.dtype != torch.float32 or gate.numel() != heads or not gate.is_contiguous():
+                raise KernelError("linear_scan: constant decays are float32, one number a head")
         else:
             raise KernelError(f"linear_scan: unknown decay mode {mode!r}")
         vc = dv if v_cols is None else int(v_cols)
@@ -984,17 +1097,17 @@ class Kernels:
         if chunk is None:
             chunk = SCAN_CHUNK if SCAN_CHUNK is not None else (128 if int(ctx.max_q_len) >= 1024 else 64)
         chunk = int(chunk)
-        code = {"channel": 0, "head": 1, "given": 2}[mode]
+        code = {"channel": 0, "head": 1, "given": 2, "constant": 3}[mode]
         need = lib.braid_linear_scan_work_floats(ctx.n_seqs, int(ctx.max_q_len), chunk, heads, dk, dv, code)
         work = torch.empty(need, dtype=torch.float32, device=out.device) if need > 0 else None
         self.launches += 3 if need > 0 else 1
         self._check_lib(lib, lib.braid_linear_scan(
             q.data_ptr(), q.stride(0), k.data_ptr(), k.stride(0), v.data_ptr(), v.stride(0), gate.data_ptr(), gate.stride(0),
-            gate_bias.data_ptr(), _ptr(a_log), _ptr(skip), out.data_ptr(), out.stride(0),
+            _ptr(gate_bias), _ptr(a_log), _ptr(skip), out.data_ptr(), out.stride(0),
             *self._state_args(state, state_offset), ctx.q_start.data_ptr(), ctx.q_len.data_ptr(), ctx.slot_ids.data_ptr(),
             dtype_code(q.dtype), code, ctx.n_seqs, heads, groups, dk, dv, float(q_scale),
             float(inv_tau), int(ctx.max_q_len), chunk, _ptr(work), need, int(gate_is_decay), _ptr(kappa), vc,
-            self._stream()), "linear_scan")
+            int(act_silu), self._stream()), "linear_scan")
 
     def mlstm_gates(self, z: torch.Tensor, bias_i: torch.Tensor, bias_f: torch.Tensor, out: torch.Tensor,
                     state: torch.Tensor, state_offset: int, ctx, heads: int, cap: float) -> None:
@@ -1041,10 +1154,10 @@ class Kernels:
                                                   z.shape[1], float(inv_tau), self._stream()), "scan_decay")
 
     def gated_norm(self, y: torch.Tensor, gate: torch.Tensor, w: torch.Tensor, out: torch.Tensor, token_seq: torch.Tensor,
-                   group: int, gate_first: bool, eps: float, out_scale: float = 1.0) -> None:
+                   group: int, gate_first: bool, eps: float, out_scale: float = 1.0, gate_sigmoid: bool = False) -> None:
         """Groups of `group` columns of y (float32 [rows, width]), each by its own root mean square: norm then
         silu(gate), or (gate_first) silu(gate) then norm; times w (one weight a group's column, or one a column of
-        the row) and out_scale."""
+        the row) and out_scale.  `gate_sigmoid`: the gate goes through a sigmoid instead of silu."""
         lib = self.part_library("scan")
         rows, width = y.shape
         if y.dtype != torch.float32 or not y.is_contiguous() or not (gate.dtype == w.dtype == out.dtype) \
@@ -1053,8 +1166,8 @@ class Kernels:
         self.launches += 1
         self._check_lib(lib, lib.braid_gated_norm(
             y.data_ptr(), gate.data_ptr(), gate.stride(0), w.data_ptr(), w.numel(), out.data_ptr(), out.stride(0),
-            token_seq.data_ptr(), dtype_code(out.dtype), rows, width, group, int(gate_first), float(eps), float(out_scale),
-            self._stream()), "gated_norm")
+            token_seq.data_ptr(), dtype_code(out.dtype), rows, width, group, int(gate_first), int(gate_sigmoid), float(eps),
+            float(out_scale), self._stream()), "gated_norm")
 
     # ------------------------------------------------------------------ matrix products
     def gemm_simt(self, x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, residual: Optional[torch.Tensor] = None) -> None:

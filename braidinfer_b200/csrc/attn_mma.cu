@@ -14,7 +14,8 @@
 // Visibility is the one rule of the whole library: key j is visible to the query at
 // position p iff j <= p and (window == 0 or p - j < window); with keep_first > 0 the sequence's first
 // keep_first positions stay visible beyond the window (their tiles are walked before the window's).
-// head_scale is a factor a head on the scores.  Compiled with -DBRAID_VH=<n> (default 1) and called with
+// head_scale is a factor a head on the scores; bias_slope and bias_rate take r1 ln(1 + r2 (p - j)) off the score of
+// key j, a number a head each.  Compiled with -DBRAID_VH=<n> (default 1) and called with
 // vh_total > 0, every query head applies its probabilities to the values of every kv head as well as
 // sharing the keys of its own kv head, n value heads a CTA (the grid grows by vh_total / n), and writes the results at
 // virtual heads head * vh_total + value head: what a mix of the heads' probabilities after the softmax needs
@@ -58,6 +59,8 @@ struct AttnMmaArgs {
     long long gate_stride;
     int keep_first;              // with a window: the first positions of a sequence stay visible
     const float* head_scale;     // [nqh] float32: a factor a head on the scores; or null
+    const float* bias_slope;     // [nqh] float32 r1 and r2 of the distance bias r1 ln(1 + r2 (p - j)); or null, both
+    const float* bias_rate;
     int vh0, vh_total;           // vh_total > 0: the values of kv heads vh0 .. vh_total - 1, VH of them a CTA, results at virtual heads
 };
 
@@ -200,11 +203,20 @@ attn_mma_kernel(AttnMmaArgs a) {
     const int row_a = warp * 16 + (lane >> 2), row_b = row_a + 8;
     int pos_a = -1, pos_b = -1;                            // -1: the row sees nothing
     float sc_a = a.scale_log2, sc_b = a.scale_log2;        // the factor on the row's scores
+    float r1_a = 0.f, r2_a = 0.f, r1_b = 0.f, r2_b = 0.f;  // the row's distance bias
     {
         const int ta = row_a / hpc, ha = row_a - ta * hpc;
         const int tb = row_b / hpc, hb = row_b - tb * hpc;
-        if (ta < n_tok && ha < n_heads) { pos_a = pos_min + ta; if (a.head_scale) sc_a *= a.head_scale[head0 + ha]; }
-        if (tb < n_tok && hb < n_heads) { pos_b = pos_min + tb; if (a.head_scale) sc_b *= a.head_scale[head0 + hb]; }
+        if (ta < n_tok && ha < n_heads) {
+            pos_a = pos_min + ta;
+            if (a.head_scale) sc_a *= a.head_scale[head0 + ha];
+            if (a.bias_slope) { r1_a = a.bias_slope[head0 + ha]; r2_a = a.bias_rate[head0 + ha]; }
+        }
+        if (tb < n_tok && hb < n_heads) {
+            pos_b = pos_min + tb;
+            if (a.head_scale) sc_b *= a.head_scale[head0 + hb];
+            if (a.bias_slope) { r1_b = a.bias_slope[head0 + hb]; r2_b = a.bias_rate[head0 + hb]; }
+        }
     }
     const int lo_a = (a.window > 0) ? pos_a - a.window + 1 : 0;
     const int lo_b = (a.window > 0) ? pos_b - a.window + 1 : 0;
@@ -247,6 +259,23 @@ attn_mma_kernel(AttnMmaArgs a) {
         // ---- mask, online softmax
         const int key0 = tile_of(i_lo + it) * BN + (lane & 3) * 2;
         float mx_a = -INFINITY, mx_b = -INFINITY;
+        if (a.bias_slope) {
+            // in units of log2: r1 ln(1 + r2 d) log2(e) = r1 log2(1 + r2 d); keys after the query (d < 0) are masked below
+            const float d_a = (float)(pos_a - key0), d_b = (float)(pos_b - key0);
+#pragma unroll
+            for (int nb = 0; nb < BN / 8; ++nb)
+#pragma unroll
+                for (int e = 0; e < 2; ++e) {
+                    s[nb][e] = fmaf(s[nb][e], sc_a, -r1_a * __log2f(fmaf(r2_a, d_a - (float)(nb * 8 + e), 1.f)));
+                    s[nb][2 + e] = fmaf(s[nb][2 + e], sc_b, -r1_b * __log2f(fmaf(r2_b, d_b - (float)(nb * 8 + e), 1.f)));
+                }
+        } else {
+#pragma unroll
+            for (int nb = 0; nb < BN / 8; ++nb) {
+                s[nb][0] *= sc_a; s[nb][1] *= sc_a;
+                s[nb][2] *= sc_b; s[nb][3] *= sc_b;
+            }
+        }
 #pragma unroll
         for (int nb = 0; nb < BN / 8; ++nb) {
 #pragma unroll
@@ -254,8 +283,8 @@ attn_mma_kernel(AttnMmaArgs a) {
                 const int j = key0 + nb * 8 + e;
                 const bool va = (j <= pos_a) && (j >= lo_a || j < a.keep_first);
                 const bool vb = (j <= pos_b) && (j >= lo_b || j < a.keep_first);
-                s[nb][e] = va ? s[nb][e] * sc_a : -INFINITY;
-                s[nb][2 + e] = vb ? s[nb][2 + e] * sc_b : -INFINITY;
+                s[nb][e] = va ? s[nb][e] : -INFINITY;
+                s[nb][2 + e] = vb ? s[nb][2 + e] : -INFINITY;
                 mx_a = fmaxf(mx_a, s[nb][e]);
                 mx_b = fmaxf(mx_b, s[nb][2 + e]);
             }
@@ -477,7 +506,8 @@ extern "C" int braid_attn_mma(const void* q, void* out, void* partial, const voi
                               int nqh, int nkh, int hd, int table_cols, int num_pages, int window, int n_splits, int kind,
                               float scale, int has_sink, float sink_score, float out_scale, const float* head_sinks,
                               const void* head_gate, long long gate_stride, int keep_first, const float* head_scale,
-                              int vh0, int vh_total, int* error_flag, void* stream) {
+                              const float* bias_slope, const float* bias_rate, int vh0, int vh_total, int* error_flag,
+                              void* stream) {
     if (rows <= 0 || n_seqs <= 0) return BRAID_OK;
     if (head_sinks) has_sink = 1;
     if (vh_total < 0 || (vh_total > 0 && (vh_total != nkh || vh0 < 0 || vh0 + BRAID_VH > vh_total || (vh_total - vh0) % BRAID_VH)))
@@ -485,6 +515,7 @@ extern "C" int braid_attn_mma(const void* q, void* out, void* partial, const voi
     if (vh_total == 0 && BRAID_VH != 1) BRAID_REFUSE("attn_mma: this library was compiled for %d value heads a query head", BRAID_VH);
     if (vh_total > 0 && (has_sink || head_gate)) BRAID_REFUSE("attn_mma: values of every kv head go with an ordinary softmax without sink or gate");
     if (keep_first < 0) BRAID_REFUSE("attn_mma: keep_first=%d must not be negative", keep_first);
+    if (!bias_slope != !bias_rate) BRAID_REFUSE("attn_mma: a distance bias has a slope and a rate a head");
     if (window <= 0) keep_first = 0;
     // a gate a head rides on the last kernel that touches a row: the merge of the slices, or the attention itself
     const __nv_bfloat16* gate_here = n_splits > 1 ? nullptr : (const __nv_bfloat16*)head_gate;
@@ -499,7 +530,7 @@ extern "C" int braid_attn_mma(const void* q, void* out, void* partial, const voi
     AttnMmaArgs a{(const __nv_bfloat16*)q, (__nv_bfloat16*)out, (float*)partial, (const __nv_bfloat16*)cache, page_table,
                   q_start, q_len, kv_before, q_row_stride, out_row_stride, nqh, nkh, table_cols, window, n_splits,
                   scale * 1.4426950408889634f, num_pages, error_flag, has_sink, sink_score * 1.4426950408889634f, out_scale,
-                  head_sinks, gate_here, gate_stride, keep_first, head_scale, vh0, vh_total};
+                  head_sinks, gate_here, gate_stride, keep_first, head_scale, bias_slope, bias_rate, vh0, vh_total};
     cudaStream_t s = (cudaStream_t)stream;
     int rc;
     // with several value tiles a key tile, tiles of 32 keys leave room for two CTAs an SM (registers and shared memory)
@@ -561,6 +592,6 @@ extern "C" int braid_attn_mma_noalloc(const void* q, void* out, const void* cach
     }
     return braid_attn_mma(q, out, n_splits > 1 ? g_noalloc_ptr[dev] : nullptr, cache, page_table, q_start, q_len,
                           kv_before, token_seq, q_row_stride, out_row_stride, rows, n_seqs, max_q_len, nqh, nkh, hd,
-                          table_cols, num_pages, window, n_splits, kind, scale, 0, 0.f, 1.f, nullptr, nullptr, 0, 0, nullptr, 0, 0,
+                          table_cols, num_pages, window, n_splits, kind, scale, 0, 0.f, 1.f, nullptr, nullptr, 0, 0, nullptr, nullptr, nullptr, 0, 0,
                           error_flag, stream);
 }

@@ -17,7 +17,9 @@
 // whatever the window (visible: j <= p and (p - j < w or j < keep_first)); head_scale is a factor a head on the
 // scores; value_heads > 1 applies a head's probabilities to the values of every kv head in turn (the item is then
 // (token, query head, value head) and the result lies at virtual head `head * value_heads + value head`), which is
-// what a mix of the heads' probabilities after the softmax needs (pointwise.cu, head_mix).
+// what a mix of the heads' probabilities after the softmax needs (pointwise.cu, head_mix).  bias_slope and bias_rate
+// (a number a head each) take r1 ln(1 + r2 (p - j)) off the score of key j: a bias that grows with the logarithm of the
+// distance instead of a rotation.
 #include "common.cuh"
 
 struct AttnSimpleArgs {
@@ -39,6 +41,8 @@ struct AttnSimpleArgs {
     int keep_first;           // the first positions of a sequence stay visible beyond the window
     const float* head_scale;  // [nqh] float32: a factor a head on the scores; or null
     int value_heads;          // 1, or nkh: every query head reads the values of every kv head
+    const float* bias_slope;  // [nqh] float32 r1 and r2 of the distance bias r1 ln(1 + r2 (p - j)); or null, both
+    const float* bias_rate;
 };
 
 #define ATTN_SIMPLE_WARPS 4
@@ -68,6 +72,7 @@ attn_simple_kernel(AttnSimpleArgs a) {
     const int kvh = head / (a.nqh / a.nkh);
     const int val_h = a.value_heads > 1 ? vhead - head * a.value_heads : kvh;
     const float scale = a.head_scale ? a.scale * a.head_scale[head] : a.scale;
+    const float r1 = a.bias_slope ? a.bias_slope[head] : 0.f, r2 = a.bias_slope ? a.bias_rate[head] : 0.f;
     const T* q = (const T*)a.q + (size_t)row * a.q_row_stride + (size_t)head * a.hd;
     for (int d = lane; d < a.hd; d += 32) qs[d] = to_f32(q[d]);
     __syncwarp();
@@ -99,6 +104,7 @@ attn_simple_kernel(AttnSimpleArgs a) {
             float dot = 0.f;
             for (int d = 0; d < a.hd; ++d) dot = fmaf(qs[d], to_f32(kbase[d]), dot);
             s = dot * scale;
+            if (a.bias_slope) s -= r1 * log1pf(r2 * (float)(pos - j));
         }
         const float cmax = warp_max(s);
         const float m_new = fmaxf(m, cmax);
@@ -145,7 +151,8 @@ extern "C" int braid_attn_simple(const void* q, void* out, int dtype, const void
                                  int page_size, int table_cols, int num_pages, int window, float scale,
                                  int has_sink, float sink_score, float out_scale, const float* head_sinks,
                                  const void* head_gate, long long gate_stride, int keep_first, const float* head_scale,
-                                 int value_heads, int* error_flag, void* stream) {
+                                 int value_heads, const float* bias_slope, const float* bias_rate, int* error_flag,
+                                 void* stream) {
     if (rows <= 0) return BRAID_OK;
     if (!error_flag) BRAID_REFUSE("attn_simple: error_flag is required");
     if (num_pages <= 0 || table_cols <= 0 || page_size <= 0) BRAID_REFUSE("attn_simple: the cache has no pages (pages=%d, table columns=%d, page size=%d)", num_pages, table_cols, page_size);
@@ -154,10 +161,11 @@ extern "C" int braid_attn_simple(const void* q, void* out, int dtype, const void
     if (value_heads != 1 && value_heads != nkh) BRAID_REFUSE("attn_simple: a head reads the values of its own kv head or of all %d, not of %d", nkh, value_heads);
     if (value_heads > 1 && head_gate) BRAID_REFUSE("attn_simple: a gate a head does not go with values of every kv head");
     if (keep_first < 0) BRAID_REFUSE("attn_simple: keep_first=%d must not be negative", keep_first);
+    if (!bias_slope != !bias_rate) BRAID_REFUSE("attn_simple: a distance bias has a slope and a rate a head");
     if (window <= 0) keep_first = 0;
     AttnSimpleArgs a{q, out, cache, page_table, positions, token_seq, q_row_stride, out_row_stride,
                      rows, nqh, nkh, hd, page_size, table_cols, num_pages, window, scale, has_sink || head_sinks != nullptr, sink_score, out_scale, error_flag, head_sinks, head_gate, gate_stride,
-                     keep_first, head_scale, value_heads};
+                     keep_first, head_scale, value_heads, bias_slope, bias_rate};
     const long long items = (long long)rows * nqh * value_heads;
     const long long blocks = (items + ATTN_SIMPLE_WARPS - 1) / ATTN_SIMPLE_WARPS;
     if (blocks > 0x7fffffffLL) BRAID_REFUSE("attn_simple: %lld (token, head) pairs exceed one launch", items);

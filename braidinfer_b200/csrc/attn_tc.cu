@@ -32,7 +32,8 @@
 // *error_flag and the kernel frees its tensor memory and returns.
 //
 // Visibility is the rule of the whole library: key j is visible to the query at position
-// p iff j <= p and (window == 0 or p - j < window).  Replaces, for prompts, the
+// p iff j <= p and (window == 0 or p - j < window).  The kernel's second form (BIAS) takes r1 log2(1 + r2 (p - j)) off
+// the scores (in units of log2), r1 and r2 a number a head each, before the maximum is looked at.  Replaces, for prompts, the
 // reference's op_attn_paged (kernels/megakernel_ops.hip:2150-2343), as attn_mma.cu does;
 // attn_mma.cu stays the kernel for other head sizes and the twin this one is tested against.
 #include "common.cuh"
@@ -164,8 +165,11 @@ struct AttnTcArgs {
     const float* head_sinks;     // [nqh] float32 natural-log scores: a sink a head (learned) instead of the one score; or null
     const __nv_bfloat16* head_gate;  // [rows, gate_stride]: head h's result is multiplied by sigmoid(head_gate[row, h]); or null
     long long gate_stride;
+    const float* bias_slope;     // BIAS: [nqh] float32 r1 and r2 of the distance bias r1 ln(1 + r2 (p - j))
+    const float* bias_rate;
 };
 
+template <bool BIAS>
 __global__ void __launch_bounds__(FA_THREADS, 2)
 attn_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_kv, AttnTcArgs a) {
     constexpr int HD = BRAID_HD;
@@ -343,6 +347,10 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant_
         const int lo = (a.window > 0) ? pos - a.window + 1 : 0;
         const uint32_t lane_addr = (uint32_t)(quarter * 32) << 16;
         float m = -INFINITY, l = 0.f;
+        float r1 = 0.f, r2 = 0.f;                             // the row's distance bias
+        if (BIAS && valid) { r1 = a.bias_slope[head0 + hl]; r2 = a.bias_rate[head0 + hl]; }
+        // with the bias the scores are scaled as it is taken off
+        const float sc = BIAS ? 1.f : a.scale_log2;
         bool ok = true;
         for (int j = 0; j < n_tiles && ok; ++j) {
             const int st = j & 1;
@@ -354,6 +362,12 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant_
             tmem_ld32x2(tmem_base + st * FA_BN + lane_addr, sv);
             const int key0 = (t_lo + j) * FA_BN;
             const bool all_visible = (key0 + FA_BN - 1 <= pos_min) && (a.window == 0 || key0 >= pos_max - a.window + 1);
+            if (BIAS) {                                       // keys after the query (a negative distance) are masked below
+                const float d0 = (float)(pos - key0);
+#pragma unroll
+                for (int i = 0; i < 64; ++i)
+                    sv[i] = fmaf(sv[i], a.scale_log2, -r1 * __log2f(fmaf(r2, d0 - (float)i, 1.f)));
+            }
             float mx0 = -INFINITY, mx1 = -INFINITY, mx2 = -INFINITY, mx3 = -INFINITY;
             if (all_visible) {
                 if (valid) {
@@ -375,7 +389,7 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant_
                     mx2 = fmaxf(mx2, sv[i + 2]); mx3 = fmaxf(mx3, sv[i + 3]);
                 }
             }
-            const float mx = fmaxf(fmaxf(mx0, mx1), fmaxf(mx2, mx3)) * a.scale_log2;   // scale > 0 commutes with the maximum
+            const float mx = fmaxf(fmaxf(mx0, mx1), fmaxf(mx2, mx3)) * sc;   // scale > 0 commutes with the maximum
             // raise m only when the tile towers over it; -inf + 8 = -inf, so the first finite maximum always does
             const bool raise = mx > m + FA_RAISE;
             const float factor = raise ? fast_exp2(m - mx) : 1.f;                     // exp2(-inf) = 0: nothing was summed yet
@@ -387,8 +401,8 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant_
             uint32_t pk[32];
 #pragma unroll
             for (int i = 0; i < 32; ++i) {
-                const float p0 = fast_exp2(fmaf(sv[2 * i], a.scale_log2, -ms));
-                const float p1 = fast_exp2(fmaf(sv[2 * i + 1], a.scale_log2, -ms));
+                const float p0 = fast_exp2(fmaf(sv[2 * i], sc, -ms));
+                const float p1 = fast_exp2(fmaf(sv[2 * i + 1], sc, -ms));
                 sum0 += p0;
                 sum1 += p1;
                 __nv_bfloat162 b = __floats2bfloat162_rn(p0, p1);
@@ -471,7 +485,8 @@ extern "C" int braid_attn_tc(const void* q, void* out, const void* cache, long l
                              int q_row_stride, int out_row_stride, int rows, int n_seqs, int max_q_len,
                              int nqh, int nkh, int hd, int table_cols, int window, float scale,
                              int has_sink, float sink_score, float out_scale, const float* head_sinks, const void* head_gate,
-                             long long gate_stride, int* error_flag, void* stream) {
+                             long long gate_stride, const float* bias_slope, const float* bias_rate, int* error_flag,
+                             void* stream) {
     if (rows <= 0 || n_seqs <= 0) return BRAID_OK;
     if (head_sinks) has_sink = 1;
     if (hd != BRAID_HD) BRAID_REFUSE("attn_tc: this library was compiled for head_dim=%d, not %d", BRAID_HD, hd);
@@ -479,6 +494,7 @@ extern "C" int braid_attn_tc(const void* q, void* out, const void* cache, long l
     if ((q_row_stride % 8) || ((uintptr_t)q & 15) || ((uintptr_t)cache & 15)) BRAID_REFUSE("attn_tc: queries and cache must be 16-byte aligned");
     if ((out_row_stride % 8) || ((uintptr_t)out & 15)) BRAID_REFUSE("attn_tc: out rows must be 16-byte aligned");
     if (!error_flag) BRAID_REFUSE("attn_tc: error_flag is required");
+    if (!bias_slope != !bias_rate) BRAID_REFUSE("attn_tc: a distance bias has a slope and a rate a head");
     TcEncodeTiledFn fn = tc_encode_tiled_fn();
     if (!fn) BRAID_REFUSE("attn_tc: the driver does not export cuTensorMapEncodeTiled");
     const int g = nqh / nkh;
@@ -506,7 +522,8 @@ extern "C" int braid_attn_tc(const void* q, void* out, const void* cache, long l
     }
     static bool configured = false;
     if (!configured) {
-        cudaError_t e = cudaFuncSetAttribute(attn_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, FA_SMEM);
+        cudaError_t e = cudaFuncSetAttribute(attn_tc_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, FA_SMEM);
+        if (e == cudaSuccess) e = cudaFuncSetAttribute(attn_tc_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, FA_SMEM);
         if (e != cudaSuccess) { braid_set_error("attn_tc: cannot reserve %d bytes of shared memory: %s", FA_SMEM, cudaGetErrorString(e)); return (int)e; }
         configured = true;
     }
@@ -516,8 +533,8 @@ extern "C" int braid_attn_tc(const void* q, void* out, const void* cache, long l
     const long long num_pages = cache_rows / (2LL * nkh * FA_PAGE);
     AttnTcArgs a{(__nv_bfloat16*)out, page_table, q_start, q_len, kv_before, out_row_stride, nqh, nkh, table_cols, window,
                  scale * 1.4426950408889634f, (int)num_pages, error_flag, has_sink, sink_score * 1.4426950408889634f, out_scale,
-                 head_sinks, (const __nv_bfloat16*)head_gate, gate_stride};
-    braid_launch(attn_tc_kernel, dim3(nkh * hchunks, n_seqs, (unsigned)gx), dim3(FA_THREADS), FA_SMEM,
+                 head_sinks, (const __nv_bfloat16*)head_gate, gate_stride, bias_slope, bias_rate};
+    braid_launch(bias_slope ? attn_tc_kernel<true> : attn_tc_kernel<false>, dim3(nkh * hchunks, n_seqs, (unsigned)gx), dim3(FA_THREADS), FA_SMEM,
                  (cudaStream_t)stream, mq, mkv, a);
     BRAID_LAUNCH_CHECK();
 }

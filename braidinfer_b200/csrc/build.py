@@ -31,7 +31,8 @@ COMMON_FLAGS = ["-O3", "-std=c++17", "-lineinfo", "-Xcompiler", "-fPIC", "--expt
 CORE_SOURCES = ["errors.cu", "elementwise.cu", "pointwise.cu", "attn_simple.cu", "gemm_simt.cu", "gemm_tc.cu", "gemm_tc2.cu",
                 "fused_reduce.cu", "sampling.cu"]
 # Kernels that only some models use: each a library of its own, compiled when a model that needs it is built.
-PART_SOURCES = {"latent": ["errors.cu", "latent.cu"], "moe": ["errors.cu", "moe.cu"], "scan": ["errors.cu", "scan.cu"]}
+PART_SOURCES = {"latent": ["errors.cu", "latent.cu"], "moe": ["errors.cu", "moe.cu"], "scan": ["errors.cu", "scan.cu"],
+                "streams": ["errors.cu", "streams.cu"]}
 HEADERS = ["common.cuh", "rowscale.cuh", "streamk.cuh", "tcgen05.cuh", "attn_noalloc.h", "page.h", "trace.cuh",
            "mma_tile.cuh"]
 

@@ -927,6 +927,181 @@ extern "C" int braid_head_prep_kv(const void* src, long long row_stride, int dty
     BRAID_LAUNCH_CHECK();
 }
 
+// ------------------------------------------------------------------ whole projections normed, values of unit size, cache write
+// The rows of head_prep_kv with another preparation: a bias on every projected number (q_bias, k_bias, v_bias; or null), then
+// ONE RMS norm over all query heads of a row together and one over all its key heads, with a weight a column
+//   q <- q / sqrt(mean over nqh * dk of q^2 + eps) * q_w        (k alike; null weights: no norm)
+// and, with `v_unit`, every value head divided by its own root mean square, sqrt(mean over dv + eps), no weight.
+// Queries, keys and values then go where head_prep_kv puts them, padded with zeros up to hd.  One CTA a row; float32
+// arithmetic; V neighbouring numbers a thread and turn.
+struct ProjPrepArgs {
+    const void* src; long long row_stride;
+    const void* q_bias; const void* k_bias; const void* v_bias;
+    const void* q_w; const void* k_w;
+    void* q_out;
+    const int* positions; const int* token_seq; const int* page_table;
+    void* cache;
+    int rows, nqh, nkh, dk, dv, hd, v_unit;
+    int page_size, table_cols, num_pages;
+    float eps;
+    int* error_flag;
+};
+
+template <typename T, int V>
+__device__ __forceinline__ void load_run(const T* p, float* v) {
+    if constexpr (V == 1) {
+        v[0] = to_f32(p[0]);
+    } else {
+        __align__(16) T raw[V];
+        *reinterpret_cast<uint4*>(raw) = *reinterpret_cast<const uint4*>(p);
+#pragma unroll
+        for (int e = 0; e < V; ++e) v[e] = to_f32(raw[e]);
+    }
+}
+template <typename T, int V>
+__device__ __forceinline__ void store_run(T* p, const float* v) {
+    if constexpr (V == 1) {
+        p[0] = from_f32<T>(v[0]);
+    } else {
+        __align__(16) T raw[V];
+#pragma unroll
+        for (int e = 0; e < V; ++e) raw[e] = from_f32<T>(v[e]);
+        *reinterpret_cast<uint4*>(p) = *reinterpret_cast<const uint4*>(raw);
+    }
+}
+// V projected numbers with their bias
+template <typename T, int V>
+__device__ __forceinline__ void load_biased(const T* p, const T* b, int c, float* v) {
+    load_run<T, V>(p + c, v);
+    if (b) {
+        float bv[V];
+        load_run<T, V>(b + c, bv);
+#pragma unroll
+        for (int e = 0; e < V; ++e) v[e] += bv[e];
+    }
+}
+
+template <typename T, int V>
+__global__ void __launch_bounds__(256)
+proj_prep_kv_kernel(ProjPrepArgs a) {
+    pdl_trigger();
+    pdl_wait();
+    __shared__ float red[32];
+    const int row = blockIdx.x, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    const int nq = a.nqh * a.dk, nk = a.nkh * a.dk;
+    T* qo = (T*)a.q_out + (size_t)row * a.nqh * a.hd;
+    const int seq = a.token_seq[row];
+    if (seq < 0) {
+        for (int c = tid; c < a.nqh * a.hd; c += blockDim.x) qo[c] = from_f32<T>(0.f);
+        return;
+    }
+    const T* q = (const T*)a.src + (size_t)row * a.row_stride;
+    const T* k = q + nq;
+    const T* v = k + nk;
+    float fq = 1.f, fk = 1.f, x[V];
+    if (a.q_w) {
+        float ss = 0.f;
+        for (int c = tid * V; c < nq; c += blockDim.x * V) {
+            load_biased<T, V>(q, (const T*)a.q_bias, c, x);
+#pragma unroll
+            for (int e = 0; e < V; ++e) ss = fmaf(x[e], x[e], ss);
+        }
+        fq = 1.f / sqrtf(block_sum(ss, red) / (float)nq + a.eps);
+    }
+    if (a.k_w) {
+        float ss = 0.f;
+        for (int c = tid * V; c < nk; c += blockDim.x * V) {
+            load_biased<T, V>(k, (const T*)a.k_bias, c, x);
+#pragma unroll
+            for (int e = 0; e < V; ++e) ss = fmaf(x[e], x[e], ss);
+        }
+        fk = 1.f / sqrtf(block_sum(ss, red) / (float)nk + a.eps);
+    }
+    // heads of `count` x dk numbers, normed, to padded heads head_stride apart
+    auto spread = [&](const T* src, const T* bias, const T* w, float f, int count, T* dst, size_t head_stride) {
+        for (int c = tid * V; c < count * a.hd; c += blockDim.x * V) {
+            const int h = c / a.hd, d = c - h * a.hd;
+            float y[V];
+            if (d < a.dk) {
+                load_biased<T, V>(src, bias, h * a.dk + d, y);
+                if (w) {
+                    float wv[V];
+                    load_run<T, V>(w + h * a.dk + d, wv);
+#pragma unroll
+                    for (int e = 0; e < V; ++e) y[e] = y[e] * f * wv[e];
+                }
+            } else {
+#pragma unroll
+                for (int e = 0; e < V; ++e) y[e] = 0.f;
+            }
+            store_run<T, V>(dst + (size_t)h * head_stride + d, y);
+        }
+    };
+    spread(q, (const T*)a.q_bias, (const T*)a.q_w, fq, a.nqh, qo, a.hd);
+    if (!a.cache) return;
+    const int pos = a.positions[row];
+    const int block = pos / a.page_size, off = pos - block * a.page_size;
+    const int page = (block < a.table_cols) ? a.page_table[(size_t)seq * a.table_cols + block] : -1;
+    if (page < 0 || page >= a.num_pages) {
+        if (tid == 0) atomicExch(a.error_flag, 1);
+        return;
+    }
+    const size_t head_stride = (size_t)a.page_size * a.hd;
+    T* kdst = (T*)a.cache + ((size_t)page * 2 * a.nkh) * head_stride + (size_t)off * a.hd;
+    spread(k, (const T*)a.k_bias, (const T*)a.k_w, fk, a.nkh, kdst, head_stride);
+    T* vdst = kdst + (size_t)a.nkh * head_stride;
+    for (int h = warp; h < a.nkh; h += blockDim.x >> 5) {                    // a warp a value head
+        float f = 1.f;
+        if (a.v_unit) {
+            float ss = 0.f;
+            for (int d = lane * V; d < a.dv; d += 32 * V) {
+                load_biased<T, V>(v, (const T*)a.v_bias, h * a.dv + d, x);
+#pragma unroll
+                for (int e = 0; e < V; ++e) ss = fmaf(x[e], x[e], ss);
+            }
+            f = 1.f / sqrtf(warp_sum(ss) / (float)a.dv + a.eps);
+        }
+        for (int d = lane * V; d < a.hd; d += 32 * V) {
+            if (d < a.dv) {
+                load_biased<T, V>(v, (const T*)a.v_bias, h * a.dv + d, x);
+#pragma unroll
+                for (int e = 0; e < V; ++e) x[e] *= f;
+            } else {
+#pragma unroll
+                for (int e = 0; e < V; ++e) x[e] = 0.f;
+            }
+            store_run<T, V>(vdst + (size_t)h * head_stride + d, x);
+        }
+    }
+}
+
+extern "C" int braid_proj_prep_kv(const void* src, long long row_stride, int dtype, const void* q_bias, const void* k_bias,
+                                  const void* v_bias, const void* q_w, const void* k_w, void* q_out, const int* positions,
+                                  const int* token_seq, const int* page_table, void* cache, int rows, int nqh, int nkh,
+                                  int dk, int dv, int hd, int v_unit, int page_size, int table_cols, int num_pages, float eps,
+                                  int* error_flag, void* stream) {
+    if (rows <= 0) return BRAID_OK;
+    if (nqh <= 0 || nkh <= 0 || dk <= 0 || dv <= 0 || hd < dk || hd < dv)
+        BRAID_REFUSE("proj_prep_kv: heads %d/%d of sizes %d and %d do not fit a padded head of %d", nqh, nkh, dk, dv, hd);
+    if (cache && (!page_table || page_size <= 0)) BRAID_REFUSE("proj_prep_kv: a cache write needs the step's page table");
+    ProjPrepArgs a{src, row_stride, q_bias, k_bias, v_bias, q_w, k_w, q_out, positions, token_seq, page_table, cache,
+                   rows, nqh, nkh, dk, dv, hd, v_unit, page_size, table_cols, num_pages, eps, error_flag};
+    cudaStream_t s = (cudaStream_t)stream;
+    const int vec = dtype == BRAID_F32 ? 4 : 8;
+    // 16 bytes at a time where every head, bias and weight starts on 16 bytes and holds a whole number of such runs
+    const bool wide = dk % vec == 0 && dv % vec == 0 && hd % vec == 0 && row_stride % vec == 0 &&
+                      (((uintptr_t)src | (uintptr_t)q_bias | (uintptr_t)k_bias | (uintptr_t)v_bias | (uintptr_t)q_w |
+                        (uintptr_t)k_w | (uintptr_t)q_out | (uintptr_t)cache) & 15) == 0;
+    const int runs = nqh * hd / (wide ? vec : 1);
+    const dim3 grid(rows), block(runs > 128 ? 256 : runs > 64 ? 128 : 64);
+    if (dtype == BRAID_F32 && wide) braid_launch(proj_prep_kv_kernel<float, 4>, grid, block, 0, s, a);
+    else if (dtype == BRAID_F32) braid_launch(proj_prep_kv_kernel<float, 1>, grid, block, 0, s, a);
+    else if (dtype == BRAID_BF16 && wide) braid_launch(proj_prep_kv_kernel<__nv_bfloat16, 8>, grid, block, 0, s, a);
+    else if (dtype == BRAID_BF16) braid_launch(proj_prep_kv_kernel<__nv_bfloat16, 1>, grid, block, 0, s, a);
+    else BRAID_REFUSE("proj_prep_kv: unknown dtype code %d", dtype);
+    BRAID_LAUNCH_CHECK();
+}
+
 // ------------------------------------------------------------------ a gate a head on attention's result
 // out[r, h * dv + c] = x[r, h * hd + c] * sigmoid(gate[r, h]) for c < dv: the first dv numbers of every padded head,
 // times the head's gate (gate: a column block of the stacked projection, row stride gate_stride; null: no gate).

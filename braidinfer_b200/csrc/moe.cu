@@ -7,7 +7,8 @@
 // their s divided by the sum of the chosen s (+ 1e-20), times `mult` (a constant factor the caller wants
 // on the layer's output).  Everything float32.  `sigmoid` routing instead scores every expert by itself,
 // s = 1 / (1 + exp(-z)), chooses the same way, and leaves the chosen scores as the weights (times `mult`), not
-// renormalised.
+// renormalised.  With `correction` (a number an expert) the choice is made on score + correction while the weights keep
+// the scores without it; `renorm` says whether the weights are divided by their sum.
 //
 // The plan: every chosen (token, choice) pair gets a slot in an array ordered by expert, each expert's run
 // padded to a multiple of `tile` slots, so that a tile of slots belongs to one expert and the products can
@@ -24,7 +25,9 @@ struct MoeRouteArgs {
     float* wgt;               // [rows, top]
     int rows, experts, top, groups, keep;
     float mult;
-    int sigmoid;              // scores are sigmoids of the logits and the weights are the chosen scores as they are
+    int sigmoid;              // scores are sigmoids of the logits, not their softmax
+    int renorm;               // the chosen scores are divided by their sum
+    const float* correction;  // [experts] float32, added to the scores for the choice alone; or null
 };
 
 #define MOE_ROUTE_WARPS 4
@@ -33,12 +36,13 @@ __global__ void __launch_bounds__(MOE_ROUTE_WARPS * 32)
 moe_route_kernel(MoeRouteArgs a) {
     pdl_trigger();
     pdl_wait();
-    extern __shared__ float smem[];          // per warp: [experts] scores, [groups] group scores
+    extern __shared__ float smem[];          // per warp: [experts] scores, [groups] group scores, [experts] choice scores
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int row = blockIdx.x * MOE_ROUTE_WARPS + warp;
     if (row >= a.rows) return;
-    float* s = smem + (size_t)warp * (a.experts + a.groups);
+    float* s = smem + (size_t)warp * (2 * a.experts + a.groups);
     float* gs = s + a.experts;
+    float* cs = gs + a.groups;               // what the choice is made on: -inf once an expert is chosen
     const float* z = a.logits + (size_t)row * a.experts;
     if (a.sigmoid) {
         for (int e = lane; e < a.experts; e += 32) s[e] = 1.f / (1.f + expf(-z[e]));
@@ -56,6 +60,7 @@ moe_route_kernel(MoeRouteArgs a) {
         const float inv = 1.f / sum;
         for (int e = lane; e < a.experts; e += 32) s[e] *= inv;
     }
+    for (int e = lane; e < a.experts; e += 32) cs[e] = a.correction ? s[e] + a.correction[e] : s[e];   // this lane's own scores
     __syncwarp();
     const int per = a.experts / a.groups;
     for (int g = lane; g < a.groups; g += 32) {
@@ -82,14 +87,14 @@ moe_route_kernel(MoeRouteArgs a) {
         if (lane == 0 && bi != 0x7fffffff) gs[bi] = 3.f;
         __syncwarp();
     }
-    // the `top` largest scores among experts of kept groups; a chosen expert's score is then hidden
+    // the `top` largest scores among experts of kept groups; a chosen expert's choice score is then hidden
     float chosen_sum = 0.f;
     for (int k = 0; k < a.top; ++k) {
         float best = -INFINITY;
         int bi = 0x7fffffff;
         for (int e = lane; e < a.experts; e += 32) {
-            const float v = s[e];
-            if (v >= 0.f && gs[e / per] > 2.f && (v > best || (v == best && e < bi))) { best = v; bi = e; }
+            const float v = cs[e];
+            if (v > -INFINITY && gs[e / per] > 2.f && (v > best || (v == best && e < bi))) { best = v; bi = e; }
         }
 #pragma unroll
         for (int o = 16; o > 0; o >>= 1) {
@@ -97,28 +102,31 @@ moe_route_kernel(MoeRouteArgs a) {
             const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
             if (ob > best || (ob == best && oi < bi)) { best = ob; bi = oi; }
         }
-        if (bi == 0x7fffffff) { bi = -1; best = 0.f; }      // fewer allowed experts than `top`
+        if (bi == 0x7fffffff) bi = -1;                      // fewer allowed experts than `top`
+        best = bi >= 0 ? s[bi] : 0.f;                       // the weight is the score without the correction
         if (lane == 0) {
             a.idx[(size_t)row * a.top + k] = bi;
             a.wgt[(size_t)row * a.top + k] = best;
-            if (bi >= 0) s[bi] = -1.f;
+            if (bi >= 0) cs[bi] = -INFINITY;
         }
         chosen_sum += best;
         __syncwarp();
     }
-    const float norm = a.sigmoid ? a.mult : a.mult / (chosen_sum + 1e-20f);
+    const float norm = a.renorm ? a.mult / (chosen_sum + 1e-20f) : a.mult;
     __syncwarp();
     for (int k = lane; k < a.top; k += 32) a.wgt[(size_t)row * a.top + k] *= norm;
 }
 
 extern "C" int braid_moe_route(const float* logits, int* idx, float* wgt, int rows, int experts, int top,
-                               int groups, int keep, float mult, int sigmoid, void* stream) {
+                               int groups, int keep, float mult, int sigmoid, int renorm, const float* correction,
+                               void* stream) {
     if (rows <= 0) return BRAID_OK;
     if (experts <= 0 || top <= 0 || top > experts) BRAID_REFUSE("moe_route: top=%d of %d experts", top, experts);
     if (groups <= 0 || experts % groups || keep <= 0 || keep > groups) BRAID_REFUSE("moe_route: %d experts in %d groups, %d kept", experts, groups, keep);
-    const size_t smem = (size_t)MOE_ROUTE_WARPS * (experts + groups) * sizeof(float);
+    if (correction && groups != 1) BRAID_REFUSE("moe_route: a correction of the choice is built for experts in one group, not %d", groups);
+    const size_t smem = (size_t)MOE_ROUTE_WARPS * (2 * experts + groups) * sizeof(float);
     if (smem > 48 * 1024) BRAID_REFUSE("moe_route: %d experts are more than one block's shared memory holds", experts);
-    MoeRouteArgs a{logits, idx, wgt, rows, experts, top, groups, keep, mult, sigmoid};
+    MoeRouteArgs a{logits, idx, wgt, rows, experts, top, groups, keep, mult, sigmoid, renorm, correction};
     braid_launch(moe_route_kernel, dim3((rows + MOE_ROUTE_WARPS - 1) / MOE_ROUTE_WARPS), dim3(MOE_ROUTE_WARPS * 32), smem,
                  (cudaStream_t)stream, a);
     BRAID_LAUNCH_CHECK();

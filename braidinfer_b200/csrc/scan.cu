@@ -183,6 +183,8 @@ extern "C" int braid_causal_conv(const void* x, long long x_stride, void* y, lon
 //       channel and kappa_t = kappa[t, h], both float32 with row stride gate_stride; no skip.  With `v_cols` < dv the
 //       value columns from v_cols on read as 1: the state's column v_cols is then the sum of the decayed keys
 //       (a normaliser), and the output's column v_cols its product with the query.
+//   DECAY_CONST (lightning attention: one constant decay a head): a_t = gate[h], float32 [heads], kappa = 1, no skip;
+//       with `act_silu` q, k and v pass through silu (in float32) as they are staged.
 // q and k: [rows, groups, dk] in the run's type (head h reads group h / (heads / groups)); v: [rows, heads, dv].
 // out: float32 [rows, heads * dv].  Everything is float32 arithmetic on the ordinary pipes: the recurrence, its
 // decays and its state are not to be rounded to fewer bits.
@@ -208,6 +210,7 @@ extern "C" int braid_causal_conv(const void* x, long long x_stride, void* y, lon
 #define DECAY_CHANNEL 0
 #define DECAY_HEAD 1
 #define DECAY_GIVEN 2
+#define DECAY_CONST 3
 
 struct ScanArgs {
     const void* q; long long q_stride;
@@ -228,6 +231,7 @@ struct ScanArgs {
     int gate_is_decay;           // DECAY_CHANNEL: `gate` holds the decays themselves (braid_scan_decay), not their logits
     const float* kappa;          // DECAY_GIVEN: the factor on the key, [rows, heads] with row stride gate_stride
     int v_cols;                  // columns a head that v really holds (row stride v_stride); the rest of dv read as 1
+    int act_silu;                // DECAY_CONST: q, k and v are silu of what is given
 };
 
 // sigmoid(z)^(1 / tau) through log sigmoid(z) = min(z, 0) - log1p(exp(-|z|)): no overflow, full precision near one
@@ -294,6 +298,8 @@ linear_scan_kernel(ScanArgs a) {
         head_bias = to_f32(((const T*)a.gate_bias)[h]);
         if (a.skip) head_skip = to_f32(((const T*)a.skip)[h]);
     }
+    if (MODE == DECAY_CONST) head_a = ((const float*)a.gate)[h];
+    const bool silu = MODE == DECAY_CONST && a.act_silu;
     pdl_wait();
     const size_t per_head = (size_t)dk * dv;
     float* S_area = (float*)(a.state + (size_t)a.slot_ids[seq] * a.state_stride + a.state_offset) + (size_t)h * per_head;
@@ -352,8 +358,9 @@ linear_scan_kernel(ScanArgs a) {
 #pragma unroll
         for (int u = 0; u < NQ; ++u) {
             const int idx = tid + u * SCAN_THREADS;
-            sq[idx] = to_f32(pq[u]) * a.q_scale;
-            sk[idx] = to_f32(pk[u]);
+            const float q0 = to_f32(pq[u]), k0 = to_f32(pk[u]);
+            sq[idx] = (silu ? silu_f32(q0) : q0) * a.q_scale;
+            sk[idx] = silu ? silu_f32(k0) : k0;
             if (MODE == DECAY_CHANNEL) {
                 float av = pa[u];
                 if (!a.gate_is_decay) {
@@ -364,7 +371,10 @@ linear_scan_kernel(ScanArgs a) {
             }
         }
 #pragma unroll
-        for (int u = 0; u < NV; ++u) sv[tid + u * SCAN_THREADS] = to_f32(pv[u]);
+        for (int u = 0; u < NV; ++u) {
+            const float v0 = to_f32(pv[u]);
+            sv[tid + u * SCAN_THREADS] = silu ? silu_f32(v0) : v0;
+        }
         if (MODE == DECAY_HEAD && tid < nt) {
             const float x = to_f32(pg) + head_bias;
             const float dt = x > 20.f ? x : log1pf(expf(x));           // softplus
@@ -384,6 +394,10 @@ linear_scan_kernel(ScanArgs a) {
 #pragma unroll
                 for (int e = 0; e < R; e += 4)
                     *reinterpret_cast<float4*>(av + e) = *reinterpret_cast<const float4*>(sa + t * DKP + rg * R + e);
+            } else if (MODE == DECAY_CONST) {
+                hprod *= head_a;
+#pragma unroll
+                for (int e = 0; e < R; ++e) av[e] = head_a;
             } else {
                 const float ah = sah[t], kap = skap[t];
                 hprod *= ah;
@@ -485,15 +499,16 @@ extern "C" int braid_linear_scan(const void* q, long long q_stride, const void* 
                                  long long state_stride, long long state_offset, const int* q_start, const int* q_len,
                                  const int* slot_ids, int dtype, int mode, int n_seqs, int heads, int groups, int dk, int dv,
                                  float q_scale, float inv_tau, int max_q_len, int chunk, float* work, long long work_floats,
-                                 int gate_is_decay, const float* kappa, int v_cols, void* stream) {
+                                 int gate_is_decay, const float* kappa, int v_cols, int act_silu, void* stream) {
     if (n_seqs <= 0) return BRAID_OK;
     if (heads <= 0 || groups <= 0 || heads % groups) BRAID_REFUSE("linear_scan: %d heads do not divide into %d groups", heads, groups);
     if (dk <= 0 || dk > SCAN_MAX_DK || dv <= 0) BRAID_REFUSE("linear_scan: key size %d must be in (0, %d], value size %d positive", dk, SCAN_MAX_DK, dv);
     if (!state || (state_offset & 3) || (state_stride & 3)) BRAID_REFUSE("linear_scan: the state area must be given, in multiples of 4 bytes");
-    if (mode != DECAY_CHANNEL && mode != DECAY_HEAD && mode != DECAY_GIVEN) BRAID_REFUSE("linear_scan: unknown decay mode %d", mode);
+    if (mode != DECAY_CHANNEL && mode != DECAY_HEAD && mode != DECAY_GIVEN && mode != DECAY_CONST) BRAID_REFUSE("linear_scan: unknown decay mode %d", mode);
     if (mode == DECAY_GIVEN && !kappa) BRAID_REFUSE("linear_scan: given decays come with the factors on the keys");
     if (v_cols <= 0 || v_cols > dv) v_cols = dv;
     if (mode != DECAY_GIVEN && v_cols != dv) BRAID_REFUSE("linear_scan: value columns that read as 1 need given decays");
+    if (act_silu && mode != DECAY_CONST) BRAID_REFUSE("linear_scan: silu on what is given goes with a constant decay a head");
     if (mode == DECAY_HEAD && !a_log) BRAID_REFUSE("linear_scan: a decay per head needs A_log");
     if (dtype != BRAID_F32 && dtype != BRAID_BF16) BRAID_REFUSE("linear_scan: unknown dtype code %d", dtype);
     const int rg = scan_rg(dk), rr = scan_rows(dk);
@@ -506,7 +521,7 @@ extern "C" int braid_linear_scan(const void* q, long long q_stride, const void* 
     if (n_seqs > 65535 || (long long)n_dvt * max_chunks > 65535) BRAID_REFUSE("linear_scan: the step exceeds the grid limits");
     ScanArgs a{q, q_stride, k, k_stride, v, v_stride, gate, gate_stride, gate_bias, a_log, skip, out, out_stride,
                (uint8_t*)state, state_stride, state_offset, q_start, q_len, slot_ids, heads, groups, dk, dv, q_scale, inv_tau,
-               nullptr, nullptr, 0, chunk, max_chunks, gate_is_decay, kappa, v_cols};
+               nullptr, nullptr, 0, chunk, max_chunks, gate_is_decay, kappa, v_cols, act_silu};
     if (chunked) {
         a.wbuf = work;
         a.dbuf = work + (long long)n_seqs * max_chunks * heads * dk * dv;
@@ -525,10 +540,12 @@ extern "C" int braid_linear_scan(const void* q, long long q_stride, const void* 
     do {                                                                                                      \
         if (dtype == BRAID_F32 && mode == DECAY_CHANNEL) SCAN_LAUNCH_RG(float, DECAY_CHANNEL, GRID);          \
         else if (dtype == BRAID_F32 && mode == DECAY_HEAD) SCAN_LAUNCH_RG(float, DECAY_HEAD, GRID);           \
-        else if (dtype == BRAID_F32) SCAN_LAUNCH_RG(float, DECAY_GIVEN, GRID);                                \
+        else if (dtype == BRAID_F32 && mode == DECAY_GIVEN) SCAN_LAUNCH_RG(float, DECAY_GIVEN, GRID);         \
+        else if (dtype == BRAID_F32) SCAN_LAUNCH_RG(float, DECAY_CONST, GRID);                                \
         else if (mode == DECAY_CHANNEL) SCAN_LAUNCH_RG(__nv_bfloat16, DECAY_CHANNEL, GRID);                   \
         else if (mode == DECAY_HEAD) SCAN_LAUNCH_RG(__nv_bfloat16, DECAY_HEAD, GRID);                         \
-        else SCAN_LAUNCH_RG(__nv_bfloat16, DECAY_GIVEN, GRID);                                                \
+        else if (mode == DECAY_GIVEN) SCAN_LAUNCH_RG(__nv_bfloat16, DECAY_GIVEN, GRID);                       \
+        else SCAN_LAUNCH_RG(__nv_bfloat16, DECAY_CONST, GRID);                                                \
     } while (0)
     if (!chunked) {
         const dim3 grid(heads, n_seqs, n_dvt);
@@ -554,13 +571,16 @@ extern "C" int braid_linear_scan(const void* q, long long q_stride, const void* 
 // columns, each normed by its own root mean square:
 //   gate_first = 0:  out = y / rms(y) * w * silu(gate) * out_scale         (norm, then gate)
 //   gate_first = 1:  u = y * silu(gate);  out = u / rms(u) * w * out_scale (gate, then norm)
+// With `gate_sigmoid` the gate goes through a sigmoid instead of silu, in either order.
 // w has w_len numbers; column c of the row reads w[c % w_len] (w_len = group: one weight for every group;
 // w_len = width: a weight per column).  One warp per (row, group).  Everything in float32; out in the run's type.
+__device__ __forceinline__ float norm_gate(float z, int sigmoid) { return sigmoid ? 1.f / (1.f + expf(-z)) : silu_f32(z); }
+
 template <typename T>
 __global__ void __launch_bounds__(128)
 gated_norm_kernel(const float* __restrict__ y, const T* __restrict__ gate, long long gate_stride, const T* __restrict__ w,
                   int w_len, T* __restrict__ out, long long out_stride, const int* __restrict__ token_seq, int rows,
-                  int width, int group, int gate_first, float eps, float out_scale) {
+                  int width, int group, int gate_first, int gate_sigmoid, float eps, float out_scale) {
     pdl_trigger();
     pdl_wait();
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -574,14 +594,14 @@ gated_norm_kernel(const float* __restrict__ y, const T* __restrict__ gate, long 
     float ss = 0.f;
     for (int c = lane; c < group; c += 32) {
         float u = yr[c];
-        if (gate_first) u *= silu_f32(to_f32(gr[c]));
+        if (gate_first) u *= norm_gate(to_f32(gr[c]), gate_sigmoid);
         ss = fmaf(u, u, ss);
     }
     ss = warp_sum(ss);
     const float r = 1.f / sqrtf(ss / (float)group + eps);
     T* orow = out + (size_t)row * out_stride + (size_t)gi * group;
     for (int c = lane; c < group; c += 32) {
-        const float sg = silu_f32(to_f32(gr[c]));
+        const float sg = norm_gate(to_f32(gr[c]), gate_sigmoid);
         const float wv = to_f32(w[(gi * group + c) % w_len]);
         float u = yr[c];
         u = gate_first ? (u * sg) * r * wv : (u * r * wv) * sg;
@@ -595,7 +615,7 @@ template <typename T>
 __global__ void __launch_bounds__(128)
 gated_norm_block_kernel(const float* __restrict__ y, const T* __restrict__ gate, long long gate_stride, const T* __restrict__ w,
                         int w_len, T* __restrict__ out, long long out_stride, const int* __restrict__ token_seq, int rows,
-                        int width, int group, int gate_first, float eps, float out_scale) {
+                        int width, int group, int gate_first, int gate_sigmoid, float eps, float out_scale) {
     pdl_trigger();
     pdl_wait();
     __shared__ float red[32];
@@ -607,14 +627,14 @@ gated_norm_block_kernel(const float* __restrict__ y, const T* __restrict__ gate,
     float ss = 0.f;
     for (int c = threadIdx.x; c < group; c += blockDim.x) {
         float u = yr[c];
-        if (gate_first) u *= silu_f32(to_f32(gr[c]));
+        if (gate_first) u *= norm_gate(to_f32(gr[c]), gate_sigmoid);
         ss = fmaf(u, u, ss);
     }
     ss = block_sum(ss, red);
     const float r = 1.f / sqrtf(ss / (float)group + eps);
     T* orow = out + (size_t)row * out_stride + (size_t)gi * group;
     for (int c = threadIdx.x; c < group; c += blockDim.x) {
-        const float sg = silu_f32(to_f32(gr[c]));
+        const float sg = norm_gate(to_f32(gr[c]), gate_sigmoid);
         const float wv = to_f32(w[(gi * group + c) % w_len]);
         float u = yr[c];
         u = gate_first ? (u * sg) * r * wv : (u * r * wv) * sg;
@@ -624,7 +644,7 @@ gated_norm_block_kernel(const float* __restrict__ y, const T* __restrict__ gate,
 
 extern "C" int braid_gated_norm(const float* y, const void* gate, long long gate_stride, const void* w, int w_len, void* out,
                                 long long out_stride, const int* token_seq, int dtype, int rows, int width, int group,
-                                int gate_first, float eps, float out_scale, void* stream) {
+                                int gate_first, int gate_sigmoid, float eps, float out_scale, void* stream) {
     if (rows <= 0) return BRAID_OK;
     if (width <= 0 || group <= 0 || width % group) BRAID_REFUSE("gated_norm: width %d is not a whole number of groups of %d", width, group);
     if (w_len <= 0) BRAID_REFUSE("gated_norm: the weight has no numbers");
@@ -635,20 +655,20 @@ extern "C" int braid_gated_norm(const float* y, const void* gate, long long gate
     if (group > 128 && items <= 0x7fffffffLL) {
         if (dtype == BRAID_F32)
             braid_launch(gated_norm_block_kernel<float>, dim3((int)items), dim3(128), 0, s, y, (const float*)gate, gate_stride,
-                         (const float*)w, w_len, (float*)out, out_stride, token_seq, rows, width, group, gate_first, eps, out_scale);
+                         (const float*)w, w_len, (float*)out, out_stride, token_seq, rows, width, group, gate_first, gate_sigmoid, eps, out_scale);
         else if (dtype == BRAID_BF16)
             braid_launch(gated_norm_block_kernel<__nv_bfloat16>, dim3((int)items), dim3(128), 0, s, y, (const __nv_bfloat16*)gate,
                          gate_stride, (const __nv_bfloat16*)w, w_len, (__nv_bfloat16*)out, out_stride, token_seq, rows, width, group,
-                         gate_first, eps, out_scale);
+                         gate_first, gate_sigmoid, eps, out_scale);
         else BRAID_REFUSE("gated_norm: unknown dtype code %d", dtype);
         BRAID_LAUNCH_CHECK();
     }
     if (dtype == BRAID_F32)
         braid_launch(gated_norm_kernel<float>, dim3((int)blocks), dim3(128), 0, s, y, (const float*)gate, gate_stride, (const float*)w,
-                     w_len, (float*)out, out_stride, token_seq, rows, width, group, gate_first, eps, out_scale);
+                     w_len, (float*)out, out_stride, token_seq, rows, width, group, gate_first, gate_sigmoid, eps, out_scale);
     else if (dtype == BRAID_BF16)
         braid_launch(gated_norm_kernel<__nv_bfloat16>, dim3((int)blocks), dim3(128), 0, s, y, (const __nv_bfloat16*)gate, gate_stride,
-                     (const __nv_bfloat16*)w, w_len, (__nv_bfloat16*)out, out_stride, token_seq, rows, width, group, gate_first, eps, out_scale);
+                     (const __nv_bfloat16*)w, w_len, (__nv_bfloat16*)out, out_stride, token_seq, rows, width, group, gate_first, gate_sigmoid, eps, out_scale);
     else BRAID_REFUSE("gated_norm: unknown dtype code %d", dtype);
     BRAID_LAUNCH_CHECK();
 }

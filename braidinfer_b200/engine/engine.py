@@ -139,6 +139,8 @@ class Engine:
                 x.normal_(0.0, ts.std, generator=g)
                 if ts.init == "one_plus_normal":
                     x += 1.0
+                elif ts.init == "eye_plus_normal":
+                    x += torch.eye(ts.shape[0], dtype=x.dtype, device=dev)
                 tensors[name] = x if run_dtype == torch.bfloat16 else x.float()
         else:
             drawn = draw_tensors(specs, seed, torch.bfloat16)

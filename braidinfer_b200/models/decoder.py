@@ -9,7 +9,8 @@ from typing import Dict, List, Optional, Tuple
 
 import torch
 
-from ..parts.base import BLOCKS, EMBEDDINGS, FEED_FORWARDS, HEADS, INJECTIONS, LAYER_INPUTS, MIXERS, NORMS
+from ..parts.base import (BLOCKS, CONNECTIONS, EMBEDDINGS, FEED_FORWARDS, HEADS, INJECTIONS, LAYER_INPUTS, MIXERS, NORMS,
+                          STREAMS)
 from ..parts.spec import CacheRequest, ModelSpec, TensorSpec
 
 
@@ -30,10 +31,17 @@ class DecoderModel:
             block = BLOCKS.get(ls.block)(mixer, mixer_norm, ffn, ffn_norm)
             if ls.layer_input is not None:
                 block.layer_input = LAYER_INPUTS.get(ls.layer_input.kind)(ls.layer_input.params, ls.prefix, runtime)
+            for what in ("mixer_connection", "feed_forward_connection"):
+                cs = getattr(ls, what)
+                if cs is not None:
+                    setattr(block, what, CONNECTIONS.get(cs.kind)(cs.params, ls.prefix, runtime))
             self.blocks.append(block)
         self.injection = None
         if spec.injection is not None:
             self.injection = INJECTIONS.get(spec.injection.kind)(spec.injection.params, "", runtime)
+        self.streams = None
+        if spec.streams is not None:
+            self.streams = STREAMS.get(spec.streams.kind)(spec.streams.params, "", runtime)
         # the embedding's output must outlive the layers, which add into the stream in place
         self._keep_h0 = any(e.inject for e in spec.schedule)
         self.final_norm = NORMS.get(spec.final_norm.kind)(spec.final_norm.params, "", runtime)
@@ -44,6 +52,8 @@ class DecoderModel:
         yield self.embedding
         if self.injection is not None:
             yield self.injection
+        if self.streams is not None:
+            yield self.streams
         for b in self.blocks:
             yield from b.parts()
         yield self.final_norm
@@ -80,7 +90,8 @@ class DecoderModel:
         """Run the step's tokens through the schedule; return float32 logits
         [wanted rows, vocab] (None when nothing is wanted).  `tap(i, h)`, if given, is shown
         the float32 residual stream [rows, width] after the embedding (i = 0) and after
-        schedule entry i - 1 (sums that a part left deferred are completed first)."""
+        schedule entry i - 1 (sums that a part left deferred are completed first; several streams are shown as one,
+        `Streams.total`)."""
         if self.embedding.uses_positions:
             h = self.embedding.forward(ctx.token_ids, ctx.rows, positions=ctx.positions)
         else:
@@ -88,6 +99,8 @@ class DecoderModel:
         if tap is not None:
             tap(0, h)
         h0 = h.clone() if self._keep_h0 else None
+        if self.streams is not None:
+            h = self.streams.open(h)
         for e, entry in enumerate(self.spec.schedule):
             if entry.inject:
                 h = self.injection.forward(ctx.resolve(h), h0, ctx)
@@ -96,10 +109,12 @@ class DecoderModel:
                 view.page_table = ctx.page_tables[view.group]
             h = self.blocks[entry.layer].forward(h, ctx, view, cache.state_view(e))
             if tap is not None:
-                tap(e + 1, ctx.resolve(h))
+                tap(e + 1, ctx.resolve(h) if self.streams is None else self.streams.total(h, ctx))
         if ctx.n_want == 0:
             ctx.drop_deferred()
             return None
+        if self.streams is not None:
+            return self.head.forward(self.streams.close(h, self.final_norm, ctx, ctx.want_rows, ctx.n_want))
         if not self.final_norm.accepts_deferred:
             ctx.resolve(h)
         x = self.final_norm.forward(h, ctx, row_index=ctx.want_rows, rows=ctx.n_want)

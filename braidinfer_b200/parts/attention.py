@@ -30,7 +30,14 @@ Options that other designs use, each off unless named:
                     p'_h = sum_g T[h, g] p_g; head h applies p'_h to the values of its own kv head.  The mix is linear, so
                     every head's own probabilities are applied to the values of every kv head (the attention kernels'
                     `value_heads`) and the results are mixed afterwards, out_h = sum_g T[h, g] O[g, kv(h)] (`head_mix`)
-unit_qk_eps, q_temp and value_dim without rotation are for heads that are not rotated (position encoding "none"): one kernel norms, scales and
+    qkv_bias        q, k and v get a bias each (stored under the projection's name with ".b" added)
+    proj_norm       {"eps", "q_name", "k_name"}: ONE RMS norm over all query heads of a token together and one over all its
+                    key heads, before they count as heads, with a plain weight a column
+    unit_v_eps      every value head is divided by its root mean square, sqrt(mean(x^2) + eps), no weight, and cached so
+    distance_bias   {"slope", "rate"} (tensor names, num_heads numbers each, r1 and r2): r1 ln(1 + r2 (p - j)) comes off the
+                    scaled score of key j at position p, float32 (the logarithmic kernel of Chi, Fan, Ramadge, Rudnicky:
+                    "KERPLE: Kernelized Relative Positional Embedding for Length Extrapolation", 2022)
+unit_qk_eps, q_temp, qkv_bias, proj_norm, unit_v_eps and value_dim without rotation are for heads that are not rotated (position encoding "none"): one kernel norms, scales and
 stores.  Keys, values and queries are then padded with zeros to one head size that the attention kernels take
 (max(head_dim, value_dim), rounded up to 16), which changes no score and no result.  Rotated heads whose value
 size differs from head_dim (or whose size is no multiple of 16) get the same padding from rows of zeros in the
@@ -53,7 +60,8 @@ class GQAAttention(Mixer):
     """params: hidden_size, num_heads, num_kv_heads, head_dim, window (int | None),
     position_encoding (PartSpec), and tensor names q_proj, k_proj, v_proj, o_proj; optional qk_norm
     ({"eps", "q_name", "k_name"}), value_from_key (bool), scale, sink (a score), out_mult, sink_name, head_gate,
-    unit_qk_eps, q_temp ({"coef", "every"}), value_dim, keep_first, head_scale (a tensor name), talk (a tensor name)."""
+    unit_qk_eps, q_temp ({"coef", "every"}), value_dim, keep_first, head_scale (a tensor name), talk (a tensor name), qkv_bias,
+    proj_norm ({"eps", "q_name", "k_name"}), unit_v_eps, distance_bias ({"slope", "rate"})."""
 
     plain_output = True
 
@@ -78,7 +86,17 @@ class GQAAttention(Mixer):
         # heads that are normed without weights, scaled by position or of two sizes go through the kernel that
         # pads them to one size
         gated = p.get("head_gate") is not None
-        self.prep = (self.unit_qk_eps is not None or self.q_temp is not None or (self.vd != self.hd and pe.kind == "none")
+        pn = p.get("proj_norm")
+        self.proj_norm = (float(pn["eps"]), prefix + pn["q_name"], prefix + pn["k_name"]) if pn else None
+        self.unit_v_eps = float(p["unit_v_eps"]) if p.get("unit_v_eps") is not None else None
+        # what the kernel that works on whole projections does (biases, norms over all heads, values of unit size)
+        self.whole_proj = bool(p.get("qkv_bias")) or self.proj_norm is not None or self.unit_v_eps is not None
+        if self.whole_proj and (self.unit_qk_eps is not None or self.q_temp):
+            raise ValueError("gqa_attention: biases, norms of whole projections and unit values do not go with unit heads or a "
+                             "query temperature")
+        if self.proj_norm and self.unit_v_eps is not None and self.proj_norm[0] != self.unit_v_eps:
+            raise ValueError("gqa_attention: the norms of whole projections and of values have one eps")
+        self.prep = (self.whole_proj or self.unit_qk_eps is not None or self.q_temp is not None or (self.vd != self.hd and pe.kind == "none")
                      or (gated and pe.kind == "none"))
         if gated and not self.prep and not (p.get("qk_norm") is not None or self.value_from_key):
             raise ValueError("gqa_attention: a gate a head rides in the stacked product, which the plain rotation kernels "
@@ -119,6 +137,11 @@ class GQAAttention(Mixer):
             names.append(prefix + p["head_gate"])
             outs.append(self.nqh)
         self.qkv = Linear(runtime, names, outs, self.hidden)
+        self.bias_names = [n + ".b" for n in names[:3]] if p.get("qkv_bias") else None
+        self.bias_sizes = outs[:3]
+        db = p.get("distance_bias")
+        self.distance_bias_names = (prefix + db["slope"], prefix + db["rate"]) if db else None
+        self.biases = self.distance_bias = self.proj_norm_w = None
         self.o = Linear(runtime, [prefix + p.get("o_proj", "self_attn.o_proj.weight")], [self.hidden],
                         self.nqh * self.vd)
         self.sink_name = prefix + p["sink_name"] if p.get("sink_name") is not None else None
@@ -147,6 +170,14 @@ class GQAAttention(Mixer):
             d[self.head_scale_name] = TensorSpec((self.nqh,), init="one_plus_normal", std=0.1)
         if self.talk_name:
             d[self.talk_name] = TensorSpec((self.nqh, self.nqh), std=0.3)
+        if self.bias_names:
+            d.update({n: TensorSpec((size,)) for n, size in zip(self.bias_names, self.bias_sizes)})
+        if self.proj_norm:
+            d[self.proj_norm[1]] = TensorSpec((self.nqh * self.hd,), init="one_plus_normal")
+            d[self.proj_norm[2]] = TensorSpec((self.nkh * self.hd,), init="one_plus_normal")
+        if self.distance_bias_names:
+            for n in self.distance_bias_names:
+                d[n] = TensorSpec((self.nqh,), init="one_plus_normal", std=0.1)
         return d
 
     def load(self, tensors) -> None:
@@ -173,6 +204,12 @@ class GQAAttention(Mixer):
             self.talk = tensors[self.talk_name].contiguous()
         if self.qk_norm:
             self.q_norm_w, self.k_norm_w = tensors[self.qk_norm[1]], tensors[self.qk_norm[2]]
+        if self.bias_names:
+            self.biases = tuple(tensors[n] for n in self.bias_names)
+        if self.proj_norm:
+            self.proj_norm_w = (tensors[self.proj_norm[1]], tensors[self.proj_norm[2]])
+        if self.distance_bias_names:         # scores are float32 in every run
+            self.distance_bias = tuple(tensors[n].float().contiguous() for n in self.distance_bias_names)
         if self.sink_name:
             self.head_sinks = tensors[self.sink_name].float().contiguous()       # scores are float32 in every run
 
@@ -216,20 +253,26 @@ class GQAAttention(Mixer):
 
     def _project(self, out, residual, ctx):
         if residual is None:
-            return self.o.forward(out, out_dtype=torch.float32)
+            # a block that does not add deferred sums up itself resolves this one
+            return self.o.forward(out, out_dtype=torch.float32, defer_to=ctx)
         return self.o.forward(out, residual=residual, defer_to=ctx)
 
     def _forward_padded(self, qkv, gate, residual, ctx, cache):
-        """Heads without rotation: norm, temperature and the padding to one head size in one kernel, attention over
+        """Heads without rotation: biases, norms, temperature and the padding to one head size in one kernel, attention over
         the padded heads, then the value columns alone go on to the output product."""
         K = self.rt.kernels
         rows, D = qkv.shape[0], self.hd_pad
         q = self.rt.empty(rows, self.nqh * D)
         coef, every = self.q_temp if self.q_temp else (0.0, 0)
         write = cache is not None and not cache.read_only
-        K.head_prep_kv(qkv, q, ctx.positions, ctx.token_seq, cache.page_table if write else None,
-                       cache.storage if write else None, self.nqh, self.nkh, self.hd, self.vd, D,
-                       self.unit_qk_eps is not None, self.unit_qk_eps or 0.0, coef, every)
+        where = (ctx.positions, ctx.token_seq, cache.page_table if write else None, cache.storage if write else None,
+                 self.nqh, self.nkh, self.hd, self.vd, D)
+        if self.whole_proj:
+            q_w, k_w = self.proj_norm_w if self.proj_norm else (None, None)
+            K.proj_prep_kv(qkv, q, *where, self.proj_norm[0] if self.proj_norm else self.unit_v_eps or 0.0, q_w=q_w, k_w=k_w,
+                           biases=self.biases, v_unit=self.unit_v_eps is not None)
+        else:
+            K.head_prep_kv(qkv, q, *where, self.unit_qk_eps is not None, self.unit_qk_eps or 0.0, coef, every)
         out = self.rt.empty(rows, self.nqh * D)
         self._attend(q, out, ctx, cache, D, gate)
         if D != self.vd:
@@ -252,13 +295,15 @@ class GQAAttention(Mixer):
             K.attn_simple(qkv, out, cache.storage, cache.page_table, ctx.positions, ctx.token_seq,
                           self.nqh, self.nkh, hd, cache.page_size, self.window, self.scale, sink=self.sink,
                           head_sinks=self.head_sinks, head_gate=gate, out_scale=self.out_mult,
-                          keep_first=self.keep_first, head_scale=self.head_scale, value_heads=value_heads)
+                          keep_first=self.keep_first, head_scale=self.head_scale, value_heads=value_heads,
+                          distance_bias=self.distance_bias)
             return
         few = ctx.max_q_len <= 8
         if not few and self.rt.attention_backend == "auto" and K.attn_tc_supports(hd) and not extras:
             K.attn_tc(qkv, out, cache.storage, cache.page_table, ctx.q_start, ctx.q_len, ctx.kv_before,
                       ctx.n_seqs, ctx.max_q_len, self.nqh, self.nkh, hd, self.window, self.scale, sink=self.sink,
-                      head_sinks=self.head_sinks, head_gate=gate, out_scale=self.out_mult)
+                      head_sinks=self.head_sinks, head_gate=gate, out_scale=self.out_mult,
+                      distance_bias=self.distance_bias)
             return
         n_splits = 1
         if few:
@@ -272,4 +317,4 @@ class GQAAttention(Mixer):
                    ctx.n_seqs, ctx.max_q_len, self.nqh, self.nkh, hd, self.window, self.scale,
                    n_splits=n_splits, few_tokens=few, sink=self.sink, head_sinks=self.head_sinks, head_gate=gate,
                    out_scale=self.out_mult, keep_first=self.keep_first, head_scale=self.head_scale,
-                   value_heads=value_heads)
+                   value_heads=value_heads, distance_bias=self.distance_bias)

@@ -151,6 +151,27 @@ class LayerInput(Part):
         raise NotImplementedError
 
 
+class Connection(Part):
+    """How one sublayer reads several residual streams and writes its result back into them; the numbers are the part's,
+    the arithmetic is done by the streams' value itself (see parts/hyper.py)."""
+
+
+class Streams(Part):
+    """Several residual streams instead of one.  Blocks that name this form get its value as `h`."""
+
+    def open(self, h: torch.Tensor):
+        """The embedding's output [rows, width] float32 -> the streams' value that the first layer gets."""
+        raise NotImplementedError
+
+    def total(self, value, ctx) -> torch.Tensor:
+        """One row a token [rows, width] float32: what a tap is shown after a layer's run (`value` is left usable)."""
+        raise NotImplementedError
+
+    def close(self, value, norm: Norm, ctx, row_index: torch.Tensor, rows: int) -> torch.Tensor:
+        """The model's final norm of the wanted rows of the streams made one."""
+        raise NotImplementedError
+
+
 class Block:
     """The arrangement of a layer's parts.  `forward(h, ctx, cache, state) -> h` runs them on
     the float32 residual stream; `cache` and `state` are the mixer's (see Mixer.forward).
@@ -164,10 +185,13 @@ class Block:
         self.feed_forward = feed_forward
         self.feed_forward_norm = feed_forward_norm
         self.layer_input = layer_input
+        # how the sublayers read several residual streams and write back (LayerSpec.mixer_connection); None: one stream
+        self.mixer_connection: Optional[Connection] = None
+        self.feed_forward_connection: Optional[Connection] = None
 
     def parts(self):
-        return [p for p in (self.mixer_norm, self.mixer, self.feed_forward_norm, self.feed_forward, self.layer_input)
-                if p is not None]
+        return [p for p in (self.mixer_norm, self.mixer, self.feed_forward_norm, self.feed_forward, self.layer_input,
+                            self.mixer_connection, self.feed_forward_connection) if p is not None]
 
     def forward(self, h: torch.Tensor, ctx, cache, state) -> torch.Tensor:
         raise NotImplementedError
@@ -207,3 +231,5 @@ EMBEDDINGS = Registry("embedding")
 HEADS = Registry("head")
 INJECTIONS = Registry("injection")
 LAYER_INPUTS = Registry("layer input")
+STREAMS = Registry("residual streams")
+CONNECTIONS = Registry("connection")

@@ -9,6 +9,9 @@ own about each token (`LayerSpec.layer_input`) applies it last: h = layer_input(
 "sublayer_norm_residual": h = h + norm(mixer(h)); h = h + norm(feed_forward(h)): the sublayers read the stream
 itself (cast to the run's type) and the norm is applied to what they return, before the residual sum.  The norm
 and the sum are one float32 kernel (`Norm.add_into`).
+
+"hyper_connected": several residual streams; each sublayer reads a weighted sum of them and its result goes back into
+all of them, which are mixed with one another on the way (parts/hyper.py).
 """
 from __future__ import annotations
 
@@ -66,3 +69,24 @@ class SublayerNormResidualBlock(Block):
             rt.kernels.cast(h, x)
         y = call(x, None if part.plain_output else torch.zeros_like(h))
         return ctx.resolve(y)
+
+
+@BLOCKS.register("hyper_connected")
+class HyperConnectedBlock(Block):
+    """h is a `StreamValue` (parts/hyper.py).  A sublayer's result is left as it comes (finished rows, a deferred sum, the
+    outputs of a token's experts): the kernel that writes it back into the streams, which is the one that also reads
+    them for the next sublayer and norms that, adds it up.  Mixer and feed-forward need `plain_output`."""
+
+    def forward(self, h, ctx, cache, state):
+        for p in (self.mixer, self.feed_forward):
+            if p is not None and not p.plain_output:
+                raise RuntimeError(f"{type(p).__name__} cannot return its result alone, which hyper-connected layers need")
+        x = h.read(self.mixer_connection, self.mixer_norm, ctx)
+        h.give(self.mixer.forward(x, None, ctx, cache, state), self.mixer_connection)
+        if self.feed_forward is not None:
+            x = h.read(self.feed_forward_connection, self.feed_forward_norm, ctx)
+            unsummed = getattr(self.feed_forward, "forward_unsummed", None)
+            h.give(unsummed(x, ctx) if unsummed else self.feed_forward.forward(x, None, ctx), self.feed_forward_connection)
+        if self.layer_input is not None:
+            raise RuntimeError("a layer's own token input works on one residual stream")
+        return h

@@ -21,7 +21,9 @@ chosen scores' sum is the softmax over the chosen logits alone, so routers that 
 mode of their own.  `scoring: "sigmoid"` scores every expert by itself, s = 1 / (1 + exp(-z)), and the chosen experts'
 weights are their scores as they are.  `weight_on: "input"` lets the weight multiply what the expert reads instead
 of what it returns, out = sum_k expert_k(w_k x); the first products being linear, the weight is applied to their
-float32 results before the activation.  `shared` is a feed-forward part that every token also runs through (its
+float32 results before the activation.  `normalize: False` leaves the chosen softmax scores as the weights, undivided.
+`correction` names a stored number an expert that is added to the scores for the choice alone; the weights are the scores
+without it (as in DeepSeek-AI, "DeepSeek-V3 Technical Report", 2024, to even out the experts' loads).  `shared` is a feed-forward part that every token also runs through (its
 result is added like an expert's with weight 1).
 """
 from __future__ import annotations
@@ -39,8 +41,8 @@ from .spec import PartSpec, TensorSpec
 class MixtureOfExperts(FeedForward):
     """params: hidden_size, intermediate_size (of one expert), experts, top, groups (default 1), keep
     (groups kept, default all), out_mult (default 1), gated (default True), activation ("silu" with a gate, "relu2"
-    without), scoring ("softmax" | "sigmoid"), weight_on ("output" | "input"), shared (a PartSpec of a feed-forward, or
-    None), and tensor names: router, and expert_gate, expert_up, expert_down as patterns with `{e}` for the expert's
+    without), scoring ("softmax" | "sigmoid"), weight_on ("output" | "input"), normalize (softmax scores over their sum;
+    default True), correction (a tensor name, or None), shared (a PartSpec of a feed-forward, or None), and tensor names: router, and expert_gate, expert_up, expert_down as patterns with `{e}` for the expert's
     number."""
 
     plain_output = True
@@ -66,6 +68,11 @@ class MixtureOfExperts(FeedForward):
             raise ValueError(f"moe: scoring {self.scoring!r} (softmax or sigmoid), weight_on {self.weight_on!r} (output or input)")
         if self.weight_on == "input" and not self.gated:
             raise ValueError("moe: a weight on the expert's input is built for gated experts")
+        self.normalize = bool(p.get("normalize", self.scoring == "softmax"))
+        self.correction_name = prefix + p["correction"] if p.get("correction") is not None else None
+        self.correction = None
+        if self.correction_name and self.groups != 1:
+            raise ValueError("moe: a correction of the choice is built for experts in one group")
         sh: PartSpec = p.get("shared")
         self.shared = FEED_FORWARDS.get(sh.kind)(sh.params, prefix, runtime) if sh is not None else None
         if self.experts % self.groups:
@@ -87,12 +94,16 @@ class MixtureOfExperts(FeedForward):
                 d[self.gate_names[e]] = TensorSpec((self.inter, self.hidden))
             d[self.up_names[e]] = TensorSpec((self.inter, self.hidden))
             d[self.down_names[e]] = TensorSpec((self.hidden, self.inter))
+        if self.correction_name:
+            d[self.correction_name] = TensorSpec((self.experts,))
         if self.shared is not None:
             d.update(self.shared.tensor_specs())
         return d
 
     def load(self, tensors) -> None:
         self.router.load(tensors)
+        if self.correction_name:
+            self.correction = tensors[self.correction_name].float().contiguous()     # routing is float32 in every run
         if self.shared is not None:
             self.shared.load(tensors)
         if self.gated:
@@ -105,12 +116,29 @@ class MixtureOfExperts(FeedForward):
         return 16 if rows * self.top <= 16 * self.experts else 64
 
     def forward(self, x, residual, ctx):
+        y, plan, wgt, top = self._run(x, ctx)
+        if residual is None:
+            residual = torch.zeros((x.shape[0], self.hidden), dtype=torch.float32, device=x.device)
+        self.rt.kernels.moe_combine(residual, y, plan, wgt, top=top)
+        if self.shared is not None:
+            residual = self.shared.forward(x, residual, ctx)
+        return residual
+
+    def forward_unsummed(self, x, ctx):
+        """For blocks that add the chosen experts' outputs up in a kernel of their own: (outputs [slots, hidden], the
+        plan, weights [rows, top] | None for 1, top).  With an expert that every token uses: the finished rows."""
+        if self.shared is not None:
+            return self.forward(x, None, ctx)
+        return self._run(x, ctx)
+
+    def _run(self, x, ctx):
         K = self.rt.kernels
         rows = x.shape[0]
         logits = self.router.forward(x, out_dtype=torch.float32)
         idx = torch.empty((rows, self.top), dtype=torch.int32, device=x.device)
         wgt = torch.empty((rows, self.top), dtype=torch.float32, device=x.device)
-        K.moe_route(logits, idx, wgt, self.groups, self.keep, mult=self.out_mult, sigmoid=self.scoring == "sigmoid")
+        K.moe_route(logits, idx, wgt, self.groups, self.keep, mult=self.out_mult, sigmoid=self.scoring == "sigmoid",
+                    renorm=self.normalize, correction=self.correction)
         tile = self.tile(rows)
         plan = K.moe_plan(idx, ctx.token_seq, self.experts, tile)
         slots = plan[4] * tile
@@ -118,12 +146,7 @@ class MixtureOfExperts(FeedForward):
         y = self.rt.empty(slots, self.hidden)
         on_input = self.weight_on == "input"
         self._experts(x, act, y, plan, tile, wgt if on_input else None)
-        if residual is None:
-            residual = torch.zeros((rows, self.hidden), dtype=torch.float32, device=x.device)
-        K.moe_combine(residual, y, plan, None if on_input else wgt, top=self.top)
-        if self.shared is not None:
-            residual = self.shared.forward(x, residual, ctx)
-        return residual
+        return y, plan, None if on_input else wgt, self.top
 
     def _experts(self, x, act, y, plan, tile, in_wgt=None) -> None:
         """bfloat16 rows that start on 16 bytes run on the tensor cores, everything else on the plain kernels."""

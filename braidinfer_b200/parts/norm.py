@@ -9,6 +9,8 @@ RMSNorm: y = x * rsqrt(mean(x^2) + eps) * w, plain w
 crates/braidinfer-runtime/src/config.rs:552).  Reads the float32 residual stream, writes
 the run's element type; the sum of squares and the scale are float32.  With `offset` the stored weight w is
 zero-centred and applied as offset + w (offset 1: y = x * rsqrt(mean(x^2) + eps) * (1 + w)), added in float32.
+With `scalar` the stored weight is one number that every column is multiplied by (it is spread over the columns when it
+is loaded, so every kernel that fuses the norm serves it).
 `add_into(y, h)` norms a branch's float32 result y and adds it to the float32 stream h in one kernel, for
 layers that norm what a sublayer returns instead of what it reads."""
 from __future__ import annotations
@@ -24,7 +26,8 @@ from .spec import TensorSpec
 
 @NORMS.register("rmsnorm")
 class RMSNorm(Norm):
-    """params: width, eps, name (tensor name under the prefix), offset (added to the stored weight; default 0)."""
+    """params: width, eps, name (tensor name under the prefix), offset (added to the stored weight; default 0), scalar (one
+    stored number instead of one a column; default False)."""
 
     accepts_deferred = True      # adds a deferred residual sum in the same kernel as the norm
 
@@ -34,12 +37,13 @@ class RMSNorm(Norm):
         self.eps = float(params["eps"])
         self.name = prefix + params["name"]
         self.offset = float(params.get("offset", 0.0))
+        self.scalar = bool(params.get("scalar", False))
         if self.offset:
             self.accepts_deferred = False        # the kernels that add up partial sums apply plain weights
         self.weight: Optional[torch.Tensor] = None
 
     def tensor_specs(self) -> Dict[str, TensorSpec]:
-        return {self.name: TensorSpec((self.width,), init="normal" if self.offset else "one_plus_normal")}
+        return {self.name: TensorSpec(() if self.scalar else (self.width,), init="normal" if self.offset else "one_plus_normal")}
 
     def add_into(self, y: torch.Tensor, h: torch.Tensor, ctx=None) -> torch.Tensor:
         """h += norm(y), both float32 [rows, width]; returns h."""
@@ -47,7 +51,8 @@ class RMSNorm(Norm):
         return h
 
     def load(self, tensors) -> None:
-        self.weight = tensors[self.name]
+        w = tensors[self.name]
+        self.weight = w.reshape(1).expand(self.width).contiguous() if self.scalar else w
 
     def forward(self, x: torch.Tensor, ctx=None, row_index: Optional[torch.Tensor] = None,
                 rows: Optional[int] = None, reader_takes_row_scale: bool = False) -> torch.Tensor:

@@ -27,6 +27,9 @@ class LayerSpec:
     mixer_norm: PartSpec
     feed_forward: Optional[PartSpec] = None
     feed_forward_norm: Optional[PartSpec] = None
+    # for blocks that keep several residual streams: how each sublayer reads them and writes back (registry CONNECTIONS)
+    mixer_connection: Optional[PartSpec] = None
+    feed_forward_connection: Optional[PartSpec] = None
     # a part (registry LAYER_INPUTS) that the block applies to the stream after its other parts: something the
     # layer reads about each token beside the stream
     layer_input: Optional[PartSpec] = None
@@ -59,10 +62,15 @@ class ModelSpec:
     # that ask for it (`ScheduleEntry.inject`): a block of layers that runs several times in a row, for one,
     # is fed the stream and the embedding's output anew at the start of every pass.
     injection: Optional[PartSpec] = None
+    # A part (registry STREAMS) that turns the embedding's output into several residual streams before the first layer and
+    # back into one after the last, for blocks that work on such streams.
+    streams: Optional[PartSpec] = None
 
     def validate(self) -> None:
         if self.injection is None and any(e.inject for e in self.schedule):
             raise ValueError("a schedule entry asks for the injection, and the model has none")
+        if self.streams is not None and self.injection is not None:
+            raise ValueError("an injection works on one residual stream, and the model keeps several")
         for i, e in enumerate(self.schedule):
             if not (0 <= e.layer < len(self.layers)):
                 raise ValueError(f"schedule entry {i} names layer {e.layer}, which does not exist")
@@ -82,7 +90,7 @@ class TensorSpec:
     """A tensor that a part needs from the model folder.
 
     `init` tells the random-weights mode how to draw it: "normal" is N(0, std),
-    "one_plus_normal" is 1 + N(0, std).  A shape of () is one stored scalar.  `integer` marks index tables, which are
+    "one_plus_normal" is 1 + N(0, std), "eye_plus_normal" (square matrices) the identity + N(0, std).  A shape of () is one stored scalar.  `integer` marks index tables, which are
     kept as int32 whatever the run's dtype.
     """
     shape: Tuple[int, ...]

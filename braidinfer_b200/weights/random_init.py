@@ -2,7 +2,8 @@
 from a configuration and a seed.
 
 Tensors are drawn on the CPU from one seeded generator in the order the model lists
-them: matrices and the embedding N(0, 0.02), norm weights 1 + N(0, 0.02), drawn in
+them: matrices and the embedding N(0, 0.02), norm weights 1 + N(0, 0.02), matrices that mix residual streams the
+identity + N(0, 0.02), drawn in
 float32 and stored in bfloat16.  The same configuration and seed give the same bytes.
 """
 from __future__ import annotations
@@ -39,6 +40,8 @@ def draw_tensors(specs: Mapping[str, TensorSpec], seed: int, dtype: torch.dtype 
         x = torch.randn(ts.shape, generator=g, dtype=torch.float32) * ts.std
         if ts.init == "one_plus_normal":
             x = x + 1.0
+        elif ts.init == "eye_plus_normal":
+            x = x + torch.eye(ts.shape[0])
         elif ts.init != "normal":
             raise ValueError(f"unknown init {ts.init!r} for {name}")
         out[name] = x.to(dtype)
