@@ -1597,6 +1597,250 @@ def ludazen_kernels(z, T, B, C, timed, frac):
     return res
 
 
+# ------------------------------------------------------------------ the Zisesun decoder beside the Birepel one
+ZISESUN_STREAMS = 4
+
+
+def zisesun_config(z):
+    """Attention and lightning layers in turn at the sizes of `LODUZEN_SIZES`: the attention heads and the window of that
+    model's attention, the lightning heads of its linear attention, four residual streams, and in every layer eight gated
+    experts of which two serve a token, sized so that a token's products equal the dense unit's."""
+    att = {"heads": z["heads"], "kv_heads": z["kv"], "dim": z["dim"], "vdim": z["dim"], "scale": z["dim"] ** -0.5,
+           "mask": {"size": z["window"]}}
+    mem = {"heads": z["lheads"], "dim": z["ldk"], "vdim": z["ldv"], "decay": [1.0 - 2.0 ** -(3 + h) for h in range(z["lheads"])]}
+    moe = {"kind": "moe", "expert": {"ff": z["ff"] // 2 // 64 * 64}, "router": {"experts": 8, "top": 2}}
+    return {"architecture": "Zisesun", "vocab": z["vocab"], "width": z["width"], "streams": ZISESUN_STREAMS, "max_positions": 16384,
+            "norm": {"eps": 1e-6},
+            "layers": [{"type": "attention", "mixer": att, "mlp": moe} if i % 2 == 0 else {"type": "lightning", "mixer": mem, "mlp": moe}
+                       for i in range(z["layers"])]}
+
+
+def birepel_twin_config(z):
+    """The Birepel decoder with experts in every layer: as many, as many a token, and (without a gate's matrix) half as wide again, so
+    that a token's products and the stored weights equal those of `zisesun_config`."""
+    cfg = birepel_config(z)
+    moe = cfg["layers"][1]["mlp"]
+    return dict(cfg, layers=[dict(L, mlp=moe) for L in cfg["layers"]])
+
+
+def run_zisesun(args):
+    """`--zisesun`: prompt and decode throughput of the Zisesun decoder at sizes like a real model's layers (random weights, four
+    layers), beside the Birepel decoder of equal size (the closest model here: attention without rotation beside recurrent layers
+    with a matrix of state, learned positions, experts), and the new kernels one by one beside that model's like kernels with
+    their fractions of the measured peaks.  Prints one JSON line of its own; the default run and its line are untouched."""
+    import torch
+    from braidinfer_b200.engine import Engine
+    pk = peaks()
+    flush = torch.empty(256 << 20, dtype=torch.uint8, device="cuda")
+
+    def timed(fn, reps=5, warm=2, graph=False):
+        for _ in range(warm):
+            fn()
+        run = fn
+        if graph:
+            torch.cuda.synchronize()
+            gr = torch.cuda.CUDAGraph()
+            with torch.cuda.graph(gr):
+                fn()
+            run = gr.replay
+            run()
+        ts = []
+        for _ in range(reps):
+            flush.zero_()
+            torch.cuda.synchronize()
+            e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+            e0.record()
+            run()
+            e1.record()
+            torch.cuda.synchronize()
+            ts.append(e0.elapsed_time(e1) / 1e3)
+        return statistics.median(ts)
+
+    def frac(seconds, flops, nbytes):
+        return max(flops / (pk["bf16_tflops"] * 1e12), nbytes / (pk["hbm_gbs"] * 1e9)) / seconds
+
+    T, B, C = args.prompt_len, args.batch, args.context
+    sizes = [n for n in LODUZEN_SIZES if not args.sizes or n in args.sizes.split(",")]
+    out = {"metric": "zisesun_beside_birepel_decoder", "unit": "tokens/s", "dtype": "bf16", "data": "synthetic, random weights",
+           "prompt_len": T, "decode_batch": B, "decode_context": C, "peaks": pk, "l2": "flushed between timed calls", "sizes": {}}
+    with ClockSampler() as clocks:
+        for name in sizes:
+            z = LODUZEN_SIZES[name]
+            row = {}
+            for label, cfg in (("zisesun", zisesun_config(z)), ("birepel", birepel_twin_config(z))):
+                eng = Engine.from_random(cfg, 1, dtype="bfloat16", on_device=True, max_tokens=max(B * (C + 192), T + 64),
+                                         max_slots=B, verbose=False)
+                g = torch.Generator().manual_seed(0)
+                prompt = torch.randint(0, z["vocab"], (T,), generator=g).tolist()
+
+                def prefill():
+                    s = eng.open()
+                    eng.step([(s, prompt)], want="last")
+                    eng.close(s)
+                tp = timed(prefill, reps=3, warm=2)
+                prompts = [torch.randint(0, z["vocab"], (C,), generator=g).tolist() for _ in range(B)]
+                secs, ctx0, launches = device_timed_decode(eng, eng.kernels, prompts, args.steps, max(args.warmup, 3))
+                eng.check()
+                row[label] = {"prefill_tokens_per_s": round(T / tp), "prefill_ms": round(tp * 1e3, 3),
+                              "decode_tokens_per_s": round(B * args.steps / secs), "decode_ms_per_step": round(secs / args.steps * 1e3, 4),
+                              "weight_gb": round(eng.weight_bytes / 1e9, 3), "state_mb_per_sequence": round(sum(
+                                  s.shape[1] for s in eng.cache.state if s is not None) / 1e6, 3),
+                              "launches_per_decode_step": launches // args.steps}
+                del eng
+                torch.cuda.empty_cache()
+            row["kernels"] = zisesun_kernels(z, T, B, C, timed, frac)
+            out["sizes"][name] = row
+    out["clocks"] = clocks.summary()
+    print(json.dumps(out))
+    return 0
+
+
+def zisesun_kernels(z, T, B, C, timed, frac):
+    """The new kernels and options alone, each beside the Birepel decoder's like kernel: seconds, and the fraction of the
+    measured peak that its algorithmic FLOPs or bytes (whichever bounds it) reach.  The recurrences' `frac` is of the copy
+    bandwidth (the bytes they must move); `tflops` says what a walk token by token computes."""
+    import torch
+    from types import SimpleNamespace
+    from braidinfer_b200.cache import PAGE_SIZE
+    from braidinfer_b200.csrc.api import get_kernels
+    K = get_kernels(verbose=False)
+    dev, bf = "cuda", torch.bfloat16
+    i32 = lambda v: torch.tensor(v, dtype=torch.int32, device=dev)        # noqa: E731
+    H, nkh, hd, Wd, win, n = z["heads"], z["kv"], z["dim"], z["width"], z["window"], ZISESUN_STREAMS
+    res = {}
+
+    def paged(n_seqs, length):
+        blocks = -(-length // PAGE_SIZE)
+        cache = torch.randn(n_seqs * blocks, 2, nkh, PAGE_SIZE, hd, device=dev, dtype=bf) * 0.5
+        return cache, torch.arange(n_seqs * blocks, dtype=torch.int32, device=dev).view(n_seqs, blocks)
+
+    def steps_of(n_seqs, each, before):
+        rows = n_seqs * each
+        return SimpleNamespace(rows=rows, n_tokens=rows, n_seqs=n_seqs, q_start=i32([i * each for i in range(n_seqs)]),
+                               q_len=i32([each] * n_seqs), kv_before=i32([before] * n_seqs), slot_ids=i32(list(range(n_seqs))), max_q_len=each,
+                               token_seq=torch.arange(n_seqs, dtype=torch.int32, device=dev).repeat_interleave(each),
+                               positions=(torch.arange(each, dtype=torch.int32, device=dev) + before).repeat(n_seqs))
+
+    def pair(what, new, old, **more):
+        """(seconds, flops, bytes) of the new kernel and of the other model's like kernel"""
+        res[what] = {"zisesun_ms": round(new[0] * 1e3, 4), "zisesun_frac": round(frac(*new), 4)}
+        if old:
+            res[what].update(birepel_ms=round(old[0] * 1e3, 4), birepel_frac=round(frac(*old), 4))
+        res[what].update(more)
+
+    st, sd = steps_of(1, T, 0), steps_of(B, 1, C - 1)
+    sinks = torch.randn(H, device=dev)
+    bias = (torch.rand(H, device=dev) * 2 + 0.1, torch.rand(H, device=dev) * 0.4 + 0.1)
+    # ---- attention: a distance bias behind a window beside a sink and a gate a head over the whole context
+    for what, stp, n_seqs, each, length in (("prompt", st, 1, T, T), ("decode", sd, B, 1, C)):
+        cache, table = paged(n_seqs, length)
+        q = torch.randn(stp.rows, H * hd + 64, device=dev, dtype=bf) * 0.3
+        o = torch.empty(stp.rows, H * hd, device=dev, dtype=bf)
+        new, old = dict(distance_bias=bias), dict(head_sinks=sinks, head_gate=q[:, H * hd:H * hd + H])
+        t = {}
+        for label, kw, w in (("new", new, win), ("old", old, None), ("window", {}, win)):
+            span = min(length, w) if w else length
+            fl = 4 * H * hd * sum(min(p + 1, w) if w else p + 1 for p in range(length - each, length)) * n_seqs
+            by = n_seqs * span * 2 * nkh * hd * 2 if each == 1 else 0
+            sp = max(1, min(K.attn_decode_slots(hd) // (B * nkh * -(-(H // nkh) // 16)), (span // 32) // 4, 64)) if each == 1 else 1
+            mma = timed(lambda: K.attn_mma(q, o, cache, table, stp.q_start, stp.q_len, stp.kv_before, stp.token_seq, n_seqs, each, H, nkh, hd,
+                                           w, hd ** -0.5, n_splits=sp, few_tokens=each == 1, **kw), reps=9, graph=True)
+            t[label] = (mma, fl if each > 1 else 0, by)
+            if each > 1 and K.attn_tc_supports(hd):
+                tc = timed(lambda: K.attn_tc(q, o, cache, table, stp.q_start, stp.q_len, stp.kv_before, 1, T, H, nkh, hd, w, hd ** -0.5, **kw),
+                           reps=9, graph=True)
+                t[label + "_tc"] = (tc, fl, 0)
+        pair(f"{what}_attention_mma", t["new"], t["old"], same_window_without_bias_ms=round(t["window"][0] * 1e3, 4))
+        if "new_tc" in t:
+            pair(f"{what}_attention_tcgen05", t["new_tc"], t["old_tc"], same_window_without_bias_ms=round(t["window_tc"][0] * 1e3, 4))
+    # ---- biases + norms of whole projections + unit values + cache write beside unit heads + temperature + cache write
+    for what, stp, n_seqs, length in (("prompt_prep", st, 1, T), ("decode_prep", sd, B, C)):
+        cache, table = paged(n_seqs, length)
+        rows = stp.rows
+        src = torch.randn(rows, (H + 2 * nkh) * hd, device=dev, dtype=bf)
+        qo = torch.empty(rows, H * hd, device=dev, dtype=bf)
+        wq, wk = torch.ones(H * hd, device=dev, dtype=bf), torch.ones(nkh * hd, device=dev, dtype=bf)
+        t1 = timed(lambda: K.proj_prep_kv(src, qo, stp.positions, stp.token_seq, table, cache, H, nkh, hd, hd, hd, 1e-6, q_w=wq, k_w=wk,
+                                          biases=(wq, wk, wk), v_unit=True), reps=9, graph=True)
+        t2 = timed(lambda: K.head_prep_kv(src, qo, stp.positions, stp.token_seq, table, cache, H, nkh, hd, hd, hd, True, 1e-6, 0.1, 1024),
+                   reps=9, graph=True)
+        by = rows * hd * 2 * (2 * H + 4 * nkh)
+        pair(what, (t1, 0, by), (t2, 0, by))
+    # ---- recurrences and read-outs, the streams, routing and the experts, for a prompt and for decoded tokens
+    heads, dk, dv = z["lheads"], z["ldk"], z["ldv"]
+    for what, stp in (("prompt", st), ("decode", sd)):
+        rows, n_seqs = stp.rows, stp.n_seqs
+        qq, kk = (torch.randn(rows, heads * dk, device=dev, dtype=bf) * 0.1 for _ in range(2))
+        vv = torch.randn(rows, heads * dv, device=dev, dtype=bf)
+        decay = torch.tensor([1.0 - 2.0 ** -(3 + h) for h in range(heads)], device=dev)
+        o1 = torch.empty(rows, heads * dv, device=dev)
+        s1 = torch.zeros(n_seqs, heads * dk * dv * 4, dtype=torch.uint8, device=dev)
+        t1 = timed(lambda: K.linear_scan(qq, kk, vv, decay, None, o1, s1, 0, stp, heads, heads, dk, dv, "constant", act_silu=True), graph=True)
+        by1 = rows * heads * (2 * dk * 2 + dv * 2 + dv * 4) + 2 * n_seqs * heads * dk * dv * 4
+        s2 = torch.zeros(n_seqs, heads * dk * (dv + 1) * 4, dtype=torch.uint8, device=dev)
+        gates = torch.rand(rows, 3 * heads, device=dev) * 0.1 + 0.9
+        o2 = torch.empty(rows, heads * (dv + 1), device=dev)
+        b0 = torch.zeros(heads, device=dev, dtype=bf)
+        t2 = timed(lambda: K.linear_scan(qq, kk, vv, gates[:, :heads], b0, o2, s2, 0, stp, heads, heads, dk, dv + 1, "given", q_scale=dk ** -0.5,
+                                         kappa=gates[:, heads:2 * heads], v_cols=dv), graph=True)
+        by2 = rows * heads * (2 * dk * 2 + dv * 2 + (dv + 1) * 4 + 8) + 2 * n_seqs * heads * dk * (dv + 1) * 4
+        pair(f"{what}_recurrence", (t1, 0, by1), (t2, 0, by2), zisesun_tflops=round(4 * rows * heads * dk * dv / t1 / 1e12, 2),
+             birepel_tflops=round(4 * rows * heads * dk * (dv + 1) / t2 / 1e12, 2))
+        inner = heads * dv
+        gt = torch.randn(rows, inner, device=dev, dtype=bf)
+        wv, ob = torch.ones(inner, device=dev, dtype=bf), torch.empty(rows, inner, device=dev, dtype=bf)
+        t1 = timed(lambda: K.gated_norm(o1, gt, wv, ob, stp.token_seq, inner, False, 1e-6, gate_sigmoid=True), reps=9, graph=True)
+        t2 = timed(lambda: K.mlstm_out(o2, gates[:, 2 * heads:], gt, wv, ob, stp.token_seq, heads, dv, 1e-6), reps=9, graph=True)
+        pair(f"{what}_read_out", (t1, 0, rows * inner * 8), (t2, 0, rows * (inner * 8 + heads * 8)))
+        # the streams: write of one sublayer and read + norm of the next, beside the other model's norm of a result + sum and the
+        # cast of the stream for the next sublayer
+        x, y = torch.randn(rows, n, Wd, device=dev), torch.randn(rows, Wd, device=dev)
+        mix, back, read = (torch.randn(*s, device=dev) * 0.3 for s in ((n, n), (n,), (n,)))
+        w1, xo = torch.ones(Wd, device=dev, dtype=bf), torch.empty(rows, Wd, device=dev, dtype=bf)
+        h = torch.zeros(rows, Wd, device=dev)
+        t1 = timed(lambda: K.streams(x, x, n, y=y, mix=mix, back=back, read=read, w=w1, eps=1e-6, out=xo), reps=9, graph=True)
+
+        def add_and_cast():
+            K.rmsnorm_add(h, y, w1, 1e-6, w_offset=1.0)
+            K.cast(h, xo)
+        t2 = timed(add_and_cast, reps=9, graph=True)
+        pair(f"{what}_streams", (t1, 0, rows * Wd * (8 * n + 4 + 2)), (t2, 0, rows * Wd * (12 + 6)))
+        E, top, J = 8, 2, z["ff"] // 2 // 64 * 64
+        lg, corr = torch.randn(rows, E, device=dev), torch.randn(E, device=dev)
+        idx, wgt = torch.empty(rows, top, dtype=torch.int32, device=dev), torch.empty(rows, top, device=dev)
+        t2 = timed(lambda: K.moe_route(lg, idx, wgt, 1, 1), reps=9, graph=True)
+        t1 = timed(lambda: K.moe_route(lg, idx, wgt, 1, 1, renorm=False, correction=corr * 0.01), reps=9, graph=True)
+        pair(f"{what}_routing", (t1, 0, rows * (E + 2 * top) * 4), (t2, 0, rows * (E + 2 * top) * 4))
+        tile = 16 if rows * top <= 16 * E else 64
+        plan = K.moe_plan(idx, stp.token_seq, E, tile)
+        ys = torch.randn(plan[4] * tile, Wd, device=dev, dtype=bf)
+        t1 = timed(lambda: K.streams(x, x, n, y=(ys, plan, wgt, top), mix=mix, back=back, read=read, w=w1, eps=1e-6, out=xo), reps=9, graph=True)
+
+        def combine():
+            h.zero_()
+            K.moe_combine(h, ys, plan, wgt, top=top)
+            add_and_cast()
+        t2 = timed(combine, reps=9, graph=True)
+        pair(f"{what}_streams_after_experts", (t1, 0, rows * Wd * (8 * n + 2 * top + 2)), (t2, 0, rows * Wd * (2 * top + 8 + 12 + 6)))
+        xin = torch.randn(rows, Wd, device=dev, dtype=bf) * 0.1
+        wg, wu = (torch.randn(E, J, Wd, device=dev, dtype=bf) * 0.02 for _ in range(2))
+        act = torch.empty(plan[4] * tile, J, device=dev, dtype=bf)
+        J2 = (3 * z["ff"] // 4) // 64 * 64
+        w2 = torch.randn(E, J2, Wd, device=dev, dtype=bf) * 0.02
+        act2 = torch.empty(plan[4] * tile, J2, device=dev, dtype=bf)
+        used = int(torch.unique(idx).numel())
+        t1 = timed(lambda: K.moe_gemm_mma(xin, wg, wu, act, plan, top, tile), graph=True)
+        t2 = timed(lambda: K.moe_gemm_mma(xin, w2, None, act2, plan, top, tile, relu2=True), graph=True)
+        pair(f"{what}_experts_first_product", (t1, 4 * rows * top * J * Wd, 2 * used * J * Wd * 2), (t2, 2 * rows * top * J2 * Wd, used * J2 * Wd * 2))
+        wd, wd2 = torch.randn(E, Wd, J, device=dev, dtype=bf) * 0.02, torch.randn(E, Wd, J2, device=dev, dtype=bf) * 0.02
+        t1 = timed(lambda: K.moe_gemm_mma(act, wd, None, ys, plan, top, tile), graph=True)
+        t2 = timed(lambda: K.moe_gemm_mma(act2, wd2, None, ys, plan, top, tile), graph=True)
+        pair(f"{what}_experts_down_product", (t1, 2 * rows * top * J * Wd, used * J * Wd * 2), (t2, 2 * rows * top * J2 * Wd, used * J2 * Wd * 2))
+        del wg, wu, w2, wd, wd2
+    K.check_device_errors()
+    return res
+
+
 def run_reference(args):
     print(json.dumps({"impl": "reference", "unavailable":
                       "mcelrath/braidinfer is Rust + HIP for AMD RDNA3: pip finds neither setup.py nor pyproject.toml, "
@@ -1641,7 +1885,10 @@ def main() -> int:
     ap.add_argument("--ludazen", action="store_true",
                     help="another measurement: the Ludazen decoder at sizes like a real model's layers beside the Bidinex "
                          "decoder of equal size, and its kernels one by one; prints its own line (see run_ludazen)")
-    ap.add_argument("--sizes", default="", help="with --bidinex / --loduzen / --birepel / --ludazen: names of the sizes, with commas (default: all)")
+    ap.add_argument("--zisesun", action="store_true",
+                    help="another measurement: the Zisesun decoder at sizes like a real model's layers beside the Birepel "
+                         "decoder of equal size, and its kernels one by one; prints its own line (see run_zisesun)")
+    ap.add_argument("--sizes", default="", help="with --bidinex / --loduzen / --birepel / --ludazen / --zisesun: names of the sizes, with commas (default: all)")
     ap.add_argument("--prompt-len", type=int, default=2048, help="with --bidinex: tokens of the timed prompt")
     ap.add_argument("--context", type=int, default=2048, help="with --bidinex: context of the timed decode steps")
     args = ap.parse_args()
@@ -1658,6 +1905,8 @@ def main() -> int:
         return run_birepel(args)
     if args.ludazen:
         return run_ludazen(args)
+    if args.zisesun:
+        return run_zisesun(args)
     if args.sweep:
         return run_sweep(args)
     if args.prompt_timeline:

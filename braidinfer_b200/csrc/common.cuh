@@ -44,7 +44,7 @@ void braid_set_error(const char* fmt, ...);
 
 // Programmatic dependent launch.  Every kernel of the library is launched with the
 // attribute that lets it begin while its predecessor in the stream drains, calls
-// pdl_trigger() at its top (so that its own successor may be scheduled early) and
+// pdl_trigger() at its top (so that its own successor may be scheduled early; later where a kernel says why) and
 // pdl_wait() before its first access to memory that an earlier kernel may have written
 // (or may still read).  What comes before pdl_wait() must touch only weights and the
 // kernel's own shared or tensor memory.  BRAIDINFER_PDL=0 in the environment turns the
@@ -102,6 +102,30 @@ __device__ __forceinline__ float glu_act(float g, int act) {
 __device__ __forceinline__ float glu_act_fast(float g, int act) {
     const float e = act == BRAID_ACT_GELU_TANH ? -1.5957691216057308f * (g + 0.044715f * g * g * g) : -g;
     return __fdividef(g, 1.f + __expf(e));
+}
+
+// V neighbouring numbers as float32, V = 1 or as many as 16 bytes hold (p on 16 bytes then).
+template <typename T, int V>
+__device__ __forceinline__ void load_run(const T* p, float* v) {
+    if constexpr (V == 1) {
+        v[0] = to_f32(p[0]);
+    } else {
+        __align__(16) T raw[V];
+        *reinterpret_cast<uint4*>(raw) = *reinterpret_cast<const uint4*>(p);
+#pragma unroll
+        for (int e = 0; e < V; ++e) v[e] = to_f32(raw[e]);
+    }
+}
+template <typename T, int V>
+__device__ __forceinline__ void store_run(T* p, const float* v) {
+    if constexpr (V == 1) {
+        p[0] = from_f32<T>(v[0]);
+    } else {
+        __align__(16) T raw[V];
+#pragma unroll
+        for (int e = 0; e < V; ++e) raw[e] = from_f32<T>(v[e]);
+        *reinterpret_cast<uint4*>(p) = *reinterpret_cast<const uint4*>(raw);
+    }
 }
 
 __device__ __forceinline__ float warp_sum(float v) {

@@ -947,28 +947,6 @@ struct ProjPrepArgs {
     int* error_flag;
 };
 
-template <typename T, int V>
-__device__ __forceinline__ void load_run(const T* p, float* v) {
-    if constexpr (V == 1) {
-        v[0] = to_f32(p[0]);
-    } else {
-        __align__(16) T raw[V];
-        *reinterpret_cast<uint4*>(raw) = *reinterpret_cast<const uint4*>(p);
-#pragma unroll
-        for (int e = 0; e < V; ++e) v[e] = to_f32(raw[e]);
-    }
-}
-template <typename T, int V>
-__device__ __forceinline__ void store_run(T* p, const float* v) {
-    if constexpr (V == 1) {
-        p[0] = from_f32<T>(v[0]);
-    } else {
-        __align__(16) T raw[V];
-#pragma unroll
-        for (int e = 0; e < V; ++e) raw[e] = from_f32<T>(v[e]);
-        *reinterpret_cast<uint4*>(p) = *reinterpret_cast<const uint4*>(raw);
-    }
-}
 // V projected numbers with their bias
 template <typename T, int V>
 __device__ __forceinline__ void load_biased(const T* p, const T* b, int c, float* v) {

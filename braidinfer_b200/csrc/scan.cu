@@ -264,6 +264,13 @@ extern "C" int braid_scan_decay(float* z, long long stride, const void* bias, in
     BRAID_LAUNCH_CHECK();
 }
 
+// silu of a projected number: with the fast exponential and division (a few units in float32's last place) where the
+// number comes in 8 bits of mantissa
+template <typename T>
+__device__ __forceinline__ float staged_silu(float z) {
+    return sizeof(T) == 2 ? glu_act_fast(z, BRAID_ACT_SILU) : silu_f32(z);
+}
+
 template <typename T, int MODE, int RG, int R>
 __global__ void __launch_bounds__(SCAN_THREADS)
 linear_scan_kernel(ScanArgs a) {
@@ -359,8 +366,8 @@ linear_scan_kernel(ScanArgs a) {
         for (int u = 0; u < NQ; ++u) {
             const int idx = tid + u * SCAN_THREADS;
             const float q0 = to_f32(pq[u]), k0 = to_f32(pk[u]);
-            sq[idx] = (silu ? silu_f32(q0) : q0) * a.q_scale;
-            sk[idx] = silu ? silu_f32(k0) : k0;
+            sq[idx] = (silu ? staged_silu<T>(q0) : q0) * a.q_scale;
+            sk[idx] = silu ? staged_silu<T>(k0) : k0;
             if (MODE == DECAY_CHANNEL) {
                 float av = pa[u];
                 if (!a.gate_is_decay) {
@@ -373,7 +380,7 @@ linear_scan_kernel(ScanArgs a) {
 #pragma unroll
         for (int u = 0; u < NV; ++u) {
             const float v0 = to_f32(pv[u]);
-            sv[tid + u * SCAN_THREADS] = silu ? silu_f32(v0) : v0;
+            sv[tid + u * SCAN_THREADS] = silu ? staged_silu<T>(v0) : v0;
         }
         if (MODE == DECAY_HEAD && tid < nt) {
             const float x = to_f32(pg) + head_bias;
@@ -642,6 +649,70 @@ gated_norm_block_kernel(const float* __restrict__ y, const T* __restrict__ gate,
     }
 }
 
+// The same for wide groups whose rows allow 16-byte moves: a CTA of up to 512 threads a (row, group), V neighbouring columns
+// a thread and turn, the first two runs of a thread kept in registers between the sum of squares and the result (a group of
+// 4,096 columns of one row: 48 -> 12 us with a CTA of 128 threads and single columns before).
+template <typename T, int V>
+__global__ void __launch_bounds__(512)
+gated_norm_wide_kernel(const float* __restrict__ y, const T* __restrict__ gate, long long gate_stride, const T* __restrict__ w,
+                       int w_len, T* __restrict__ out, long long out_stride, const int* __restrict__ token_seq, int rows,
+                       int width, int group, int gate_first, int gate_sigmoid, float eps, float out_scale) {
+    pdl_trigger();
+    pdl_wait();
+    __shared__ float red[32];
+    const int groups = width / group;
+    const int row = blockIdx.x / groups, gi = blockIdx.x - row * groups;
+    if (token_seq[row] < 0) return;
+    const float* yr = y + (size_t)row * width + (size_t)gi * group;
+    const T* gr = gate + (size_t)row * gate_stride + (size_t)gi * group;
+    const T* wr = w + (w_len == group ? 0 : (size_t)gi * group);
+    constexpr int KEEP = 2;
+    float u[KEEP][V], sg[KEEP][V];
+    auto fetch = [&](int c, float* uu, float* ss) {
+#pragma unroll
+        for (int e = 0; e < V; e += 4) load_run<float, 4>(yr + c + e, uu + e);
+        load_run<T, V>(gr + c, ss);
+#pragma unroll
+        for (int e = 0; e < V; ++e) {
+            ss[e] = norm_gate(ss[e], gate_sigmoid);
+            if (gate_first) uu[e] *= ss[e];
+        }
+    };
+    const int step = blockDim.x * V, c0 = threadIdx.x * V;
+    float ss = 0.f;
+#pragma unroll
+    for (int k = 0; k < KEEP; ++k)
+        if (c0 + k * step < group) {
+            fetch(c0 + k * step, u[k], sg[k]);
+#pragma unroll
+            for (int e = 0; e < V; ++e) ss = fmaf(u[k][e], u[k][e], ss);
+        }
+    for (int c = c0 + KEEP * step; c < group; c += step) {
+        float uu[V], gg[V];
+        fetch(c, uu, gg);
+#pragma unroll
+        for (int e = 0; e < V; ++e) ss = fmaf(uu[e], uu[e], ss);
+    }
+    ss = block_sum(ss, red);
+    const float r = 1.f / sqrtf(ss / (float)group + eps);
+    T* orow = out + (size_t)row * out_stride + (size_t)gi * group;
+    auto finish = [&](int c, const float* uu, const float* gg) {
+        float wv[V], o[V];
+        load_run<T, V>(wr + c, wv);
+#pragma unroll
+        for (int e = 0; e < V; ++e) o[e] = (gate_first ? uu[e] * r * wv[e] : (uu[e] * r * wv[e]) * gg[e]) * out_scale;
+        store_run<T, V>(orow + c, o);
+    };
+#pragma unroll
+    for (int k = 0; k < KEEP; ++k)
+        if (c0 + k * step < group) finish(c0 + k * step, u[k], sg[k]);
+    for (int c = c0 + KEEP * step; c < group; c += step) {
+        float uu[V], gg[V];
+        fetch(c, uu, gg);
+        finish(c, uu, gg);
+    }
+}
+
 extern "C" int braid_gated_norm(const float* y, const void* gate, long long gate_stride, const void* w, int w_len, void* out,
                                 long long out_stride, const int* token_seq, int dtype, int rows, int width, int group,
                                 int gate_first, int gate_sigmoid, float eps, float out_scale, void* stream) {
@@ -652,6 +723,21 @@ extern "C" int braid_gated_norm(const float* y, const void* gate, long long gate
     const long long blocks = (items + 3) / 4;
     if (blocks > 0x7fffffffLL) BRAID_REFUSE("gated_norm: %lld (row, group) pairs exceed one launch", items);
     cudaStream_t s = (cudaStream_t)stream;
+    const int vec = dtype == BRAID_F32 ? 4 : 8;
+    if (group > 128 && items <= 0x7fffffffLL && group % vec == 0 && gate_stride % vec == 0 && out_stride % vec == 0 &&
+        (w_len == group || w_len == width) && (((uintptr_t)y | (uintptr_t)gate | (uintptr_t)w | (uintptr_t)out) & 15) == 0) {
+        const int runs = (group / vec + 31) / 32 * 32;
+        const dim3 block(runs < 64 ? 64 : runs > 512 ? 512 : runs);
+        if (dtype == BRAID_F32)
+            braid_launch(gated_norm_wide_kernel<float, 4>, dim3((int)items), block, 0, s, y, (const float*)gate, gate_stride,
+                         (const float*)w, w_len, (float*)out, out_stride, token_seq, rows, width, group, gate_first, gate_sigmoid, eps, out_scale);
+        else if (dtype == BRAID_BF16)
+            braid_launch(gated_norm_wide_kernel<__nv_bfloat16, 8>, dim3((int)items), block, 0, s, y, (const __nv_bfloat16*)gate, gate_stride,
+                         (const __nv_bfloat16*)w, w_len, (__nv_bfloat16*)out, out_stride, token_seq, rows, width, group, gate_first,
+                         gate_sigmoid, eps, out_scale);
+        else BRAID_REFUSE("gated_norm: unknown dtype code %d", dtype);
+        BRAID_LAUNCH_CHECK();
+    }
     if (group > 128 && items <= 0x7fffffffLL) {
         if (dtype == BRAID_F32)
             braid_launch(gated_norm_block_kernel<float>, dim3((int)items), dim3(128), 0, s, y, (const float*)gate, gate_stride,

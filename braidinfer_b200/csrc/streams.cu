@@ -95,7 +95,6 @@ __device__ __forceinline__ void sublayer_result(const StreamsArgs& a, int row, i
 template <int N>
 __global__ void __launch_bounds__(256)
 streams_kernel(StreamsArgs a) {
-    pdl_trigger();
     extern __shared__ float sm[];            // [cols] u of this CTA's columns, then [top] slots and weights
     __shared__ float coef[STREAMS_MAX * (STREAMS_MAX + 2)];
     __shared__ float red[32];
@@ -117,6 +116,7 @@ streams_kernel(StreamsArgs a) {
     int* slots = (int*)(sm + a.cols);
     float* wgts = (float*)(slots + a.top);
     pdl_wait();
+    pdl_trigger();                           // not before: the kernels of a whole layer would queue up on the SMs behind the experts
     if (a.y_kind == Y_EXPERTS)
         for (int k = tid; k < a.top; k += blockDim.x) {
             slots[k] = a.pair_slot[(size_t)row * a.top + k];
