@@ -479,13 +479,23 @@ scan_carry_kernel(ScanArgs a) {
     const int i = (int)((idx / a.dv) % a.dk);
     float* S_area = (float*)(a.state + (size_t)a.slot_ids[seq] * a.state_stride + a.state_offset);
     float S = S_area[idx];
-    for (int c = 0; c < n_chunks; ++c) {
-        const size_t base = (size_t)(seq * a.max_chunks + c);
-        float* w = a.wbuf + base * per_seq + idx;
-        const float u = *w;
-        const float d = MODE != DECAY_CHANNEL ? a.dbuf[base * a.heads + h] : a.dbuf[(base * a.heads + h) * a.dk + i];
-        *w = S;                                             // the state that chunk c starts from
-        S = fmaf(d, S, u);
+    // eight chunks' numbers are asked for before any of them is used: they do not depend on one another, the chain does
+    constexpr int B = 8;
+    for (int c0 = 0; c0 < n_chunks; c0 += B) {
+        float u[B], d[B];
+#pragma unroll
+        for (int j = 0; j < B; ++j) {
+            const size_t base = (size_t)(seq * a.max_chunks + c0 + j);
+            const bool in = c0 + j < n_chunks;
+            u[j] = in ? a.wbuf[base * per_seq + idx] : 0.f;
+            d[j] = !in ? 0.f : MODE != DECAY_CHANNEL ? a.dbuf[base * a.heads + h] : a.dbuf[(base * a.heads + h) * a.dk + i];
+        }
+#pragma unroll
+        for (int j = 0; j < B; ++j)
+            if (c0 + j < n_chunks) {
+                a.wbuf[(size_t)(seq * a.max_chunks + c0 + j) * per_seq + idx] = S;      // the state that chunk c0 + j starts from
+                S = fmaf(d[j], S, u[j]);
+            }
     }
     S_area[idx] = S;
 }
