@@ -10,6 +10,7 @@ from __future__ import annotations
 import ctypes
 import os
 from ctypes import c_int, c_longlong, c_float, c_void_p, c_char_p
+from dataclasses import dataclass
 from typing import List, Optional, Tuple
 
 import torch
@@ -70,6 +71,21 @@ PAIR_TOKEN_TILE = 256        # the token tile of the kernel that runs on pairs o
 # longest sequence brings less than two chunks walk in one pass.  BRAIDINFER_SCAN_CHUNK names one length for all
 # (0: never in chunks), for measurements.
 SCAN_CHUNK = int(os.environ["BRAIDINFER_SCAN_CHUNK"]) if os.environ.get("BRAIDINFER_SCAN_CHUNK") else None
+
+
+@dataclass(frozen=True)
+class ConvSegment:
+    """See `Kernels.conv_segment`."""
+    heads: int
+    size: int
+    pad: int
+    norm: int
+    weight: Optional[torch.Tensor]
+    silu: bool
+    rotate: bool
+    factor: float
+    out: Optional[torch.Tensor]
+    plane: int
 
 
 class RowScale:
@@ -146,7 +162,7 @@ class Kernels:
                                         [c_float, c_float, c_int, c_void_p, c_void_p]
         L.braid_proj_prep_kv.argtypes = [c_void_p, c_longlong, c_int] + [c_void_p] * 10 + [c_int] * 10 + \
                                         [c_float, c_void_p, c_void_p]
-        L.braid_head_gate.argtypes = [c_void_p, c_longlong, c_void_p, c_longlong, c_void_p] + [c_int] * 5 + [c_void_p]
+        L.braid_head_gate.argtypes = [c_void_p, c_longlong, c_void_p, c_longlong, c_void_p] + [c_int] * 6 + [c_void_p]
         L.braid_glu_clamp.argtypes = [c_void_p, c_void_p, c_int, c_int, c_int, c_float, c_float, c_void_p]
         L.braid_silu_mul.argtypes = [c_void_p, c_void_p, c_int, c_int, c_int, c_void_p]
         L.braid_act_mul.argtypes = [c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p]
@@ -165,7 +181,7 @@ class Kernels:
         L.braid_attn_simple.argtypes = [c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p,
                                         c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
                                         c_float, c_int, c_float, c_float, c_void_p, c_void_p, c_longlong, c_int, c_void_p,
-                                        c_int, c_void_p, c_void_p, c_void_p, c_void_p]
+                                        c_int, c_void_p, c_void_p, c_float, c_void_p, c_void_p]
         L.braid_head_mix.argtypes = [c_void_p, c_longlong, c_void_p, c_int, c_void_p, c_longlong, c_int, c_void_p] + \
                                     [c_int] * 5 + [c_void_p]
         L.braid_bias_xielu.argtypes = [c_void_p, c_longlong, c_void_p, c_void_p, c_int, c_void_p, c_longlong] + [c_int] * 4 + \
@@ -377,15 +393,17 @@ class Kernels:
             page_table.shape[1] if page_table is not None else 0, cache.shape[0] if cache is not None else 0, float(eps),
             self._error_flag.data_ptr(), self._stream()), "proj_prep_kv")
 
-    def head_gate(self, x: torch.Tensor, gate: Optional[torch.Tensor], out: torch.Tensor, heads: int, hd: int, dv: int) -> None:
-        """out[r, h * dv + c] = x[r, h * hd + c] * sigmoid(gate[r, h]), c < dv (gate None: the copy alone)."""
+    def head_gate(self, x: torch.Tensor, gate: Optional[torch.Tensor], out: torch.Tensor, heads: int, hd: int, dv: int,
+                  per_column: bool = False) -> None:
+        """out[r, h * dv + c] = x[r, h * hd + c] * sigmoid(gate[r, h]), c < dv (gate None: the copy alone); with `per_column`
+        the gate is one number a column, sigmoid(gate[r, h * dv + c])."""
         rows = out.shape[0]
         if x.stride(1) != 1 or not out.is_contiguous() or out.shape[1] != heads * dv or x.dtype != out.dtype \
-                or (gate is not None and (gate.dtype != x.dtype or gate.stride(1) != 1 or gate.shape[1] < heads)):
+                or (gate is not None and (gate.dtype != x.dtype or gate.stride(1) != 1 or gate.shape[1] < heads * (dv if per_column else 1))):
             raise KernelError("head_gate: x, gate and out of one element type; out contiguous [rows, heads * dv]")
         self.launches += 1
         self._check(self.lib.braid_head_gate(x.data_ptr(), x.stride(0), _ptr(gate), gate.stride(0) if gate is not None else 0,
-                                             out.data_ptr(), dtype_code(out.dtype), rows, heads, hd, dv, self._stream()),
+                                             out.data_ptr(), dtype_code(out.dtype), rows, heads, hd, dv, int(per_column), self._stream()),
                     "head_gate")
 
     def glu_clamp(self, gu: torch.Tensor, out: torch.Tensor, limit: float, alpha: float) -> None:
@@ -430,7 +448,7 @@ class Kernels:
                     out_scale: float = 1.0, head_sinks: Optional[torch.Tensor] = None,
                     head_gate: Optional[torch.Tensor] = None, keep_first: int = 0,
                     head_scale: Optional[torch.Tensor] = None, value_heads: int = 1,
-                    distance_bias: Optional[Tuple[torch.Tensor, torch.Tensor]] = None) -> None:
+                    distance_bias: Optional[Tuple[torch.Tensor, torch.Tensor]] = None, softcap: Optional[float] = None) -> None:
         """q: [rows, >= nqh*hd] (a view of the qkv rows is fine), out: [rows, nqh*hd].  `keep_first`: with a window,
         a sequence's first positions stay visible; `head_scale` (float32 [nqh]): a factor a head on the scores;
         `value_heads` = nkh: every query head reads the values of every kv head, out is [rows, nqh*nkh*hd] with
@@ -438,6 +456,7 @@ class Kernels:
         attention sink, one more term of the softmax's denominator that has no value (None: no sink);
         `head_sinks` (float32 [nqh]): a sink score a head instead; `out_scale`: a constant factor on the result;
         `distance_bias` (r1, r2; float32 [nqh] each): r1 ln(1 + r2 (p - j)) comes off the score of key j at position p;
+        `softcap`: the scaled scores become softcap * tanh(score / softcap);
         `head_gate` ([rows, >= nqh] of the rows' type, a view is fine): head h's result times sigmoid(head_gate[row, h])."""
         rows = out.shape[0]
         self._check_head_extras(head_sinks, head_gate, nqh, out.dtype, head_scale, distance_bias)
@@ -450,7 +469,7 @@ class Kernels:
             page_size, page_table.shape[1], cache.shape[0], int(window or 0), float(scale),
             int(sink is not None), float(sink or 0.0), float(out_scale), _ptr(head_sinks), _ptr(head_gate),
             head_gate.stride(0) if head_gate is not None else 0, int(keep_first or 0), _ptr(head_scale), int(value_heads),
-            *self._bias_args(distance_bias), self._error_flag.data_ptr() + 16, self._stream()),
+            *self._bias_args(distance_bias), float(softcap or 0.0), self._error_flag.data_ptr() + 16, self._stream()),
             "attn_simple")
 
     def head_mix(self, src: torch.Tensor, talk: torch.Tensor, out: torch.Tensor, token_seq: Optional[torch.Tensor],
@@ -516,7 +535,7 @@ class Kernels:
             lib.braid_last_error.restype = c_char_p
             lib.braid_attn_mma.restype = c_int
             lib.braid_attn_mma.argtypes = [c_void_p] * 9 + [c_int] * 13 + [c_float, c_int, c_float, c_float, c_void_p, c_void_p,
-                                           c_longlong, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p]
+                                           c_longlong, c_int, c_void_p, c_void_p, c_void_p, c_float, c_int, c_int, c_void_p, c_void_p]
             lib.braid_attn_mma_partial_floats.restype = c_longlong
             lib.braid_attn_mma_partial_floats.argtypes = [c_int, c_int, c_int]
             if lib.braid_attn_mma_value_heads() != value_heads:
@@ -529,7 +548,7 @@ class Kernels:
                 lib.braid_attn_tc.restype = c_int
                 lib.braid_attn_tc.argtypes = [c_void_p, c_void_p, c_void_p, c_longlong] + [c_void_p] * 4 + [c_int] * 10 + \
                                              [c_float, c_int, c_float, c_float, c_void_p, c_void_p, c_longlong, c_void_p, c_void_p,
-                                              c_void_p, c_void_p]
+                                              c_float, c_void_p, c_void_p]
             lib.braid_attn_mma_decode_slots.restype = c_int
             lib.braid_attn_mma_decode_slots.argtypes = [c_int]
             lib.decode_slots = lib.braid_attn_mma_decode_slots(1)     # CTAs of the few-token kernel held at once
@@ -552,9 +571,9 @@ class Kernels:
                 nqh: int, nkh: int, hd: int, window: Optional[int], scale: float, sink: Optional[float] = None,
                 out_scale: float = 1.0, head_sinks: Optional[torch.Tensor] = None,
                 head_gate: Optional[torch.Tensor] = None,
-                distance_bias: Optional[Tuple[torch.Tensor, torch.Tensor]] = None) -> None:
+                distance_bias: Optional[Tuple[torch.Tensor, torch.Tensor]] = None, softcap: Optional[float] = None) -> None:
         """bfloat16 attention of prompts over the cache on tcgen05 (head sizes 64 and 128); `sink`, `head_sinks`,
-        `out_scale`, `head_gate` and `distance_bias` as in `attn_simple`."""
+        `out_scale`, `head_gate`, `distance_bias` and `softcap` as in `attn_simple`."""
         lib = self.attn_mma_library(hd)
         self._check_head_extras(head_sinks, head_gate, nqh, out.dtype, distance_bias=distance_bias)
         self._check_pages(cache)
@@ -567,7 +586,8 @@ class Kernels:
                                out.shape[0], n_seqs, max_q_len, nqh, nkh, hd, page_table.shape[1], int(window or 0),
                                float(scale), int(sink is not None), float(sink or 0.0), float(out_scale),
                                _ptr(head_sinks), _ptr(head_gate), head_gate.stride(0) if head_gate is not None else 0,
-                               *self._bias_args(distance_bias), self._error_flag.data_ptr() + 12, self._stream())
+                               *self._bias_args(distance_bias), float(softcap or 0.0), self._error_flag.data_ptr() + 12,
+                               self._stream())
         if rc != 0:
             raise KernelError(f"attn_tc: {lib.braid_last_error().decode(errors='replace')} (code {rc})")
 
@@ -582,10 +602,10 @@ class Kernels:
                  out_scale: float = 1.0, head_sinks: Optional[torch.Tensor] = None,
                  head_gate: Optional[torch.Tensor] = None, keep_first: int = 0,
                  head_scale: Optional[torch.Tensor] = None, value_heads: int = 1,
-                 distance_bias: Optional[Tuple[torch.Tensor, torch.Tensor]] = None) -> None:
+                 distance_bias: Optional[Tuple[torch.Tensor, torch.Tensor]] = None, softcap: Optional[float] = None) -> None:
         """bfloat16 attention over the cache on the tensor cores; `n_splits` > 1 slices the
         context (for steps of few tokens) and merges the slices in a second kernel.  `sink`, `head_sinks`,
-        `out_scale`, `head_gate`, `keep_first`, `head_scale`, `distance_bias` and `value_heads` as in `attn_simple` (the sink is counted
+        `out_scale`, `head_gate`, `keep_first`, `head_scale`, `distance_bias`, `softcap` and `value_heads` as in `attn_simple` (the sink is counted
         once, where the slices merge; where the accumulators do not hold the values of all kv heads, groups of them
         go to CTAs of their own)."""
         vh = self.attn_value_heads_a_launch(hd, value_heads) if value_heads > 1 else 1
@@ -612,7 +632,7 @@ class Kernels:
                                     1 if few_tokens else 0, float(scale), int(sink is not None), float(sink or 0.0),
                                     float(out_scale), _ptr(head_sinks), _ptr(head_gate),
                                     head_gate.stride(0) if head_gate is not None else 0, int(keep_first or 0),
-                                    _ptr(head_scale), *self._bias_args(distance_bias), vh0, value_heads if value_heads > 1 else 0,
+                                    _ptr(head_scale), *self._bias_args(distance_bias), float(softcap or 0.0), vh0, value_heads if value_heads > 1 else 0,
                                     self._error_flag.data_ptr() + 16, self._stream())
             if rc != 0:
                 raise KernelError(f"attn_mma: {lib.braid_last_error().decode(errors='replace')} (code {rc})")
@@ -656,12 +676,12 @@ class Kernels:
             lib.braid_last_error.restype = c_char_p
             if name == "latent":
                 lib.braid_latent_prep.argtypes = [c_void_p, c_longlong, c_int] + [c_void_p] * 7 + [c_int] * 10 + \
-                                                 [c_float, c_int, c_void_p, c_void_p]
+                                                 [c_float, c_int, c_void_p, c_longlong, c_void_p, c_int, c_void_p, c_void_p]
                 lib.braid_gemm_heads.argtypes = [c_void_p] * 4 + [c_int] * 5 + [c_longlong] * 5 + [c_float, c_void_p]
                 lib.braid_gemm_heads_mma.argtypes = [c_void_p] * 4 + [c_int] * 4 + [c_longlong] * 5 + [c_float, c_void_p]
                 lib.braid_gemm_heads_mma.restype = c_int
                 lib.braid_attn_latent_simple.argtypes = [c_void_p, c_void_p, c_int] + [c_void_p] * 4 + \
-                                                        [c_longlong, c_longlong] + [c_int] * 8 + [c_float, c_void_p, c_void_p]
+                                                        [c_longlong, c_longlong] + [c_int] * 8 + [c_float, c_void_p, c_void_p, c_void_p]
                 names = ("braid_latent_prep", "braid_gemm_heads", "braid_attn_latent_simple")
             elif name == "scan":
                 lib.braid_causal_conv.argtypes = [c_void_p, c_longlong, c_void_p, c_longlong, c_void_p, c_void_p, c_int,
@@ -692,6 +712,20 @@ class Kernels:
                                                   [c_void_p, c_void_p]
                 lib.braid_moe_gemm_mma.restype = c_int
                 names = ("braid_moe_route", "braid_moe_plan", "braid_moe_gemm_simt", "braid_moe_combine")
+            elif name == "conv":
+                lib.braid_conv_heads.argtypes = [c_void_p, c_longlong, c_void_p, c_void_p, c_int, c_void_p, c_longlong, c_longlong] + \
+                                                [c_void_p] * 7 + [c_int] * 3 + [c_void_p, c_int, c_int, c_float, c_float] + \
+                                                [c_int] * 5 + [c_void_p] * 5 + [c_int, c_void_p, c_void_p]
+                names = ("braid_conv_heads",)
+            elif name == "delta":
+                lib.braid_delta_rule.argtypes = [c_void_p, c_longlong] * 4 + [c_void_p, c_void_p, c_void_p, c_longlong, c_int,
+                                                 c_void_p, c_longlong, c_void_p, c_longlong, c_longlong] + [c_void_p] * 3 + \
+                                                [c_int] * 7 + [c_void_p, c_longlong, c_void_p]
+                lib.braid_delta_gated_norm.argtypes = [c_void_p, c_void_p, c_longlong, c_void_p, c_int, c_void_p, c_longlong,
+                                                       c_void_p] + [c_int] * 4 + [c_float, c_void_p]
+                lib.braid_delta_work_floats.argtypes = [c_int] * 6
+                lib.braid_delta_work_floats.restype = c_longlong
+                names = ("braid_delta_rule", "braid_delta_gated_norm")
             elif name == "streams":
                 lib.braid_streams.argtypes = [c_void_p, c_void_p] + [c_int] * 4 + [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int,
                                               c_longlong, c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_int,
@@ -735,7 +769,30 @@ class Kernels:
             proj.data_ptr(), proj.stride(0), q_cols, _ptr(norm_w), inv_freq.data_ptr(), positions.data_ptr(),
             token_seq.data_ptr(), _ptr(page_table), _ptr(cache), q_lat.data_ptr(), dtype_code(proj.dtype),
             proj.shape[0], heads, dim, rot, rank, rot_dims, page_size, cols, cache.shape[0] if cache is not None else 0,
-            float(eps), int(adjacent), self._error_flag.data_ptr(), self._stream()), "latent_prep")
+            float(eps), int(adjacent), None, 0, None, 0, self._error_flag.data_ptr(), self._stream()), "latent_prep")
+
+    def latent_down(self, proj: torch.Tensor, c_col: int, c_q: torch.Tensor, q_norm_w: torch.Tensor, norm_w: Optional[torch.Tensor],
+                    inv_freq: torch.Tensor, positions: torch.Tensor, token_seq: torch.Tensor, page_table: Optional[torch.Tensor],
+                    cache: Optional[torch.Tensor], rot: int, rank: int, rot_dims: int, page_size: int, eps: float,
+                    adjacent: bool = False) -> None:
+        """A step's low-rank rows: proj [rows, >= c_col (+ rank + rot)] starts with the queries' low-rank part
+        (q_norm_w.numel() numbers), whose RMS norm goes to c_q [rows, >= that many columns, zeros beyond]; from column
+        c_col on lies what `latent_prep` norms, rotates and writes into `cache` (None: nothing)."""
+        lib = self.part_library("latent")
+        if cache is None:
+            norm_w = None
+        elif norm_w is None or cache.shape[3] != page_size or cache.shape[4] != rank + rot or proj.shape[1] < c_col + rank + rot:
+            raise KernelError(f"latent_down: a cache [pages, 1, 1, {page_size}, {rank + rot}] wants a norm weight and rows that hold it")
+        if any(t is not None and t.dtype != proj.dtype for t in (c_q, q_norm_w, norm_w, cache)) or proj.stride(1) != 1 \
+                or not c_q.is_contiguous() or c_q.shape[0] != proj.shape[0]:
+            raise KernelError("latent_down: rows, weights, result and cache of one element type, contiguous rows")
+        cols = page_table.shape[1] if page_table is not None else 0
+        self.launches += 1
+        self._check_lib(lib, lib.braid_latent_prep(
+            proj.data_ptr(), proj.stride(0), c_col, _ptr(norm_w), inv_freq.data_ptr(), positions.data_ptr(),
+            token_seq.data_ptr(), _ptr(page_table), _ptr(cache), None, dtype_code(proj.dtype), proj.shape[0], 0, 0, rot, rank,
+            rot_dims, page_size, cols, cache.shape[0] if cache is not None else 0, float(eps), int(adjacent), c_q.data_ptr(),
+            c_q.shape[1], q_norm_w.data_ptr(), q_norm_w.numel(), self._error_flag.data_ptr(), self._stream()), "latent_down")
 
     def gemm_heads(self, x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, gate: Optional[torch.Tensor] = None,
                    mult: float = 1.0, tensor_cores: bool = True) -> None:
@@ -769,12 +826,13 @@ class Kernels:
 
     def attn_latent_simple(self, q_lat: torch.Tensor, out: torch.Tensor, cache: torch.Tensor, page_table: torch.Tensor,
                            positions: torch.Tensor, token_seq: torch.Tensor, rank: int, window: Optional[int],
-                           scale: float) -> None:
+                           scale: float, sinks: Optional[torch.Tensor] = None) -> None:
         """Multi-query attention over the latent cache, one warp per (token, head): q_lat [rows, heads, D],
         out [rows, heads, rank], cache [pages, 1, 1, page_size, D]; a cached row is the key, its first `rank`
-        numbers the value."""
+        numbers the value.  `sinks` (float32 [heads]): a score a head that joins the denominator and has no value."""
         lib = self.part_library("latent")
         rows, heads, d = q_lat.shape
+        self._check_head_extras(sinks, None, heads, out.dtype)
         if not q_lat.is_contiguous() or not out.is_contiguous() or tuple(out.shape) != (rows, heads, rank):
             raise KernelError("attn_latent_simple: q_lat [rows, heads, D] and out [rows, heads, rank] must be contiguous")
         if cache.dim() != 5 or cache.shape[1] != 1 or cache.shape[2] != 1 or cache.shape[4] != d or cache.dtype != q_lat.dtype:
@@ -783,7 +841,7 @@ class Kernels:
         self._check_lib(lib, lib.braid_attn_latent_simple(
             q_lat.data_ptr(), out.data_ptr(), dtype_code(out.dtype), cache.data_ptr(), page_table.data_ptr(),
             positions.data_ptr(), token_seq.data_ptr(), q_lat.stride(0), out.stride(0), rows, heads, d, rank,
-            cache.shape[3], page_table.shape[1], cache.shape[0], int(window or 0), float(scale),
+            cache.shape[3], page_table.shape[1], cache.shape[0], int(window or 0), float(scale), _ptr(sinks),
             self._error_flag.data_ptr() + 16, self._stream()), "attn_latent_simple")
 
     # ------------------------------------------------------------------ mixture of experts
@@ -906,7 +964,7 @@ class Kernels:
             lib = ctypes.CDLL(str(build.latent_attention_library(rank, rot, verbose=self._verbose)))
             lib.braid_last_error.restype = c_char_p
             lib.braid_latent_attn_mma.restype = c_int
-            lib.braid_latent_attn_mma.argtypes = [c_void_p] * 9 + [c_int] * 8 + [c_float, c_void_p, c_void_p]
+            lib.braid_latent_attn_mma.argtypes = [c_void_p] * 9 + [c_int] * 8 + [c_float, c_void_p, c_void_p, c_void_p]
             lib.braid_latent_attn_partial_floats.restype = c_longlong
             lib.braid_latent_attn_partial_floats.argtypes = [c_int, c_int, c_int]
             lib.vparts = lib.braid_latent_attn_vparts()
@@ -928,12 +986,13 @@ class Kernels:
     def attn_latent_mma(self, q_lat: torch.Tensor, out: torch.Tensor, cache: torch.Tensor, page_table: torch.Tensor,
                         q_start: torch.Tensor, q_len: torch.Tensor, kv_before: torch.Tensor, token_seq: torch.Tensor,
                         n_seqs: int, max_q_len: int, rank: int, window: Optional[int], scale: float,
-                        n_splits: int = 1) -> None:
+                        n_splits: int = 1, sinks: Optional[torch.Tensor] = None) -> None:
         """`attn_latent_simple` in bfloat16 on the tensor cores.  Rows of padding are not written.  `n_splits` > 1
         slices the context (steps of few tokens) and merges the slices in a second kernel."""
         rows, heads, d = q_lat.shape
         lib = self.latent_attention_library(rank, d - rank)
         self._check_pages(cache)
+        self._check_head_extras(sinks, None, heads, out.dtype)
         if q_lat.dtype != torch.bfloat16 or out.dtype != torch.bfloat16 or cache.dtype != torch.bfloat16 \
                 or not q_lat.is_contiguous() or not out.is_contiguous() or tuple(out.shape) != (rows, heads, rank) \
                 or cache.dim() != 5 or cache.shape[1] != 1 or cache.shape[2] != 1 or cache.shape[4] != d:
@@ -951,7 +1010,7 @@ class Kernels:
         self._check_lib(lib, lib.braid_latent_attn_mma(
             q_lat.data_ptr(), out.data_ptr(), _ptr(partial), cache.data_ptr(), page_table.data_ptr(), q_start.data_ptr(),
             q_len.data_ptr(), kv_before.data_ptr(), token_seq.data_ptr(), rows, n_seqs, max_q_len, heads,
-            page_table.shape[1], cache.shape[0], int(window or 0), n_splits, float(scale),
+            page_table.shape[1], cache.shape[0], int(window or 0), n_splits, float(scale), _ptr(sinks),
             self._error_flag.data_ptr() + 16, self._stream()), "attn_latent_mma")
 
     def moe_combine(self, h: torch.Tensor, y: torch.Tensor, plan, wgt: Optional[torch.Tensor], top: Optional[int] = None) -> None:
@@ -1048,6 +1107,102 @@ class Kernels:
             *self._state_args(state, state_offset), ctx.token_seq.data_ptr(), ctx.q_start.data_ptr(),
             ctx.q_len.data_ptr(), ctx.slot_ids.data_ptr(), rows, ctx.n_seqs, channels, taps, int(silu), self._stream()),
             "causal_conv")
+
+    @staticmethod
+    def conv_segment(heads: int, size: int, *, pad: Optional[int] = None, norm: Optional[str] = None,
+                     weight: Optional[torch.Tensor] = None, silu: bool = False, rotate: bool = False, factor: float = 1.0,
+                     out: Optional[torch.Tensor] = None, plane: Optional[int] = None) -> "ConvSegment":
+        """One run of channels of `conv_heads`: `heads` heads of `size` channels, written as heads of `pad` numbers (default
+        size; zeros beyond).  silu, then norm ("rms" with `weight` [size], "unit", or None), then `factor`, then the rotation;
+        the result goes to `out` [rows, heads * pad], or into the cache's key (`plane` 0) or value (1) plane."""
+        if norm not in (None, "rms", "unit"):
+            raise KernelError(f"conv_heads: unknown norm {norm!r} (rms, unit)")
+        return ConvSegment(heads, size, pad or size, {None: 0, "rms": 1, "unit": 2}[norm], weight, silu, rotate, float(factor), out,
+                           -1 if plane is None else int(plane))
+
+    def conv_heads(self, x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], state: Optional[torch.Tensor],
+                   state_offset: int, ctx, segments: List["ConvSegment"], *, eps: float, inv_freq: Optional[torch.Tensor] = None,
+                   adjacent: bool = True, amplitude: float = 1.0, page_table: Optional[torch.Tensor] = None,
+                   cache: Optional[torch.Tensor] = None) -> None:
+        """A causal convolution along each sequence of the step over x + bias (x [rows, channels], a view is fine; w
+        [channels, taps], the last tap meets the current token; inputs before the step come from the state, float32
+        [taps - 1, channels] at `state_offset` bytes of each slot, which is then moved on), and head by head what the
+        segments ask for (see `conv_segment` and csrc/conv_heads.cu).  `eps` is every norm's; `inv_freq` [pairs] float32
+        rotates the first numbers of the heads that want it, neighbouring pairs or (adjacent False) halves, sine and cosine
+        times `amplitude`.  Results are float32 where the segments' `out` is, else in the rows' type."""
+        lib = self.part_library("conv")
+        rows, channels = x.shape
+        taps = w.shape[1]
+        outs = [s.out for s in segments if s.out is not None]
+        f32 = bool(outs) and outs[0].dtype == torch.float32 and x.dtype != torch.float32
+        if x.stride(1) != 1 or w.dtype != x.dtype or not w.is_contiguous() or w.shape[0] != channels \
+                or (bias is not None and (bias.dtype != x.dtype or bias.numel() != channels or not bias.is_contiguous())) \
+                or sum(s.heads * s.size for s in segments) != channels:
+            raise KernelError("conv_heads: x, w and bias of one element type, w contiguous [channels, taps], and segments that make "
+                              "up the channels")
+        if any(o.dtype != outs[0].dtype or o.stride(1) != 1 or o.shape[0] != rows for o in outs) \
+                or (outs and outs[0].dtype not in (x.dtype, torch.float32)) \
+                or any(s.out is not None and s.out.shape[1] < s.heads * s.pad for s in segments):
+            raise KernelError("conv_heads: the segments' results hold their heads, in the rows' type or float32")
+        for s in segments:
+            if s.weight is not None and (s.weight.dtype != x.dtype or s.weight.numel() != s.size or not s.weight.is_contiguous()):
+                raise KernelError("conv_heads: a norm's weight holds a head's numbers, in the rows' type")
+            if s.plane >= 0 and cache is not None and (cache.dim() != 5 or cache.dtype != x.dtype or cache.shape[1] != 2
+                                                       or cache.shape[2] != s.heads or cache.shape[4] != s.pad):
+                raise KernelError("conv_heads: the cache is [pages, 2, kv heads, page, padded size] of the rows' type")
+        n = len(segments)
+        ints = (c_int * (7 * n))(*[v for s in segments for v in (s.heads, s.size, s.pad, s.norm, int(s.silu), int(s.rotate), s.plane)])
+        factors = (c_float * n)(*[s.factor for s in segments])
+        weights = (c_void_p * n)(*[_ptr(s.weight) for s in segments])
+        out_ptrs = (c_void_p * n)(*[_ptr(s.out) for s in segments])
+        strides = (c_longlong * n)(*[s.out.stride(0) if s.out is not None else 0 for s in segments])
+        self.launches += 2 if taps > 1 and int(ctx.max_q_len) > 1 else 1
+        self._check_lib(lib, lib.braid_conv_heads(
+            x.data_ptr(), x.stride(0), _ptr(bias), w.data_ptr(), dtype_code(x.dtype),
+            *(self._state_args(state, state_offset) if taps > 1 else (None, 0, 0)), ctx.token_seq.data_ptr(),
+            ctx.positions.data_ptr(), ctx.q_start.data_ptr(), ctx.q_len.data_ptr(), ctx.slot_ids.data_ptr(), _ptr(page_table),
+            _ptr(cache), cache.shape[3] if cache is not None else 0, page_table.shape[1] if page_table is not None else 0,
+            cache.shape[0] if cache is not None else 0, _ptr(inv_freq), 2 * inv_freq.numel() if inv_freq is not None else 0,
+            int(adjacent), float(amplitude), float(eps), rows, ctx.n_seqs, int(ctx.max_q_len), taps, n, ints, factors, weights,
+            out_ptrs, strides, int(f32), self._error_flag.data_ptr(), self._stream()), "conv_heads")
+
+    def delta_rule(self, q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, z: torch.Tensor, bias: torch.Tensor,
+                   rate: torch.Tensor, b: torch.Tensor, out: torch.Tensor, state: torch.Tensor, state_offset: int, ctx,
+                   heads: int, groups: int, dk: int, dv: int, chunked: bool) -> None:
+        """The gated delta rule along each sequence of the step (csrc/delta.cu): S <- diag(g) S; u = beta (v - S^T k);
+        S <- S + k u^T; out = S^T q, with g = exp(-rate softplus(z + bias)) and beta = sigmoid(b); S float32 [heads, dk, dv] at
+        `state_offset` bytes of each slot.  q, k [rows, groups * dk], v, out [rows, heads * dv], z [rows, heads * dk], bias
+        [heads * dk], rate [heads]: float32; b [rows, heads] in the run's type.  `chunked`: 64 tokens at a time instead of one
+        (the results differ by rounding only)."""
+        lib = self.part_library("delta")
+        if any(t.dtype != torch.float32 or t.stride(-1) != 1 for t in (q, k, v, z, bias, rate, out)) or b.stride(1) != 1:
+            raise KernelError("delta_rule: float32 rows with contiguous elements")
+        if q.shape[1] != groups * dk or k.shape[1] != groups * dk or v.shape[1] != heads * dv or z.shape[1] != heads * dk \
+                or bias.numel() != heads * dk or rate.numel() != heads or b.shape[1] < heads or out.shape[1] != heads * dv:
+            raise KernelError("delta_rule: the rows do not hold the heads")
+        rows = out.shape[0]
+        need = lib.braid_delta_work_floats(rows, ctx.n_seqs, int(ctx.max_q_len), heads, dk, dv) if chunked else 0
+        work = torch.empty(need, dtype=torch.float32, device=out.device) if need > 0 else None
+        self.launches += 3 if work is not None else 1
+        self._check_lib(lib, lib.braid_delta_rule(
+            q.data_ptr(), q.stride(0), k.data_ptr(), k.stride(0), v.data_ptr(), v.stride(0), z.data_ptr(), z.stride(0),
+            bias.data_ptr(), rate.data_ptr(), b.data_ptr(), b.stride(0), dtype_code(b.dtype), out.data_ptr(), out.stride(0),
+            *self._state_args(state, state_offset), ctx.q_start.data_ptr(), ctx.q_len.data_ptr(), ctx.slot_ids.data_ptr(), rows,
+            ctx.n_seqs, int(ctx.max_q_len), heads, groups, dk, dv, _ptr(work), need, self._stream()), "delta_rule")
+
+    def delta_gated_norm(self, y: torch.Tensor, gate: torch.Tensor, w: torch.Tensor, out: torch.Tensor, token_seq: torch.Tensor,
+                         group: int, eps: float) -> None:
+        """`gated_norm` with a float32 gate that goes through a sigmoid: groups of y's columns normed, times w, gated."""
+        lib = self.part_library("delta")
+        rows, width = y.shape
+        if y.dtype != torch.float32 or not y.is_contiguous() or gate.dtype != torch.float32 or gate.stride(1) != 1 \
+                or w.dtype != out.dtype or out.stride(1) != 1 or w.numel() not in (group, width) or tuple(out.shape) != (rows, width) \
+                or gate.shape[1] < width:
+            raise KernelError("delta_gated_norm: y contiguous float32, gate float32; w, out of one element type")
+        self.launches += 1
+        self._check_lib(lib, lib.braid_delta_gated_norm(
+            y.data_ptr(), gate.data_ptr(), gate.stride(0), w.data_ptr(), w.numel(), out.data_ptr(), out.stride(0),
+            token_seq.data_ptr(), dtype_code(out.dtype), rows, width, group, float(eps), self._stream()), "delta_gated_norm")
 
     def linear_scan(self, q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, gate: torch.Tensor, gate_bias: torch.Tensor,
                     out: torch.Tensor, state: torch.Tensor, state_offset: int, ctx, heads: int, groups: int, dk: int,

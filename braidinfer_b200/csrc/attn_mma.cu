@@ -15,7 +15,7 @@
 // position p iff j <= p and (window == 0 or p - j < window); with keep_first > 0 the sequence's first
 // keep_first positions stay visible beyond the window (their tiles are walked before the window's).
 // head_scale is a factor a head on the scores; bias_slope and bias_rate take r1 ln(1 + r2 (p - j)) off the score of
-// key j, a number a head each.  Compiled with -DBRAID_VH=<n> (default 1) and called with
+// key j, a number a head each; softcap caps the scores (softcap.cuh).  Compiled with -DBRAID_VH=<n> (default 1) and called with
 // vh_total > 0, every query head applies its probabilities to the values of every kv head as well as
 // sharing the keys of its own kv head, n value heads a CTA (the grid grows by vh_total / n), and writes the results at
 // virtual heads head * vh_total + value head: what a mix of the heads' probabilities after the softmax needs
@@ -24,6 +24,7 @@
 // Replaces the reference's op_attn_paged, one 256-thread block per query head walking
 // the context token by token (kernels/megakernel_ops.hip:2150-2343).
 #include "common.cuh"
+#include "softcap.cuh"
 
 #ifndef BRAID_HD
 #error "compile with -DBRAID_HD=<head_dim>"
@@ -48,7 +49,8 @@ struct AttnMmaArgs {
     const int* kv_before;        // [n_seqs] cache length before this step
     int q_row_stride, out_row_stride;
     int nqh, nkh, table_cols, window, n_splits;
-    float scale_log2;            // softmax scale * log2(e)
+    float scale_log2;            // softmax scale * log2(e); with cap_log2 > 0: scale / cap, the tanh's argument
+    float cap_log2;              // the cap on the scores * log2(e); 0: not capped
     int num_pages;               // pages of the cache: a table entry outside [0, num_pages) is never followed
     int* error_flag;             // raised when a tile of visible keys has no page or one outside the cache
     int has_sink;                // the denominator counts one more term 2^sink_log2 that has no value (an attention sink)
@@ -275,6 +277,7 @@ attn_mma_kernel(AttnMmaArgs a) {
                 s[nb][0] *= sc_a; s[nb][1] *= sc_a;
                 s[nb][2] *= sc_b; s[nb][3] *= sc_b;
             }
+            if (a.cap_log2 > 0.f) softcap_scores<BN / 2>(&s[0][0], 1.f, a.cap_log2);
         }
 #pragma unroll
         for (int nb = 0; nb < BN / 8; ++nb) {
@@ -506,7 +509,7 @@ extern "C" int braid_attn_mma(const void* q, void* out, void* partial, const voi
                               int nqh, int nkh, int hd, int table_cols, int num_pages, int window, int n_splits, int kind,
                               float scale, int has_sink, float sink_score, float out_scale, const float* head_sinks,
                               const void* head_gate, long long gate_stride, int keep_first, const float* head_scale,
-                              const float* bias_slope, const float* bias_rate, int vh0, int vh_total, int* error_flag,
+                              const float* bias_slope, const float* bias_rate, float softcap, int vh0, int vh_total, int* error_flag,
                               void* stream) {
     if (rows <= 0 || n_seqs <= 0) return BRAID_OK;
     if (head_sinks) has_sink = 1;
@@ -516,6 +519,7 @@ extern "C" int braid_attn_mma(const void* q, void* out, void* partial, const voi
     if (vh_total > 0 && (has_sink || head_gate)) BRAID_REFUSE("attn_mma: values of every kv head go with an ordinary softmax without sink or gate");
     if (keep_first < 0) BRAID_REFUSE("attn_mma: keep_first=%d must not be negative", keep_first);
     if (!bias_slope != !bias_rate) BRAID_REFUSE("attn_mma: a distance bias has a slope and a rate a head");
+    if (softcap > 0.f && bias_slope) BRAID_REFUSE("attn_mma: a cap on the scores and a distance bias are not combined");
     if (window <= 0) keep_first = 0;
     // a gate a head rides on the last kernel that touches a row: the merge of the slices, or the attention itself
     const __nv_bfloat16* gate_here = n_splits > 1 ? nullptr : (const __nv_bfloat16*)head_gate;
@@ -529,7 +533,7 @@ extern "C" int braid_attn_mma(const void* q, void* out, void* partial, const voi
     if (n_splits > 1 && !partial) BRAID_REFUSE("attn_mma: n_splits > 1 needs the partial buffer");
     AttnMmaArgs a{(const __nv_bfloat16*)q, (__nv_bfloat16*)out, (float*)partial, (const __nv_bfloat16*)cache, page_table,
                   q_start, q_len, kv_before, q_row_stride, out_row_stride, nqh, nkh, table_cols, window, n_splits,
-                  scale * 1.4426950408889634f, num_pages, error_flag, has_sink, sink_score * 1.4426950408889634f, out_scale,
+                  softcap > 0.f ? scale / softcap : scale * 1.4426950408889634f, softcap * 1.4426950408889634f, num_pages, error_flag, has_sink, sink_score * 1.4426950408889634f, out_scale,
                   head_sinks, gate_here, gate_stride, keep_first, head_scale, bias_slope, bias_rate, vh0, vh_total};
     cudaStream_t s = (cudaStream_t)stream;
     int rc;
@@ -592,6 +596,6 @@ extern "C" int braid_attn_mma_noalloc(const void* q, void* out, const void* cach
     }
     return braid_attn_mma(q, out, n_splits > 1 ? g_noalloc_ptr[dev] : nullptr, cache, page_table, q_start, q_len,
                           kv_before, token_seq, q_row_stride, out_row_stride, rows, n_seqs, max_q_len, nqh, nkh, hd,
-                          table_cols, num_pages, window, n_splits, kind, scale, 0, 0.f, 1.f, nullptr, nullptr, 0, 0, nullptr, nullptr, nullptr, 0, 0,
+                          table_cols, num_pages, window, n_splits, kind, scale, 0, 0.f, 1.f, nullptr, nullptr, 0, 0, nullptr, nullptr, nullptr, 0.f, 0, 0,
                           error_flag, stream);
 }

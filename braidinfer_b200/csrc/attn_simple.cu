@@ -19,7 +19,7 @@
 // (token, query head, value head) and the result lies at virtual head `head * value_heads + value head`), which is
 // what a mix of the heads' probabilities after the softmax needs (pointwise.cu, head_mix).  bias_slope and bias_rate
 // (a number a head each) take r1 ln(1 + r2 (p - j)) off the score of key j: a bias that grows with the logarithm of the
-// distance instead of a rotation.
+// distance instead of a rotation.  softcap > 0 caps the scores: softcap * tanh(score / softcap).
 #include "common.cuh"
 
 struct AttnSimpleArgs {
@@ -43,6 +43,7 @@ struct AttnSimpleArgs {
     int value_heads;          // 1, or nkh: every query head reads the values of every kv head
     const float* bias_slope;  // [nqh] float32 r1 and r2 of the distance bias r1 ln(1 + r2 (p - j)); or null, both
     const float* bias_rate;
+    float softcap;            // 0: scores are not capped
 };
 
 #define ATTN_SIMPLE_WARPS 4
@@ -104,6 +105,7 @@ attn_simple_kernel(AttnSimpleArgs a) {
             float dot = 0.f;
             for (int d = 0; d < a.hd; ++d) dot = fmaf(qs[d], to_f32(kbase[d]), dot);
             s = dot * scale;
+            if (a.softcap > 0.f) s = a.softcap * tanhf(s / a.softcap);
             if (a.bias_slope) s -= r1 * log1pf(r2 * (float)(pos - j));
         }
         const float cmax = warp_max(s);
@@ -151,7 +153,7 @@ extern "C" int braid_attn_simple(const void* q, void* out, int dtype, const void
                                  int page_size, int table_cols, int num_pages, int window, float scale,
                                  int has_sink, float sink_score, float out_scale, const float* head_sinks,
                                  const void* head_gate, long long gate_stride, int keep_first, const float* head_scale,
-                                 int value_heads, const float* bias_slope, const float* bias_rate, int* error_flag,
+                                 int value_heads, const float* bias_slope, const float* bias_rate, float softcap, int* error_flag,
                                  void* stream) {
     if (rows <= 0) return BRAID_OK;
     if (!error_flag) BRAID_REFUSE("attn_simple: error_flag is required");
@@ -162,10 +164,11 @@ extern "C" int braid_attn_simple(const void* q, void* out, int dtype, const void
     if (value_heads > 1 && head_gate) BRAID_REFUSE("attn_simple: a gate a head does not go with values of every kv head");
     if (keep_first < 0) BRAID_REFUSE("attn_simple: keep_first=%d must not be negative", keep_first);
     if (!bias_slope != !bias_rate) BRAID_REFUSE("attn_simple: a distance bias has a slope and a rate a head");
+    if (softcap > 0.f && bias_slope) BRAID_REFUSE("attn_simple: a cap on the scores and a distance bias are not combined");
     if (window <= 0) keep_first = 0;
     AttnSimpleArgs a{q, out, cache, page_table, positions, token_seq, q_row_stride, out_row_stride,
                      rows, nqh, nkh, hd, page_size, table_cols, num_pages, window, scale, has_sink || head_sinks != nullptr, sink_score, out_scale, error_flag, head_sinks, head_gate, gate_stride,
-                     keep_first, head_scale, value_heads, bias_slope, bias_rate};
+                     keep_first, head_scale, value_heads, bias_slope, bias_rate, softcap};
     const long long items = (long long)rows * nqh * value_heads;
     const long long blocks = (items + ATTN_SIMPLE_WARPS - 1) / ATTN_SIMPLE_WARPS;
     if (blocks > 0x7fffffffLL) BRAID_REFUSE("attn_simple: %lld (token, head) pairs exceed one launch", items);

@@ -33,10 +33,12 @@
 //
 // Visibility is the rule of the whole library: key j is visible to the query at position
 // p iff j <= p and (window == 0 or p - j < window).  The kernel's second form (BIAS) takes r1 log2(1 + r2 (p - j)) off
-// the scores (in units of log2), r1 and r2 a number a head each, before the maximum is looked at.  Replaces, for prompts, the
+// the scores (in units of log2), r1 and r2 a number a head each, before the maximum is looked at; the third (CAP) caps the
+// scores (softcap.cuh).  Replaces, for prompts, the
 // reference's op_attn_paged (kernels/megakernel_ops.hip:2150-2343), as attn_mma.cu does;
 // attn_mma.cu stays the kernel for other head sizes and the twin this one is tested against.
 #include "common.cuh"
+#include "softcap.cuh"
 #include "tcgen05.cuh"
 
 #ifndef BRAID_HD
@@ -156,7 +158,7 @@ struct AttnTcArgs {
     const int* q_len;
     const int* kv_before;
     int out_row_stride, nqh, nkh, table_cols, window;
-    float scale_log2;
+    float scale_log2;            // scale * log2(e); CAP: scale / cap, the tanh's argument
     int num_pages;
     int* error_flag;
     int has_sink;                // the denominator counts one more term 2^sink_log2 that has no value (an attention sink)
@@ -167,12 +169,17 @@ struct AttnTcArgs {
     long long gate_stride;
     const float* bias_slope;     // BIAS: [nqh] float32 r1 and r2 of the distance bias r1 ln(1 + r2 (p - j))
     const float* bias_rate;
+    float cap_log2;              // CAP: the cap on the scores * log2(e)
 };
 
-template <bool BIAS>
+#define FA_PLAIN 0
+#define FA_BIAS 1
+#define FA_CAP 2
+template <int FORM>
 __global__ void __launch_bounds__(FA_THREADS, 2)
 attn_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_kv, AttnTcArgs a) {
     constexpr int HD = BRAID_HD;
+    constexpr bool BIAS = FORM == FA_BIAS, CAP = FORM == FA_CAP;
     pdl_trigger();
     // the swizzled tiles want 1024-byte alignment; two CTAs an SM leave no room for slack, so
     // the start of dynamic shared memory is checked instead of rounded up
@@ -349,8 +356,8 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant_
         float m = -INFINITY, l = 0.f;
         float r1 = 0.f, r2 = 0.f;                             // the row's distance bias
         if (BIAS && valid) { r1 = a.bias_slope[head0 + hl]; r2 = a.bias_rate[head0 + hl]; }
-        // with the bias the scores are scaled as it is taken off
-        const float sc = BIAS ? 1.f : a.scale_log2;
+        // with the bias or the cap the scores are scaled there
+        const float sc = BIAS || CAP ? 1.f : a.scale_log2;
         bool ok = true;
         for (int j = 0; j < n_tiles && ok; ++j) {
             const int st = j & 1;
@@ -368,6 +375,7 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant_
                 for (int i = 0; i < 64; ++i)
                     sv[i] = fmaf(sv[i], a.scale_log2, -r1 * __log2f(fmaf(r2, d0 - (float)i, 1.f)));
             }
+            if (CAP) softcap_scores<64>(sv, a.scale_log2, a.cap_log2);
             float mx0 = -INFINITY, mx1 = -INFINITY, mx2 = -INFINITY, mx3 = -INFINITY;
             if (all_visible) {
                 if (valid) {
@@ -485,7 +493,7 @@ extern "C" int braid_attn_tc(const void* q, void* out, const void* cache, long l
                              int q_row_stride, int out_row_stride, int rows, int n_seqs, int max_q_len,
                              int nqh, int nkh, int hd, int table_cols, int window, float scale,
                              int has_sink, float sink_score, float out_scale, const float* head_sinks, const void* head_gate,
-                             long long gate_stride, const float* bias_slope, const float* bias_rate, int* error_flag,
+                             long long gate_stride, const float* bias_slope, const float* bias_rate, float softcap, int* error_flag,
                              void* stream) {
     if (rows <= 0 || n_seqs <= 0) return BRAID_OK;
     if (head_sinks) has_sink = 1;
@@ -495,6 +503,7 @@ extern "C" int braid_attn_tc(const void* q, void* out, const void* cache, long l
     if ((out_row_stride % 8) || ((uintptr_t)out & 15)) BRAID_REFUSE("attn_tc: out rows must be 16-byte aligned");
     if (!error_flag) BRAID_REFUSE("attn_tc: error_flag is required");
     if (!bias_slope != !bias_rate) BRAID_REFUSE("attn_tc: a distance bias has a slope and a rate a head");
+    if (softcap > 0.f && bias_slope) BRAID_REFUSE("attn_tc: a cap on the scores and a distance bias are not combined");
     TcEncodeTiledFn fn = tc_encode_tiled_fn();
     if (!fn) BRAID_REFUSE("attn_tc: the driver does not export cuTensorMapEncodeTiled");
     const int g = nqh / nkh;
@@ -522,8 +531,9 @@ extern "C" int braid_attn_tc(const void* q, void* out, const void* cache, long l
     }
     static bool configured = false;
     if (!configured) {
-        cudaError_t e = cudaFuncSetAttribute(attn_tc_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, FA_SMEM);
-        if (e == cudaSuccess) e = cudaFuncSetAttribute(attn_tc_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, FA_SMEM);
+        cudaError_t e = cudaFuncSetAttribute(attn_tc_kernel<FA_PLAIN>, cudaFuncAttributeMaxDynamicSharedMemorySize, FA_SMEM);
+        if (e == cudaSuccess) e = cudaFuncSetAttribute(attn_tc_kernel<FA_BIAS>, cudaFuncAttributeMaxDynamicSharedMemorySize, FA_SMEM);
+        if (e == cudaSuccess) e = cudaFuncSetAttribute(attn_tc_kernel<FA_CAP>, cudaFuncAttributeMaxDynamicSharedMemorySize, FA_SMEM);
         if (e != cudaSuccess) { braid_set_error("attn_tc: cannot reserve %d bytes of shared memory: %s", FA_SMEM, cudaGetErrorString(e)); return (int)e; }
         configured = true;
     }
@@ -532,9 +542,10 @@ extern "C" int braid_attn_tc(const void* q, void* out, const void* cache, long l
         BRAID_REFUSE("attn_tc: the step exceeds the grid limits (%lld token tiles, %d sequences)", gx, n_seqs);
     const long long num_pages = cache_rows / (2LL * nkh * FA_PAGE);
     AttnTcArgs a{(__nv_bfloat16*)out, page_table, q_start, q_len, kv_before, out_row_stride, nqh, nkh, table_cols, window,
-                 scale * 1.4426950408889634f, (int)num_pages, error_flag, has_sink, sink_score * 1.4426950408889634f, out_scale,
-                 head_sinks, (const __nv_bfloat16*)head_gate, gate_stride, bias_slope, bias_rate};
-    braid_launch(bias_slope ? attn_tc_kernel<true> : attn_tc_kernel<false>, dim3(nkh * hchunks, n_seqs, (unsigned)gx), dim3(FA_THREADS), FA_SMEM,
+                 softcap > 0.f ? scale / softcap : scale * 1.4426950408889634f, (int)num_pages, error_flag, has_sink, sink_score * 1.4426950408889634f, out_scale,
+                 head_sinks, (const __nv_bfloat16*)head_gate, gate_stride, bias_slope, bias_rate,
+                 softcap * 1.4426950408889634f};
+    braid_launch(softcap > 0.f ? attn_tc_kernel<FA_CAP> : bias_slope ? attn_tc_kernel<FA_BIAS> : attn_tc_kernel<FA_PLAIN>, dim3(nkh * hchunks, n_seqs, (unsigned)gx), dim3(FA_THREADS), FA_SMEM,
                  (cudaStream_t)stream, mq, mkv, a);
     BRAID_LAUNCH_CHECK();
 }

@@ -32,9 +32,10 @@ CORE_SOURCES = ["errors.cu", "elementwise.cu", "pointwise.cu", "attn_simple.cu",
                 "fused_reduce.cu", "sampling.cu"]
 # Kernels that only some models use: each a library of its own, compiled when a model that needs it is built.
 PART_SOURCES = {"latent": ["errors.cu", "latent.cu"], "moe": ["errors.cu", "moe.cu"], "scan": ["errors.cu", "scan.cu"],
-                "streams": ["errors.cu", "streams.cu"]}
+                "streams": ["errors.cu", "streams.cu"], "conv": ["errors.cu", "conv_heads.cu"],
+                "delta": ["errors.cu", "delta.cu"]}
 HEADERS = ["common.cuh", "rowscale.cuh", "streamk.cuh", "tcgen05.cuh", "attn_noalloc.h", "page.h", "trace.cuh",
-           "mma_tile.cuh"]
+           "mma_tile.cuh", "softcap.cuh", "gated_norm.cuh"]
 
 
 class BuildError(RuntimeError):

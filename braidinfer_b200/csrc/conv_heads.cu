@@ -1,0 +1,363 @@
+// A short causal convolution over time on projected heads, and what the heads need right after it, in one kernel:
+//     u_t = x_t + bias                                        (x: projected rows in the run's type, bias optional)
+//     y_t[c] = sum_j w[c, j] u_(t - taps + 1 + j)[c]          (zeros before the sequence's start)
+// then, head by head, silu, a norm (root mean square with a weight of the head's size; or unit length,
+// y / sqrt(sum y^2 + eps)), a constant factor, a rotation of the head's first numbers (neighbouring pairs, or halves), zeros
+// up to a padded head size, and the store: rows of a buffer (float32 or the run's type), or the key or value plane of the
+// paged cache at the token's position.
+//
+// The channels fall into up to three segments (queries, keys, values), each with heads of its own size and its own choice
+// of these.  A sequence's state is its last taps - 1 rows u, float32 [taps - 1][channels] at state + slot * state_stride +
+// state_offset, the newest last, zero at the start: rows before the step come from there.  A sequence that brings one token
+// has its state moved on by the threads that read it; the others by conv_heads_state_kernel.  Everything is float32
+// arithmetic.
+#include "common.cuh"
+
+#define CONV_MAX_SEGS 3
+#define CONV_NORM_NONE 0
+#define CONV_NORM_RMS 1
+#define CONV_NORM_UNIT 2
+#define CONV_MAX_SIZE 512
+
+struct ConvSegment {
+    int heads, size, pad;        // heads of `size` channels, written as heads of `pad` numbers
+    int norm, silu, rotate;
+    int plane;                   // -1: to `out`; 0, 1: the cache's key or value plane
+    float factor;
+    const void* weight;          // CONV_NORM_RMS: [size] in the run's type
+    void* out;                   // [rows, out_stride], head h at column h * pad
+    long long out_stride;
+};
+
+struct ConvHeadsArgs {
+    const void* x;               // [rows, x_stride]: segment after segment, head after head
+    long long x_stride;
+    const void* bias;            // [channels] or null
+    const void* w;               // [channels, taps]
+    uint8_t* state;              // null with one tap
+    long long state_stride, state_offset;
+    const int *token_seq, *positions, *q_start, *q_len, *slot_ids;
+    const int* page_table;       // [n_seqs, table_cols]
+    void* cache;                 // one layer: [page][2][kv heads][page_size][pad], or null
+    int page_size, table_cols, num_pages;
+    const float* inv_freq;       // [rope_dim / 2]
+    int rope_dim, adjacent;
+    float amp, eps;
+    int rows, channels, taps, n_segs;
+    int* error_flag;
+    ConvSegment seg[CONV_MAX_SEGS];
+};
+
+// Where head `h` of segment s and row `row` is stored (its first number), or null.
+template <typename T, typename TO>
+__device__ __forceinline__ TO* conv_dst(const ConvHeadsArgs& a, const ConvSegment& s, int h, int row, int seq, bool flag) {
+    if (s.plane < 0) return (TO*)s.out + (size_t)row * s.out_stride + (size_t)h * s.pad;
+    if (!a.cache) return nullptr;
+    const int pos = a.positions[row];
+    const int block = pos / a.page_size, off = pos - block * a.page_size;
+    const int page = (block < a.table_cols) ? a.page_table[(size_t)seq * a.table_cols + block] : -1;
+    if (page < 0 || page >= a.num_pages) {
+        if (flag) atomicExch(a.error_flag, 1);
+        return nullptr;
+    }
+    return (TO*)a.cache + ((((size_t)page * 2 + s.plane) * s.heads + h) * a.page_size + off) * s.pad;
+}
+
+// 16 bytes of neighbouring channels a thread, LPH lanes a head, RPT neighbouring rows a thread: for sizes, strides and taps
+// that allow it (neighbouring pairs in the rotation).  TO: the type of what is stored.
+template <typename T, typename TO, int TAPS, int LPH, int RPT>
+__global__ void __launch_bounds__(128)
+conv_heads_vec_kernel(ConvHeadsArgs a) {
+    constexpr int VEC = 16 / sizeof(T), HPC = 128 / LPH, SPAN = RPT + TAPS - 1;
+    pdl_trigger();
+    const int sub = threadIdx.x / LPH, l = threadIdx.x % LPH, i0 = l * VEC;
+    // which segment and head: the CTAs of a row walk the segments' groups of HPC heads
+    int g = blockIdx.x, si = 0, c_seg = 0;
+    for (; si < a.n_segs - 1; ++si) {
+        const int groups = (a.seg[si].heads + HPC - 1) / HPC;
+        if (g < groups) break;
+        g -= groups;
+        c_seg += a.seg[si].heads * a.seg[si].size;
+    }
+    const ConvSegment& s = a.seg[si];
+    const int head = g * HPC + sub;
+    const bool live = head < s.heads, in = live && i0 < s.size;
+    const int c0 = c_seg + head * s.size + i0;
+    float wl[VEC * TAPS], bl[VEC];
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) bl[e] = 0.f;
+    if (in) {
+#pragma unroll
+        for (int u = 0; u < TAPS; ++u) load_run<T, VEC>((const T*)a.w + (size_t)c0 * TAPS + u * VEC, wl + u * VEC);
+        if (a.bias) load_run<T, VEC>((const T*)a.bias + c0, bl);
+    }
+    pdl_wait();
+    const int row0 = blockIdx.y * RPT;
+    float xin[SPAN][VEC];
+#pragma unroll
+    for (int u = 0; u < SPAN; ++u) {
+        const int r = row0 - (TAPS - 1) + u;
+        if (in && r >= 0 && r < a.rows) {
+            load_run<T, VEC>((const T*)a.x + (size_t)r * a.x_stride + c0, xin[u]);
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) xin[u][e] += bl[e];
+        } else {
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) xin[u][e] = 0.f;
+        }
+    }
+    float nw[VEC];
+    if (in && s.norm == CONV_NORM_RMS) load_run<T, VEC>((const T*)s.weight + i0, nw);
+#pragma unroll
+    for (int rr = 0; rr < RPT; ++rr) {
+        const int row = row0 + rr;
+        if (row >= a.rows) break;                          // the whole CTA: rows are the grid's
+        const int seq = a.token_seq[row];
+        if (seq < 0) continue;
+        const int o = row - a.q_start[seq];
+        float* st = a.state ? (float*)(a.state + (size_t)a.slot_ids[seq] * a.state_stride + a.state_offset) : nullptr;
+        float y[VEC];
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) y[e] = 0.f;
+        if (in) {
+            float old[TAPS > 1 ? TAPS - 1 : 1][VEC];       // rows before the step that this row's taps reach
+#pragma unroll
+            for (int j = 0; j < TAPS; ++j) {
+                const int back = TAPS - 1 - j;
+                float xv[VEC];
+                if (o - back >= 0) {
+#pragma unroll
+                    for (int e = 0; e < VEC; ++e) xv[e] = xin[rr + j][e];
+                } else {
+                    const float* sp = st + (size_t)(TAPS - 1 + (o - back)) * a.channels + c0;
+#pragma unroll
+                    for (int e = 0; e < VEC; e += 4) load_run<float, 4>(sp + e, xv + e);
+                }
+                if (j < TAPS - 1) {
+#pragma unroll
+                    for (int e = 0; e < VEC; ++e) old[j][e] = xv[e];
+                }
+#pragma unroll
+                for (int e = 0; e < VEC; ++e) y[e] = fmaf(wl[e * TAPS + j], xv[e], y[e]);
+            }
+            if (TAPS > 1 && a.q_len[seq] == 1) {           // one token: nobody else reads these channels of the state
+#pragma unroll
+                for (int j = 0; j < TAPS - 1; ++j)
+#pragma unroll
+                    for (int e = 0; e < VEC; e += 4)
+                        store_run<float, 4>(st + (size_t)j * a.channels + c0 + e, (j < TAPS - 2 ? old[j + 1 < TAPS - 1 ? j + 1 : j] : xin[rr + TAPS - 1]) + e);
+            }
+        }
+        if (s.silu) {
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) y[e] = sizeof(T) == 2 ? glu_act_fast(y[e], BRAID_ACT_SILU) : silu_f32(y[e]);
+        }
+        if (s.norm != CONV_NORM_NONE) {
+            float ss = 0.f;
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) ss = fmaf(y[e], y[e], ss);
+#pragma unroll
+            for (int b = LPH / 2; b > 0; b >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, b);
+            const float r = s.factor / sqrtf((s.norm == CONV_NORM_RMS ? ss / (float)s.size : ss) + a.eps);
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) y[e] *= s.norm == CONV_NORM_RMS && in ? r * nw[e] : r;
+        } else {
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) y[e] *= s.factor;
+        }
+        if (!live || i0 >= s.pad) continue;
+        if (s.rotate && i0 < a.rope_dim) {
+            const float pos = (float)a.positions[row];
+#pragma unroll
+            for (int e = 0; e < VEC; e += 2) {
+                const int p = (i0 + e) >> 1;
+                if (2 * p < a.rope_dim) {
+                    float sn, cs;
+                    sincosf(pos * a.inv_freq[p], &sn, &cs);
+                    sn *= a.amp; cs *= a.amp;
+                    const float u = y[e], v = y[e + 1];
+                    y[e] = u * cs - v * sn;
+                    y[e + 1] = v * cs + u * sn;
+                }
+            }
+        }
+        TO* dst = conv_dst<T, TO>(a, s, head, row, seq, l == 0);
+        if (!dst) continue;
+        constexpr int VO = 16 / sizeof(TO) < VEC ? 16 / sizeof(TO) : VEC;
+#pragma unroll
+        for (int e = 0; e < VEC; e += VO) store_run<TO, VO>(dst + i0 + e, y + e);
+    }
+}
+
+// Any sizes, taps and pairing: a warp a (row, head), lane-strided pairs of channels.
+#define CONV_ANY_WARPS 4
+template <typename T, typename TO>
+__global__ void __launch_bounds__(CONV_ANY_WARPS * 32)
+conv_heads_kernel(ConvHeadsArgs a) {
+    __shared__ float stage[CONV_ANY_WARPS][CONV_MAX_SIZE];
+    pdl_trigger();
+    pdl_wait();
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    int h = blockIdx.x * CONV_ANY_WARPS + warp, si = 0, c_seg = 0;
+    for (; si < a.n_segs; ++si) {
+        if (h < a.seg[si].heads) break;
+        h -= a.seg[si].heads;
+        c_seg += a.seg[si].heads * a.seg[si].size;
+    }
+    if (si == a.n_segs) return;
+    const ConvSegment& s = a.seg[si];
+    const int row = blockIdx.y, seq = a.token_seq[row];
+    if (seq < 0) return;
+    const int o = row - a.q_start[seq], c0 = c_seg + h * s.size;
+    float* st = a.state ? (float*)(a.state + (size_t)a.slot_ids[seq] * a.state_stride + a.state_offset) : nullptr;
+    const bool alone = a.q_len[seq] == 1;
+    float* y = stage[warp];
+    float ss = 0.f;
+    for (int i = lane; i < s.size; i += 32) {
+        const int c = c0 + i;
+        const float b = a.bias ? to_f32(((const T*)a.bias)[c]) : 0.f;
+        float acc = 0.f, u = 0.f;
+        for (int j = 0; j < a.taps; ++j) {
+            const int back = a.taps - 1 - j;
+            if (o - back >= 0) u = to_f32(((const T*)a.x)[(size_t)(row - back) * a.x_stride + c]) + b;
+            else u = st[(size_t)(a.taps - 1 + (o - back)) * a.channels + c];
+            // one token: the state moves on behind the reads (entry j - 1 takes what entry j held; nobody else reads it)
+            if (alone && j > 0) st[(size_t)(j - 1) * a.channels + c] = u;
+            acc = fmaf(to_f32(((const T*)a.w)[(size_t)c * a.taps + j]), u, acc);
+        }
+        if (s.silu) acc = silu_f32(acc);
+        ss = fmaf(acc, acc, ss);
+        y[i] = acc;
+    }
+    float r = s.factor;
+    if (s.norm != CONV_NORM_NONE) {
+        ss = warp_sum(ss);
+        r = s.factor / sqrtf((s.norm == CONV_NORM_RMS ? ss / (float)s.size : ss) + a.eps);
+    }
+    __syncwarp();
+    for (int i = lane; i < s.size; i += 32) y[i] *= s.norm == CONV_NORM_RMS ? r * to_f32(((const T*)s.weight)[i]) : r;
+    __syncwarp();
+    if (s.rotate) {
+        const int half = a.rope_dim / 2;
+        const float pos = (float)a.positions[row];
+        for (int p = lane; p < half; p += 32) {
+            float sn, cs;
+            sincosf(pos * a.inv_freq[p], &sn, &cs);
+            sn *= a.amp; cs *= a.amp;
+            const int e0 = a.adjacent ? 2 * p : p, e1 = a.adjacent ? 2 * p + 1 : p + half;
+            const float u = y[e0], v = y[e1];
+            y[e0] = u * cs - v * sn;
+            y[e1] = v * cs + u * sn;
+        }
+        __syncwarp();
+    }
+    TO* dst = conv_dst<T, TO>(a, s, h, row, seq, lane == 0);
+    if (!dst) return;
+    for (int i = lane; i < s.pad; i += 32) dst[i] = from_f32<TO>(i < s.size ? y[i] : 0.f);
+}
+
+// The state after the step of every sequence that brings more than one token: its last taps - 1 rows.  One thread per
+// (sequence, channel) reads what it needs of the old state before it writes, in rising order.
+template <typename T>
+__global__ void __launch_bounds__(256)
+conv_heads_state_kernel(ConvHeadsArgs a, int n_seqs) {
+    pdl_trigger();
+    pdl_wait();
+    const int c = blockIdx.x * blockDim.x + threadIdx.x, seq = blockIdx.y;
+    if (c >= a.channels || seq >= n_seqs) return;
+    const int n = a.q_len[seq], r0 = a.q_start[seq], keep = a.taps - 1;
+    if (n <= 1) return;
+    const float b = a.bias ? to_f32(((const T*)a.bias)[c]) : 0.f;
+    float* st = (float*)(a.state + (size_t)a.slot_ids[seq] * a.state_stride + a.state_offset);
+    for (int i = 0; i < keep; ++i) {
+        const int o = n - keep + i;                  // the step's token that entry i holds, if not negative
+        st[(size_t)i * a.channels + c] = o >= 0 ? to_f32(((const T*)a.x)[(size_t)(r0 + o) * a.x_stride + c]) + b
+                                                : st[(size_t)(i + n) * a.channels + c];
+    }
+}
+
+template <typename T, typename TO, int TAPS, int LPH>
+static void launch_conv_vec(const ConvHeadsArgs& a, cudaStream_t s) {
+    constexpr int HPC = 128 / LPH;
+    int groups = 0;
+    for (int i = 0; i < a.n_segs; ++i) groups += (a.seg[i].heads + HPC - 1) / HPC;
+    // neighbouring rows a thread: four where the rows alone fill the machine
+    if ((long long)a.rows * groups >= 148 * 16)
+        braid_launch(conv_heads_vec_kernel<T, TO, TAPS, LPH, 4>, dim3(groups, (a.rows + 3) / 4), dim3(128), 0, s, a);
+    else
+        braid_launch(conv_heads_vec_kernel<T, TO, TAPS, LPH, 1>, dim3(groups, a.rows), dim3(128), 0, s, a);
+}
+
+template <typename T, typename TO>
+static void launch_conv(const ConvHeadsArgs& a, bool wide, int lanes, cudaStream_t s) {
+    if (wide) {
+#define CONV_LPH(TAPS)                                                        \
+    do {                                                                      \
+        if (lanes <= 4) launch_conv_vec<T, TO, TAPS, 4>(a, s);                \
+        else if (lanes <= 8) launch_conv_vec<T, TO, TAPS, 8>(a, s);           \
+        else if (lanes <= 16) launch_conv_vec<T, TO, TAPS, 16>(a, s);         \
+        else launch_conv_vec<T, TO, TAPS, 32>(a, s);                          \
+    } while (0)
+        if (a.taps == 2) CONV_LPH(2);
+        else if (a.taps == 3) CONV_LPH(3);
+        else CONV_LPH(4);
+#undef CONV_LPH
+        return;
+    }
+    int heads = 0;
+    for (int i = 0; i < a.n_segs; ++i) heads += a.seg[i].heads;
+    braid_launch(conv_heads_kernel<T, TO>, dim3((heads + CONV_ANY_WARPS - 1) / CONV_ANY_WARPS, a.rows), dim3(CONV_ANY_WARPS * 32), 0, s, a);
+}
+
+// `segs`: n_segs records of 7 ints {heads, size, pad, norm, silu, rotate, plane}; factors, weights, outs, out_strides: one
+// entry a segment.  out_f32: what goes to `outs` is float32 whatever the run's type (no cache then).
+extern "C" int braid_conv_heads(const void* x, long long x_stride, const void* bias, const void* w, int dtype, void* state,
+                                long long state_stride, long long state_offset, const int* token_seq, const int* positions,
+                                const int* q_start, const int* q_len, const int* slot_ids, const int* page_table, void* cache,
+                                int page_size, int table_cols, int num_pages, const float* inv_freq, int rope_dim, int adjacent,
+                                float amp, float eps, int rows, int n_seqs, int max_q_len, int taps, int n_segs, const int* segs,
+                                const float* factors, const void* const* weights, void* const* outs,
+                                const long long* out_strides, int out_f32, int* error_flag, void* stream) {
+    if (rows <= 0 || n_seqs <= 0) return BRAID_OK;
+    if (n_segs < 1 || n_segs > CONV_MAX_SEGS) BRAID_REFUSE("conv_heads: %d segments, 1 to %d are built", n_segs, CONV_MAX_SEGS);
+    if (taps < 1 || (taps > 1 && !state) || (state_offset & 3) || (state_stride & 3))
+        BRAID_REFUSE("conv_heads: %d taps want a state area in multiples of 4 bytes", taps);
+    if (dtype != BRAID_F32 && dtype != BRAID_BF16) BRAID_REFUSE("conv_heads: unknown dtype code %d", dtype);
+    if (!error_flag) BRAID_REFUSE("conv_heads: error_flag is required");
+    if (rope_dim < 0 || (rope_dim & 1)) BRAID_REFUSE("conv_heads: rope_dim=%d must be even", rope_dim);
+    ConvHeadsArgs a{x, x_stride, bias, w, (uint8_t*)(taps > 1 ? state : nullptr), state_stride, state_offset, token_seq, positions,
+                    q_start, q_len, slot_ids, page_table, cache, page_size, table_cols, num_pages, inv_freq, rope_dim, adjacent,
+                    amp, eps, rows, 0, taps, n_segs, error_flag, {}};
+    const int vec = dtype == BRAID_F32 ? 4 : 8;
+    bool wide = taps >= 2 && taps <= 4 && x_stride % vec == 0 && state_stride % 16 == 0 && state_offset % 16 == 0 &&
+                (((uintptr_t)x | (uintptr_t)bias | (uintptr_t)w | (uintptr_t)cache | (uintptr_t)state) & 15) == 0 && rows <= 65535;
+    int widest = 0;
+    for (int i = 0; i < n_segs; ++i) {
+        const int* g = segs + 7 * i;
+        a.seg[i] = ConvSegment{g[0], g[1], g[2], g[3], g[4], g[5], g[6], factors[i], weights[i], outs[i], out_strides[i]};
+        const ConvSegment& s = a.seg[i];
+        if (s.heads <= 0 || s.size <= 0 || s.pad < s.size || s.pad > CONV_MAX_SIZE || (s.rotate && rope_dim > s.size))
+            BRAID_REFUSE("conv_heads: heads of %d in %d numbers (at most %d), %d of them rotated", s.size, s.pad, CONV_MAX_SIZE, rope_dim);
+        if (s.norm == CONV_NORM_RMS && !s.weight) BRAID_REFUSE("conv_heads: this norm has a weight");
+        if (s.plane < 0 ? !s.out : (out_f32 || (cache && (!page_table || page_size <= 0 || num_pages <= 0))))
+            BRAID_REFUSE("conv_heads: a segment goes to a buffer, or to a cache with pages in the run's type");
+        if (s.plane > 1) BRAID_REFUSE("conv_heads: the cache has a key plane (0) and a value plane (1)");
+        a.channels += s.heads * s.size;
+        if (s.pad > widest) widest = s.pad;
+        wide = wide && s.size % vec == 0 && s.pad % vec == 0 && (!s.rotate || adjacent || rope_dim == 0) &&
+               (((uintptr_t)s.weight | (uintptr_t)s.out) & 15) == 0 && (s.plane >= 0 || s.out_stride % vec == 0);
+    }
+    const int lanes = (widest + vec - 1) / vec;
+    wide = wide && lanes <= 32;
+    if (rows > 65535 || n_seqs > 65535) BRAID_REFUSE("conv_heads: %d rows exceed one launch", rows);
+    cudaStream_t st = (cudaStream_t)stream;
+    if (dtype == BRAID_F32) launch_conv<float, float>(a, wide, lanes, st);
+    else if (out_f32) launch_conv<__nv_bfloat16, float>(a, wide, lanes, st);
+    else launch_conv<__nv_bfloat16, __nv_bfloat16>(a, wide, lanes, st);
+    if (taps > 1 && max_q_len > 1) {
+        const dim3 grid((a.channels + 255) / 256, n_seqs);
+        if (dtype == BRAID_F32) braid_launch(conv_heads_state_kernel<float>, grid, dim3(256), 0, st, a, n_seqs);
+        else braid_launch(conv_heads_state_kernel<__nv_bfloat16>, grid, dim3(256), 0, st, a, n_seqs);
+    }
+    BRAID_LAUNCH_CHECK();
+}

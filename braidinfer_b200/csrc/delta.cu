@@ -1,0 +1,666 @@
+// The gated delta rule with a decay a key channel: per sequence and head a state S [dk, dv], float32, and per token
+//     S <- diag(g) S;   u = beta (v - S^T k);   S <- S + k u^T;   o = S^T q
+// with g = exp(-rate softplus(z + bias)) a channel and beta = sigmoid(b) a head.  (The delta rule as a fast-weight update is
+// Schlag, Irie, Schmidhuber: "Linear Transformers Are Secretly Fast Weight Programmers", 2021; the form over chunks follows
+// Yang, Wang, Zhang, Shen, Kim: "Parallelizing Linear Transformers with the Delta Rule over Sequence Length", 2024, here with
+// a decay a channel.)  q, k, v arrive as float32 rows (convolved, of unit length and scaled: conv_heads.cu), z as float32
+// logits, b in the run's type; everything here is float32 arithmetic on the ordinary pipes.
+//
+// Short steps are walked token by token (delta_walk_kernel).  Long ones are cut into chunks of 64 tokens.  With L_t the
+// running sum of log2 g inside a chunk (a channel), S_0 the state it starts from, and every product weighed by the decay
+// between its two tokens, the walk over a chunk is
+//     A_ts = sum_i k_t k_s 2^(L_t - L_s)  (s < t),     P_ts = sum_i q_t k_s 2^(L_t - L_s)  (s <= t)
+//     (I + diag(beta) A) [W | U0] = diag(beta) [k_t 2^(L_t) | v_t]                    (forward substitution)
+//     U = U0 - W S_0
+//     O = (q_t 2^(L_t)) S_0 + P U
+//     S_64 = diag(2^(L_64)) S_0 + (k_t 2^(L_64 - L_t))^T U
+// so all but the two products with S_0 that make U and the next S run for all chunks side by side:
+//     delta_intra_kernel   W, U0, P and the decayed q and k of every chunk
+//     delta_state_kernel   chunk after chunk, a tile of value columns a CTA: U, and the state every chunk starts from
+//     delta_out_kernel     O of every chunk
+// Every 2^x above has x <= 0 where it is taken: sub-chunks of 16 tokens are related through the running sum at their edges,
+// and inside a sub-chunk 2^(L_t - L_s) is taken as 2^(L_t - edge) 2^(edge - L_s) only while the second factor stays below
+// 2^60, pair by pair beyond.  log2 g is held at or above -32 (a token that forgets more than 32 binary digits of a channel
+// forgets all that float32 holds), which keeps the running sums' own rounding small.
+#include "common.cuh"
+#include "gated_norm.cuh"
+
+#define DELTA_MAX_DK 256
+#define DELTA_CV 4
+#define DELTA_WALK_THREADS 128
+#define DELTA_C 64                 // tokens a chunk
+#define DELTA_SUB 16               // tokens a sub-chunk
+#define DELTA_NSUB (DELTA_C / DELTA_SUB)
+#define DELTA_DVT 32               // value columns a CTA of the chunk-after-chunk kernel
+#define DELTA_OUT_COLS 64          // value columns a CTA of the output kernel
+#define DELTA_LOG_MIN (-32.f)
+#define DELTA_SPREAD 60.f
+
+struct DeltaArgs {
+    const float* q; long long q_stride;          // [rows, groups * dk]
+    const float* k; long long k_stride;
+    const float* v; long long v_stride;          // [rows, heads * dv]
+    const float* z; long long z_stride;          // [rows, heads * dk]: decay logits
+    const float* bias;                           // [heads * dk]
+    const float* rate;                           // [heads], positive
+    const void* b; long long b_stride;           // [rows, heads], run type: the step sizes' logits
+    float* out; long long out_stride;            // [rows, heads * dv]
+    uint8_t* state; long long state_stride, state_offset;
+    const int *q_start, *q_len, *slot_ids;
+    int heads, groups, dk, dv;
+    // scratch of the chunked form; row-wise buffers are [rows][heads][n]
+    float *w, *u, *qd, *kd, *p;                  // n = dk4, dv4, dk4, dk4, 64
+    float *gc, *sc;                              // [seq][chunk][head][dk4], [seq][chunk][head][dk][dv4]
+    int dk4, dv4, max_chunks;
+};
+
+// log2 of a decay from its logit: -rate softplus(x) log2(e), held at DELTA_LOG_MIN
+__device__ __forceinline__ float delta_log_decay(float x, float rate) {
+    const float sp = fmaxf(x, 0.f) + log1pf(expf(-fabsf(x)));
+    return fmaxf(-rate * sp * 1.4426950408889634f, DELTA_LOG_MIN);
+}
+__device__ __forceinline__ float delta_sigmoid(float x) { return 1.f / (1.f + expf(-x)); }
+
+// ------------------------------------------------------------------ token by token
+// A CTA of 128 threads owns (head, sequence, a tile of value columns); a thread keeps R rows x 4 columns of S in registers,
+// the RG row groups of a column lie in one warp.  The read-out of the new state is taken from the decayed one,
+// S_new^T q = (g S)^T q + (k . q) u, so that a token costs one round of sums.  The state is asked for before the wait for
+// the kernel's predecessor: no other kernel of a step touches it.
+template <typename T, int RG, int R>
+__global__ void __launch_bounds__(DELTA_WALK_THREADS)
+delta_walk_kernel(DeltaArgs a) {
+    constexpr int CV = DELTA_CV, CG = DELTA_WALK_THREADS / RG, DVT = CG * CV, DKP = RG * R;
+    constexpr int TB = DKP <= 128 ? 8 : 4;
+    constexpr int NQ = TB * DKP / DELTA_WALK_THREADS, NV = TB * DVT / DELTA_WALK_THREADS;
+    static_assert((TB * DKP) % DELTA_WALK_THREADS == 0 && (TB * DVT) % DELTA_WALK_THREADS == 0, "a batch is a whole number of elements a thread");
+    __shared__ __align__(16) float sq[TB * DKP], sk[TB * DKP], sa[TB * DKP], sv[TB * DVT], sb[TB];
+    pdl_trigger();
+    const int h = blockIdx.x, seq = blockIdx.y, dvt = blockIdx.z, tid = threadIdx.x;
+    const int rg = (tid >> 1) % RG, cg = (tid & 1) | ((tid / (2 * RG)) << 1);
+    const int j0 = dvt * DVT + cg * CV;
+    const int n = a.q_len[seq], r0 = a.q_start[seq];
+    if (n <= 0) return;
+    const int dk = a.dk, dv = a.dv, g = h / (a.heads / a.groups);
+    float* S_area = (float*)(a.state + (size_t)a.slot_ids[seq] * a.state_stride + a.state_offset) + (size_t)h * dk * dv;
+    float s[R][CV];
+#pragma unroll
+    for (int e = 0; e < R; ++e)
+#pragma unroll
+        for (int x = 0; x < CV; ++x) {
+            const int i = rg * R + e, j = j0 + x;
+            s[e][x] = (i < dk && j < dv) ? S_area[(size_t)i * dv + j] : 0.f;
+        }
+    const float rate = a.rate[h];
+    pdl_wait();
+    float pq[NQ], pk[NQ], pz[NQ], pv[NV], pb = 0.f;
+    auto fetch = [&](int t0) {
+        const int nt = min(TB, n - t0);
+#pragma unroll
+        for (int w = 0; w < NQ; ++w) {
+            const int idx = tid + w * DELTA_WALK_THREADS, t = idx / DKP, i = idx - t * DKP;
+            const size_t row = (size_t)(r0 + t0 + t);
+            const bool in = t < nt && i < dk;
+            pq[w] = in ? a.q[row * a.q_stride + (size_t)g * dk + i] : 0.f;
+            pk[w] = in ? a.k[row * a.k_stride + (size_t)g * dk + i] : 0.f;
+            pz[w] = in ? a.z[row * a.z_stride + (size_t)h * dk + i] : 0.f;
+        }
+#pragma unroll
+        for (int w = 0; w < NV; ++w) {
+            const int idx = tid + w * DELTA_WALK_THREADS, t = idx / DVT, jj = idx - t * DVT, col = dvt * DVT + jj;
+            pv[w] = (t < nt && col < dv) ? a.v[(size_t)(r0 + t0 + t) * a.v_stride + (size_t)h * dv + col] : 0.f;
+        }
+        if (tid < nt) pb = to_f32(((const T*)a.b)[(size_t)(r0 + t0 + tid) * a.b_stride + h]);
+    };
+    fetch(0);
+    for (int t0 = 0; t0 < n; t0 += TB) {
+        const int nt = min(TB, n - t0);
+        __syncthreads();                                    // the batch before has been read
+#pragma unroll
+        for (int w = 0; w < NQ; ++w) {
+            const int idx = tid + w * DELTA_WALK_THREADS, t = idx / DKP, i = idx - t * DKP;
+            sq[idx] = pq[w];
+            sk[idx] = pk[w];
+            if (t < nt) sa[idx] = i < dk ? exp2f(delta_log_decay(pz[w] + a.bias[(size_t)h * dk + i], rate)) : 0.f;
+        }
+#pragma unroll
+        for (int w = 0; w < NV; ++w) sv[tid + w * DELTA_WALK_THREADS] = pv[w];
+        if (tid < nt) sb[tid] = delta_sigmoid(pb);
+        if (t0 + TB < n) fetch(t0 + TB);
+        __syncthreads();
+        for (int t = 0; t < nt; ++t) {
+            float qv[R], kv[R], av[R], vv[CV];
+#pragma unroll
+            for (int e = 0; e < R; e += 4) {
+                *reinterpret_cast<float4*>(kv + e) = *reinterpret_cast<const float4*>(sk + t * DKP + rg * R + e);
+                *reinterpret_cast<float4*>(qv + e) = *reinterpret_cast<const float4*>(sq + t * DKP + rg * R + e);
+                *reinterpret_cast<float4*>(av + e) = *reinterpret_cast<const float4*>(sa + t * DKP + rg * R + e);
+            }
+            *reinterpret_cast<float4*>(vv) = *reinterpret_cast<const float4*>(sv + t * DVT + cg * CV);
+            float sums[2 * CV + 1];
+#pragma unroll
+            for (int x = 0; x < 2 * CV + 1; ++x) sums[x] = 0.f;
+#pragma unroll
+            for (int e = 0; e < R; ++e) {
+                sums[2 * CV] = fmaf(kv[e], qv[e], sums[2 * CV]);
+#pragma unroll
+                for (int x = 0; x < CV; ++x) {
+                    s[e][x] *= av[e];
+                    sums[x] = fmaf(s[e][x], kv[e], sums[x]);
+                    sums[CV + x] = fmaf(s[e][x], qv[e], sums[CV + x]);
+                }
+            }
+#pragma unroll
+            for (int o = RG; o >= 2; o >>= 1)               // the row groups are lane bits 1 ...
+#pragma unroll
+                for (int x = 0; x < 2 * CV + 1; ++x) sums[x] += __shfl_xor_sync(0xffffffffu, sums[x], o);
+            const float beta = sb[t];
+            float u[CV];
+#pragma unroll
+            for (int x = 0; x < CV; ++x) u[x] = beta * (vv[x] - sums[x]);
+#pragma unroll
+            for (int e = 0; e < R; ++e)
+#pragma unroll
+                for (int x = 0; x < CV; ++x) s[e][x] = fmaf(kv[e], u[x], s[e][x]);
+            if (rg == 0) {
+                float* orow = a.out + (size_t)(r0 + t0 + t) * a.out_stride + (size_t)h * dv;
+#pragma unroll
+                for (int x = 0; x < CV; ++x)
+                    if (j0 + x < dv) orow[j0 + x] = fmaf(sums[2 * CV], u[x], sums[CV + x]);
+            }
+        }
+    }
+#pragma unroll
+    for (int e = 0; e < R; ++e)
+#pragma unroll
+        for (int x = 0; x < CV; ++x) {
+            const int i = rg * R + e, j = j0 + x;
+            if (i < dk && j < dv) S_area[(size_t)i * dv + j] = s[e][x];
+        }
+}
+
+// ------------------------------------------------------------------ inside every chunk
+#define DELTA_INTRA_THREADS 256
+template <int DKP> constexpr int delta_intra_smem() {
+    return (3 * DELTA_C * (DKP + 4) + DELTA_C * (DELTA_C + 4) + DELTA_C + (DELTA_NSUB + 1) * DKP) * 4;
+}
+
+template <typename T, int DKP>
+__global__ void __launch_bounds__(DELTA_INTRA_THREADS)
+delta_intra_kernel(DeltaArgs a) {
+    constexpr int C = DELTA_C, LD = DKP + 4, LA = C + 4, NT = DELTA_INTRA_THREADS;
+    extern __shared__ __align__(16) float sm[];
+    float* sK = sm;                          // k, then k 2^(edge - L) for the edge reached so far
+    float* sQ = sK + C * LD;                 // q, then q 2^(L - edge of its sub-chunk)
+    float* sL = sQ + C * LD;                 // L, then k 2^(L - edge), then k 2^L
+    float* sA = sL + C * LD;                 // beta_t A_ts
+    float* sB = sA + C * LA;                 // beta
+    float* sR = sB + C;                      // [5][DKP]: L at the edges of the sub-chunks
+    __shared__ int steep;                    // bit J: sub-chunk J decays by more than DELTA_SPREAD in some channel
+    pdl_trigger();
+    const int h = blockIdx.x, seq = blockIdx.y, c = blockIdx.z, tid = threadIdx.x;
+    const int n = min(C, a.q_len[seq] - c * C), r0 = a.q_start[seq] + c * C;
+    if (n <= 0) return;
+    const int dk = a.dk, dv = a.dv, g = h / (a.heads / a.groups);
+    const float rate = a.rate[h];
+    if (tid == 0) steep = 0;
+    pdl_wait();
+    for (int idx = tid; idx < C * DKP; idx += NT) {
+        const int t = idx / DKP, i = idx - t * DKP;
+        const size_t row = (size_t)(r0 + t);
+        const bool in = t < n && i < dk;
+        sK[t * LD + i] = in ? a.k[row * a.k_stride + (size_t)g * dk + i] : 0.f;
+        sQ[t * LD + i] = in ? a.q[row * a.q_stride + (size_t)g * dk + i] : 0.f;
+        sL[t * LD + i] = in ? delta_log_decay(a.z[row * a.z_stride + (size_t)h * dk + i] + a.bias[(size_t)h * dk + i], rate) : 0.f;
+    }
+    if (tid < C) sB[tid] = tid < n ? delta_sigmoid(to_f32(((const T*)a.b)[(size_t)(r0 + tid) * a.b_stride + h])) : 0.f;
+    __syncthreads();
+    for (int i = tid; i < DKP; i += NT) {
+        float L = 0.f;
+        sR[i] = 0.f;
+#pragma unroll 1
+        for (int J = 0; J < DELTA_NSUB; ++J) {
+            const float edge = L;
+#pragma unroll
+            for (int t = 0; t < DELTA_SUB; ++t) {
+                float* p = sL + (J * DELTA_SUB + t) * LD + i;
+                L += *p;
+                *p = L;
+            }
+            sR[(J + 1) * DKP + i] = L;
+            if (edge - L > DELTA_SPREAD) atomicOr(&steep, 1 << J);
+        }
+    }
+    __syncthreads();
+    const int all_steep = steep;
+    const int ty = tid >> 4, tx = tid & 15;
+    const size_t hrow0 = (size_t)r0 * a.heads + h;                 // + t * heads: index of (row, head)
+#pragma unroll 1
+    for (int J = 0; J < DELTA_NSUB; ++J) {
+        const bool direct = (all_steep >> J) & 1;
+        const float *edge = sR + J * DKP, *next = edge + DKP;
+        // this sub-chunk's rows; a steep one's pairs first, while k, q and L are there as they came
+        const int t = J * DELTA_SUB + ty;
+        float accA[DELTA_NSUB], accP[DELTA_NSUB];
+#pragma unroll
+        for (int I = 0; I < DELTA_NSUB; ++I) { accA[I] = 0.f; accP[I] = 0.f; }
+        float dA = 0.f, dP = 0.f;
+        if (direct) {
+            const int s = J * DELTA_SUB + tx;
+            if (tx <= ty)
+                for (int i = 0; i < dk; ++i) {
+                    const float ks = sK[s * LD + i] * exp2f(sL[t * LD + i] - sL[s * LD + i]);
+                    dA = fmaf(sK[t * LD + i], ks, dA);
+                    dP = fmaf(sQ[t * LD + i], ks, dP);
+                }
+            __syncthreads();
+        }
+        for (int idx = tid; idx < (J + 1) * DELTA_SUB * DKP; idx += NT) {
+            const int r = idx / DKP, i = idx - r * DKP;
+            if (r < J * DELTA_SUB) {
+                // an earlier row: on to this sub-chunk's edge (a steep sub-chunk's rows are there already when it is the last)
+                const int Jr = r / DELTA_SUB;
+                if (!(Jr == J - 1 && ((all_steep >> Jr) & 1))) sK[r * LD + i] *= exp2f(edge[i] - (edge - DKP)[i]);
+            } else {
+                const float L = sL[r * LD + i], kk = sK[r * LD + i], d = L - edge[i], e = exp2f(d);
+                sQ[r * LD + i] *= e;
+                sL[r * LD + i] = kk * e;
+                sK[r * LD + i] = kk * (direct ? exp2f(next[i] - L) : exp2f(-d));
+            }
+        }
+        __syncthreads();
+        {
+            const float *ra = sL + t * LD, *rq = sQ + t * LD, *rk = sK + tx * LD;
+            const int last = direct ? J : J + 1;                    // the diagonal block is one of the products unless steep
+#pragma unroll 1
+            for (int i = 0; i < DKP; i += 4) {
+                const float4 ka = *reinterpret_cast<const float4*>(ra + i), qa = *reinterpret_cast<const float4*>(rq + i);
+#pragma unroll
+                for (int I = 0; I < DELTA_NSUB; ++I)
+                    if (I < last) {
+                        const float4 kb = *reinterpret_cast<const float4*>(rk + I * DELTA_SUB * LD + i);
+                        accA[I] = fmaf(ka.x, kb.x, fmaf(ka.y, kb.y, fmaf(ka.z, kb.z, fmaf(ka.w, kb.w, accA[I]))));
+                        accP[I] = fmaf(qa.x, kb.x, fmaf(qa.y, kb.y, fmaf(qa.z, kb.z, fmaf(qa.w, kb.w, accP[I]))));
+                    }
+            }
+            const float beta = sB[t];
+#pragma unroll
+            for (int I = 0; I < DELTA_NSUB; ++I)
+                if (I <= J) {
+                    const int s = I * DELTA_SUB + tx;
+                    const float A = (direct && I == J) ? dA : accA[I], P = (direct && I == J) ? dP : accP[I];
+                    sA[t * LA + s] = s < t ? beta * A : 0.f;
+                    if (t < n) a.p[(hrow0 + (size_t)t * a.heads) * C + s] = s <= t ? P : 0.f;
+                }
+        }
+        __syncthreads();
+        // k 2^L stays for the substitution, q 2^L goes out
+        for (int idx = tid; idx < DELTA_SUB * DKP; idx += NT) {
+            const int r = J * DELTA_SUB + idx / DKP, i = idx % DKP;
+            const float e = exp2f(edge[i]);
+            sL[r * LD + i] *= e;
+            if (r < n && i < a.dk4) a.qd[(hrow0 + (size_t)r * a.heads) * a.dk4 + i] = sQ[r * LD + i] * e;
+        }
+    }
+    __syncthreads();
+    {
+        const float *edge = sR + (DELTA_NSUB - 1) * DKP, *end = edge + DKP;
+        for (int idx = tid; idx < n * DKP; idx += NT) {
+            const int r = idx / DKP, i = idx - r * DKP;
+            const bool there = r / DELTA_SUB == DELTA_NSUB - 1 && ((all_steep >> (DELTA_NSUB - 1)) & 1);
+            if (i < a.dk4) a.kd[(hrow0 + (size_t)r * a.heads) * a.dk4 + i] = sK[r * LD + i] * (there ? 1.f : exp2f(end[i] - edge[i]));
+        }
+        float* gc = a.gc + ((size_t)(seq * a.max_chunks + c) * a.heads + h) * a.dk4;
+        for (int i = tid; i < a.dk4; i += NT) gc[i] = exp2f(end[i]);
+    }
+    // forward substitution: a thread a column, its 64 numbers in registers
+    for (int col = tid; col < a.dk4 + a.dv4; col += NT) {
+        const bool is_w = col < a.dk4;
+        const int vc = col - a.dk4;
+        float x[C];
+#pragma unroll
+        for (int t = 0; t < C; ++t)
+            x[t] = is_w ? sL[t * LD + col] : (t < n && vc < dv) ? a.v[(size_t)(r0 + t) * a.v_stride + (size_t)h * dv + vc] : 0.f;
+#pragma unroll
+        for (int t = 0; t < C; ++t) {
+            float acc = x[t] * sB[t];
+#pragma unroll
+            for (int s = 0; s < t; s += 4) {                       // columns at and beyond t hold zeros
+                const float4 m = *reinterpret_cast<const float4*>(sA + t * LA + s);
+                acc = fmaf(-m.x, x[s], acc);
+                if (s + 1 < t) acc = fmaf(-m.y, x[s + 1], acc);
+                if (s + 2 < t) acc = fmaf(-m.z, x[s + 2], acc);
+                if (s + 3 < t) acc = fmaf(-m.w, x[s + 3], acc);
+            }
+            x[t] = acc;
+        }
+        float* dst = is_w ? a.w + hrow0 * a.dk4 + col : a.u + hrow0 * a.dv4 + vc;
+        const size_t step = (size_t)a.heads * (is_w ? a.dk4 : a.dv4);
+#pragma unroll
+        for (int t = 0; t < C; ++t)
+            if (t < n) dst[t * step] = x[t];
+    }
+}
+
+// ------------------------------------------------------------------ chunk after chunk
+__device__ __forceinline__ void delta_cp16(void* smem, const void* gmem, bool in) {
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"((uint32_t)__cvta_generic_to_shared(smem)), "l"(gmem), "r"(in ? 16 : 0) : "memory");
+}
+__device__ __forceinline__ void delta_cp_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
+template <int N> __device__ __forceinline__ void delta_cp_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
+
+#define DELTA_STATE_THREADS 256
+template <int DKP> constexpr int delta_state_smem() { return (DKP * (DELTA_DVT + 4) + 2 * DELTA_C * (DKP + 4) + DELTA_C * (DELTA_DVT + 4)) * 4; }
+
+template <int DKP>
+__global__ void __launch_bounds__(DELTA_STATE_THREADS)
+delta_state_kernel(DeltaArgs a) {
+    constexpr int C = DELTA_C, LD = DKP + 4, LS = DELTA_DVT + 4, NT = DELTA_STATE_THREADS, RI = DKP / 32;
+    extern __shared__ __align__(16) float sm[];
+    float* sS = sm;                          // [DKP][LS]
+    float* sW = sS + DKP * LS;               // [C][LD]
+    float* sK = sW + C * LD;
+    float* sU = sK + C * LD;                 // [C][LS]
+    pdl_trigger();
+    const int h = blockIdx.x, seq = blockIdx.y, col0 = blockIdx.z * DELTA_DVT, tid = threadIdx.x;
+    const int n_all = a.q_len[seq], r0 = a.q_start[seq];
+    if (n_all <= 0) return;
+    const int dk = a.dk, dv = a.dv, n_chunks = (n_all + C - 1) / C;
+    const int ty = tid >> 3, tx = tid & 7;   // 2 rows of U or RI rows of S, and 4 columns
+    const int j0 = col0 + tx * 4;
+    float* S_area = (float*)(a.state + (size_t)a.slot_ids[seq] * a.state_stride + a.state_offset) + (size_t)h * dk * dv;
+    float s[RI][4];
+#pragma unroll
+    for (int e = 0; e < RI; ++e)
+#pragma unroll
+        for (int x = 0; x < 4; ++x) {
+            const int i = ty * RI + e;
+            s[e][x] = (i < dk && j0 + x < dv) ? S_area[(size_t)i * dv + j0 + x] : 0.f;
+            sS[i * LS + tx * 4 + x] = s[e][x];
+        }
+    for (int idx = tid; idx < 2 * C * LD; idx += NT) sW[idx] = 0.f;      // columns that no copy touches stay zero
+    __syncthreads();
+    pdl_wait();
+    const int ch = a.dk4 / 4;
+    auto load = [&](float* dst, const float* src, int c) {
+        const int n = min(C, n_all - c * C);
+        for (int idx = tid; idx < C * ch; idx += NT) {
+            const int t = idx / ch, i = (idx - t * ch) * 4;
+            const bool in = t < n;
+            delta_cp16(dst + t * LD + i, src + ((size_t)(r0 + c * C + (in ? t : 0)) * a.heads + h) * a.dk4 + i, in);
+        }
+    };
+    float4 u0[2];
+    auto load_u = [&](int c) {
+        const int n = min(C, n_all - c * C);
+#pragma unroll
+        for (int r = 0; r < 2; ++r) {
+            const int t = ty * 2 + r;
+            u0[r] = (t < n && j0 < a.dv4) ? *reinterpret_cast<const float4*>(a.u + ((size_t)(r0 + c * C + t) * a.heads + h) * a.dv4 + j0)
+                                          : make_float4(0.f, 0.f, 0.f, 0.f);
+        }
+    };
+    float gn[RI];
+    auto load_g = [&](int c) {
+        const float* gc = a.gc + ((size_t)(seq * a.max_chunks + c) * a.heads + h) * a.dk4;
+#pragma unroll
+        for (int e = 0; e < RI; ++e) gn[e] = ty * RI + e < a.dk4 ? gc[ty * RI + e] : 0.f;
+    };
+    load(sW, a.w, 0);
+    delta_cp_commit();
+    load(sK, a.kd, 0);
+    delta_cp_commit();
+    load_u(0);
+    load_g(0);
+    for (int c = 0; c < n_chunks; ++c) {
+        const int n = min(C, n_all - c * C);
+        // the state that this chunk starts from, for the output kernel
+        float* sc = a.sc + ((size_t)(seq * a.max_chunks + c) * a.heads + h) * dk * a.dv4;
+#pragma unroll
+        for (int e = 0; e < RI; ++e)
+            if (ty * RI + e < dk && j0 < a.dv4)
+                *reinterpret_cast<float4*>(sc + (size_t)(ty * RI + e) * a.dv4 + j0) = make_float4(s[e][0], s[e][1], s[e][2], s[e][3]);
+        delta_cp_wait<1>();
+        __syncthreads();
+        // U = U0 - W S
+        float u[2][4];
+#pragma unroll
+        for (int r = 0; r < 2; ++r) { u[r][0] = u0[r].x; u[r][1] = u0[r].y; u[r][2] = u0[r].z; u[r][3] = u0[r].w; }
+        if (c + 1 < n_chunks) load_u(c + 1);
+        const float* w0 = sW + (ty * 2) * LD;
+#pragma unroll 4
+        for (int i = 0; i < DKP; i += 4) {
+            float wv[2][4], sv[4][4];
+#pragma unroll
+            for (int r = 0; r < 2; ++r) *reinterpret_cast<float4*>(wv[r]) = *reinterpret_cast<const float4*>(w0 + r * LD + i);
+#pragma unroll
+            for (int e = 0; e < 4; ++e) *reinterpret_cast<float4*>(sv[e]) = *reinterpret_cast<const float4*>(sS + (i + e) * LS + tx * 4);
+#pragma unroll
+            for (int e = 0; e < 4; ++e)
+#pragma unroll
+                for (int r = 0; r < 2; ++r)
+#pragma unroll
+                    for (int x = 0; x < 4; ++x) u[r][x] = fmaf(-wv[r][e], sv[e][x], u[r][x]);
+        }
+#pragma unroll
+        for (int r = 0; r < 2; ++r) {
+            const int t = ty * 2 + r;
+            const float4 uv = make_float4(u[r][0], u[r][1], u[r][2], u[r][3]);
+            *reinterpret_cast<float4*>(sU + t * LS + tx * 4) = uv;
+            if (t < n && j0 < a.dv4) *reinterpret_cast<float4*>(a.u + ((size_t)(r0 + c * C + t) * a.heads + h) * a.dv4 + j0) = uv;
+        }
+        __syncthreads();                                   // W has been read, U is there
+        if (c + 1 < n_chunks) load(sW, a.w, c + 1);
+        delta_cp_commit();
+        delta_cp_wait<1>();                                // this chunk's k
+        __syncthreads();
+        // S = diag(2^L) S + K^T U
+#pragma unroll
+        for (int e = 0; e < RI; ++e)
+#pragma unroll
+            for (int x = 0; x < 4; ++x) s[e][x] *= gn[e];
+        if (c + 1 < n_chunks) load_g(c + 1);
+#pragma unroll 4
+        for (int t = 0; t < C; ++t) {
+            float kv[RI], uv[4];
+            if (RI >= 4) {
+#pragma unroll
+                for (int e = 0; e < RI; e += 4) *reinterpret_cast<float4*>(kv + e) = *reinterpret_cast<const float4*>(sK + t * LD + ty * RI + e);
+            } else {
+#pragma unroll
+                for (int e = 0; e < RI; ++e) kv[e] = sK[t * LD + ty * RI + e];
+            }
+            *reinterpret_cast<float4*>(uv) = *reinterpret_cast<const float4*>(sU + t * LS + tx * 4);
+#pragma unroll
+            for (int e = 0; e < RI; ++e)
+#pragma unroll
+                for (int x = 0; x < 4; ++x) s[e][x] = fmaf(kv[e], uv[x], s[e][x]);
+        }
+#pragma unroll
+        for (int e = 0; e < RI; ++e)
+            *reinterpret_cast<float4*>(sS + (ty * RI + e) * LS + tx * 4) = make_float4(s[e][0], s[e][1], s[e][2], s[e][3]);
+        __syncthreads();                                   // k has been read, the new S is there
+        if (c + 1 < n_chunks) load(sK, a.kd, c + 1);
+        delta_cp_commit();
+    }
+    delta_cp_wait<0>();
+#pragma unroll
+    for (int e = 0; e < RI; ++e)
+#pragma unroll
+        for (int x = 0; x < 4; ++x) {
+            const int i = ty * RI + e;
+            if (i < dk && j0 + x < dv) S_area[(size_t)i * dv + j0 + x] = s[e][x];
+        }
+}
+
+// ------------------------------------------------------------------ outputs of every chunk
+#define DELTA_OUT_THREADS 256
+template <int DKP> constexpr int delta_out_smem() {
+    return (DELTA_C * (DKP + 4) + DKP * (DELTA_OUT_COLS + 4) + DELTA_C * (DELTA_C + 4) + DELTA_C * (DELTA_OUT_COLS + 4)) * 4;
+}
+
+template <int DKP>
+__global__ void __launch_bounds__(DELTA_OUT_THREADS)
+delta_out_kernel(DeltaArgs a) {
+    constexpr int C = DELTA_C, LD = DKP + 4, LS = DELTA_OUT_COLS + 4, LP = C + 4, NT = DELTA_OUT_THREADS;
+    extern __shared__ __align__(16) float sm[];
+    float* sQ = sm;                          // [C][LD]
+    float* sS = sQ + C * LD;                 // [DKP][LS]
+    float* sP = sS + DKP * LS;               // [C][LP]
+    float* sU = sP + C * LP;                 // [C][LS]
+    pdl_trigger();
+    const int tiles = (a.dv4 + DELTA_OUT_COLS - 1) / DELTA_OUT_COLS;
+    const int h = blockIdx.x, seq = blockIdx.y, c = blockIdx.z / tiles, col0 = (blockIdx.z - c * tiles) * DELTA_OUT_COLS, tid = threadIdx.x;
+    const int n = min(C, a.q_len[seq] - c * C), r0 = a.q_start[seq] + c * C;
+    if (n <= 0) return;
+    const int dk = a.dk;
+    const size_t hrow0 = (size_t)r0 * a.heads + h;
+    pdl_wait();
+    for (int idx = tid; idx < C * (DKP / 4); idx += NT) {
+        const int t = idx / (DKP / 4), i = (idx - t * (DKP / 4)) * 4;
+        const bool in = t < n && i < a.dk4;
+        delta_cp16(sQ + t * LD + i, in ? a.qd + (hrow0 + (size_t)t * a.heads) * a.dk4 + i : a.qd, in);
+    }
+    const float* sc = a.sc + ((size_t)(seq * a.max_chunks + c) * a.heads + h) * dk * a.dv4;
+    constexpr int CQ = DELTA_OUT_COLS / 4;
+    for (int idx = tid; idx < DKP * CQ; idx += NT) {
+        const int i = idx / CQ, j = col0 + (idx - i * CQ) * 4;
+        const bool in = i < dk && j < a.dv4;
+        delta_cp16(sS + i * LS + j - col0, in ? sc + (size_t)i * a.dv4 + j : a.sc, in);
+    }
+    for (int idx = tid; idx < C * (C / 4); idx += NT) {
+        const int t = idx / (C / 4), s = (idx - t * (C / 4)) * 4;
+        const bool in = t < n && s / DELTA_SUB <= t / DELTA_SUB;       // the blocks beyond were not written
+        delta_cp16(sP + t * LP + s, in ? a.p + (hrow0 + (size_t)t * a.heads) * C + s : a.p, in);
+    }
+    for (int idx = tid; idx < C * CQ; idx += NT) {
+        const int t = idx / CQ, j = col0 + (idx - t * CQ) * 4;
+        const bool in = t < n && j < a.dv4;
+        delta_cp16(sU + t * LS + j - col0, in ? a.u + (hrow0 + (size_t)t * a.heads) * a.dv4 + j : a.u, in);
+    }
+    delta_cp_commit();
+    delta_cp_wait<0>();
+    __syncthreads();
+    const int ty = tid >> 4, tx = tid & 15;
+    float o[4][4];
+#pragma unroll
+    for (int r = 0; r < 4; ++r)
+#pragma unroll
+        for (int x = 0; x < 4; ++x) o[r][x] = 0.f;
+    auto product = [&](const float* m, int ld, const float* rhs, int kk) {
+#pragma unroll 2
+        for (int i = 0; i < kk; i += 4) {
+            float mv[4][4], sv[4][4];
+#pragma unroll
+            for (int r = 0; r < 4; ++r) *reinterpret_cast<float4*>(mv[r]) = *reinterpret_cast<const float4*>(m + (ty * 4 + r) * ld + i);
+#pragma unroll
+            for (int e = 0; e < 4; ++e) *reinterpret_cast<float4*>(sv[e]) = *reinterpret_cast<const float4*>(rhs + (i + e) * LS + tx * 4);
+#pragma unroll
+            for (int e = 0; e < 4; ++e)
+#pragma unroll
+                for (int r = 0; r < 4; ++r)
+#pragma unroll
+                    for (int x = 0; x < 4; ++x) o[r][x] = fmaf(mv[r][e], sv[e][x], o[r][x]);
+        }
+    };
+    product(sQ, LD, sS, DKP);
+    product(sP, LP, sU, ty * 4 + 4);                       // P is lower triangular
+#pragma unroll
+    for (int r = 0; r < 4; ++r) {
+        const int t = ty * 4 + r;
+        if (t >= n) continue;
+        float* orow = a.out + (size_t)(r0 + t) * a.out_stride + (size_t)h * a.dv;
+#pragma unroll
+        for (int x = 0; x < 4; ++x)
+            if (col0 + tx * 4 + x < a.dv) orow[col0 + tx * 4 + x] = o[r][x];
+    }
+}
+
+// ------------------------------------------------------------------ host side
+static int delta_up4(int n) { return (n + 3) / 4 * 4; }
+
+// Floats of scratch that the chunked form of a step needs: row-wise buffers, then the chunks' decays and states.
+extern "C" long long braid_delta_work_floats(int rows, int n_seqs, int max_q_len, int heads, int dk, int dv) {
+    const long long dk4 = delta_up4(dk), dv4 = delta_up4(dv), chunks = (max_q_len + DELTA_C - 1) / DELTA_C;
+    return (long long)rows * heads * (3 * dk4 + dv4 + DELTA_C) + n_seqs * chunks * heads * (dk4 + dk * dv4);
+}
+
+template <typename T, int DKP>
+static int launch_delta_chunks(const DeltaArgs& a, int n_seqs, cudaStream_t s) {
+    static bool configured = false;
+    if (!configured) {
+        cudaError_t e = cudaFuncSetAttribute(delta_intra_kernel<T, DKP>, cudaFuncAttributeMaxDynamicSharedMemorySize, delta_intra_smem<DKP>());
+        if (e == cudaSuccess) e = cudaFuncSetAttribute(delta_state_kernel<DKP>, cudaFuncAttributeMaxDynamicSharedMemorySize, delta_state_smem<DKP>());
+        if (e == cudaSuccess) e = cudaFuncSetAttribute(delta_out_kernel<DKP>, cudaFuncAttributeMaxDynamicSharedMemorySize, delta_out_smem<DKP>());
+        if (e != cudaSuccess) { braid_set_error("delta_rule: cannot reserve shared memory: %s", cudaGetErrorString(e)); return (int)e; }
+        configured = true;
+    }
+    const int tiles = (a.dv4 + DELTA_OUT_COLS - 1) / DELTA_OUT_COLS;
+    braid_launch(delta_intra_kernel<T, DKP>, dim3(a.heads, n_seqs, a.max_chunks), dim3(DELTA_INTRA_THREADS), delta_intra_smem<DKP>(), s, a);
+    braid_launch(delta_state_kernel<DKP>, dim3(a.heads, n_seqs, (a.dv4 + DELTA_DVT - 1) / DELTA_DVT), dim3(DELTA_STATE_THREADS), delta_state_smem<DKP>(), s, a);
+    braid_launch(delta_out_kernel<DKP>, dim3(a.heads, n_seqs, a.max_chunks * tiles), dim3(DELTA_OUT_THREADS), delta_out_smem<DKP>(), s, a);
+    BRAID_LAUNCH_CHECK();
+}
+
+template <typename T>
+static int launch_delta(const DeltaArgs& a, int n_seqs, bool chunked, cudaStream_t s) {
+    if (chunked) {
+        if (a.dk <= 32) return launch_delta_chunks<T, 32>(a, n_seqs, s);
+        if (a.dk <= 64) return launch_delta_chunks<T, 64>(a, n_seqs, s);
+        if (a.dk <= 128) return launch_delta_chunks<T, 128>(a, n_seqs, s);
+        return launch_delta_chunks<T, 256>(a, n_seqs, s);
+    }
+    const int rg = a.dk <= 32 ? 4 : a.dk <= 64 ? 8 : 16;
+    const int dvt = (DELTA_WALK_THREADS / rg) * DELTA_CV;
+    const dim3 grid(a.heads, n_seqs, (a.dv + dvt - 1) / dvt), block(DELTA_WALK_THREADS);
+    if (rg == 4) braid_launch(delta_walk_kernel<T, 4, 8>, grid, block, 0, s, a);
+    else if (rg == 8) braid_launch(delta_walk_kernel<T, 8, 8>, grid, block, 0, s, a);
+    else if (a.dk <= 128) braid_launch(delta_walk_kernel<T, 16, 8>, grid, block, 0, s, a);
+    else braid_launch(delta_walk_kernel<T, 16, 16>, grid, block, 0, s, a);
+    BRAID_LAUNCH_CHECK();
+}
+
+// `work`: braid_delta_work_floats floats, on 16 bytes, for the chunked form; null: token by token.
+extern "C" int braid_delta_rule(const float* q, long long q_stride, const float* k, long long k_stride, const float* v,
+                                long long v_stride, const float* z, long long z_stride, const float* bias, const float* rate,
+                                const void* b, long long b_stride, int dtype, float* out, long long out_stride, void* state,
+                                long long state_stride, long long state_offset, const int* q_start, const int* q_len,
+                                const int* slot_ids, int rows, int n_seqs, int max_q_len, int heads, int groups, int dk, int dv,
+                                float* work, long long work_floats, void* stream) {
+    if (n_seqs <= 0 || rows <= 0 || max_q_len <= 0) return BRAID_OK;
+    if (heads <= 0 || groups <= 0 || heads % groups) BRAID_REFUSE("delta_rule: %d heads do not divide into %d groups", heads, groups);
+    if (dk <= 0 || dk > DELTA_MAX_DK || dv <= 0) BRAID_REFUSE("delta_rule: key size %d must be in (0, %d], value size %d positive", dk, DELTA_MAX_DK, dv);
+    if (!state || (state_offset & 3) || (state_stride & 3)) BRAID_REFUSE("delta_rule: the state area must be given, in multiples of 4 bytes");
+    if (dtype != BRAID_F32 && dtype != BRAID_BF16) BRAID_REFUSE("delta_rule: unknown dtype code %d", dtype);
+    DeltaArgs a{q, q_stride, k, k_stride, v, v_stride, z, z_stride, bias, rate, b, b_stride, out, out_stride, (uint8_t*)state,
+                state_stride, state_offset, q_start, q_len, slot_ids, heads, groups, dk, dv,
+                nullptr, nullptr, nullptr, nullptr, nullptr, nullptr, nullptr, delta_up4(dk), delta_up4(dv),
+                (max_q_len + DELTA_C - 1) / DELTA_C};
+    const long long tiles = (a.dv4 + DELTA_OUT_COLS - 1) / DELTA_OUT_COLS;
+    if (n_seqs > 65535 || (dv + 31) / 32 > 65535 || (work && a.max_chunks * tiles > 65535)) BRAID_REFUSE("delta_rule: the step exceeds the grid limits");
+    if (work) {
+        const long long need = braid_delta_work_floats(rows, n_seqs, max_q_len, heads, dk, dv);
+        if (need > work_floats || ((uintptr_t)work & 15)) BRAID_REFUSE("delta_rule: the chunked form needs %lld floats of scratch on 16 bytes, it was given %lld", need, work_floats);
+        const long long rh = (long long)rows * heads;
+        a.w = work;
+        a.u = a.w + rh * a.dk4;
+        a.qd = a.u + rh * a.dv4;
+        a.kd = a.qd + rh * a.dk4;
+        a.p = a.kd + rh * a.dk4;
+        a.gc = a.p + rh * DELTA_C;
+        a.sc = a.gc + (long long)n_seqs * a.max_chunks * heads * a.dk4;
+    }
+    if (dtype == BRAID_F32) return launch_delta<float>(a, n_seqs, work != nullptr, (cudaStream_t)stream);
+    return launch_delta<__nv_bfloat16>(a, n_seqs, work != nullptr, (cudaStream_t)stream);
+}
+
+// The read-out's norm and gate (gated_norm.cuh), the gate's logits in float32.
+extern "C" int braid_delta_gated_norm(const float* y, const float* gate, long long gate_stride, const void* w, int w_len, void* out,
+                                      long long out_stride, const int* token_seq, int dtype, int rows, int width, int group,
+                                      float eps, void* stream) {
+    cudaStream_t s = (cudaStream_t)stream;
+    if (dtype == BRAID_F32)
+        return gated_norm_launch(y, gate, gate_stride, (const float*)w, w_len, (float*)out, out_stride, token_seq, rows, width, group, 0, 1, eps, 1.f, s);
+    if (dtype == BRAID_BF16)
+        return gated_norm_launch(y, gate, gate_stride, (const __nv_bfloat16*)w, w_len, (__nv_bfloat16*)out, out_stride, token_seq, rows, width, group, 0, 1, eps, 1.f, s);
+    BRAID_REFUSE("gated_norm: unknown dtype code %d", dtype);
+}

@@ -1082,36 +1082,48 @@ extern "C" int braid_proj_prep_kv(const void* src, long long row_stride, int dty
 
 // ------------------------------------------------------------------ a gate a head on attention's result
 // out[r, h * dv + c] = x[r, h * hd + c] * sigmoid(gate[r, h]) for c < dv: the first dv numbers of every padded head,
-// times the head's gate (gate: a column block of the stacked projection, row stride gate_stride; null: no gate).
-template <typename T>
-__global__ void head_gate_kernel(const T* __restrict__ x, long long x_stride, const T* __restrict__ gate, long long gate_stride,
-                                 T* __restrict__ out, long long total, int heads, int hd, int dv) {
+// times the head's gate (gate: a column block of the stacked projection, row stride gate_stride; null: no gate), or, with
+// per_column, times a gate of the column's own, sigmoid(gate[r, h * dv + c]).  V neighbouring columns a thread.
+template <typename T, int V>
+__global__ void __launch_bounds__(256)
+head_gate_kernel(const T* __restrict__ x, long long x_stride, const T* __restrict__ gate, long long gate_stride,
+                 T* __restrict__ out, long long total, int heads, int hd, int dv, int per_column) {
     pdl_trigger();
     pdl_wait();
-    const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
+    const long long i = ((long long)blockIdx.x * blockDim.x + threadIdx.x) * V;
     if (i >= total) return;
     const int per_row = heads * dv;
     const long long r = i / per_row;
     const int rem = (int)(i - r * per_row), h = rem / dv, c = rem - h * dv;
-    float v = to_f32(x[r * x_stride + (size_t)h * hd + c]);
-    if (gate) v *= 1.f / (1.f + expf(-to_f32(gate[r * gate_stride + h])));
-    out[i] = from_f32<T>(v);
+    float v[V], g[V];
+    load_run<T, V>(x + r * x_stride + (size_t)h * hd + c, v);
+    if (gate) {
+        if (per_column) load_run<T, V>(gate + r * gate_stride + rem, g);
+        const float gh = per_column ? 0.f : to_f32(gate[r * gate_stride + h]);
+#pragma unroll
+        for (int e = 0; e < V; ++e) v[e] *= 1.f / (1.f + expf(-(per_column ? g[e] : gh)));
+    }
+    store_run<T, V>(out + i, v);
 }
 
 extern "C" int braid_head_gate(const void* x, long long x_stride, const void* gate, long long gate_stride, void* out,
-                               int dtype, int rows, int heads, int hd, int dv, void* stream) {
+                               int dtype, int rows, int heads, int hd, int dv, int per_column, void* stream) {
     if (rows <= 0) return BRAID_OK;
     if (heads <= 0 || dv <= 0 || hd < dv) BRAID_REFUSE("head_gate: %d heads of %d numbers in heads of %d", heads, dv, hd);
-    const long long total = (long long)rows * heads * dv, blocks = (total + 255) / 256;
+    if (dtype != BRAID_F32 && dtype != BRAID_BF16) BRAID_REFUSE("head_gate: unknown dtype code %d", dtype);
+    const int vec = dtype == BRAID_F32 ? 4 : 8;
+    const bool wide = dv % vec == 0 && hd % vec == 0 && x_stride % vec == 0 && (((uintptr_t)x | (uintptr_t)out) & 15) == 0 &&
+                      (!gate || !per_column || (gate_stride % vec == 0 && ((uintptr_t)gate & 15) == 0));
+    const long long total = (long long)rows * heads * dv, runs = total / (wide ? vec : 1), blocks = (runs + 255) / 256;
     if (blocks > 0x7fffffffLL) BRAID_REFUSE("head_gate: %lld elements exceed one launch", total);
     cudaStream_t s = (cudaStream_t)stream;
-    if (dtype == BRAID_F32)
-        braid_launch(head_gate_kernel<float>, dim3((int)blocks), dim3(256), 0, s, (const float*)x, x_stride, (const float*)gate,
-                     gate_stride, (float*)out, total, heads, hd, dv);
-    else if (dtype == BRAID_BF16)
-        braid_launch(head_gate_kernel<__nv_bfloat16>, dim3((int)blocks), dim3(256), 0, s, (const __nv_bfloat16*)x, x_stride,
-                     (const __nv_bfloat16*)gate, gate_stride, (__nv_bfloat16*)out, total, heads, hd, dv);
-    else BRAID_REFUSE("head_gate: unknown dtype code %d", dtype);
+#define HG_LAUNCH(T, V) braid_launch(head_gate_kernel<T, V>, dim3((int)blocks), dim3(256), 0, s, (const T*)x, x_stride,  \
+                                     (const T*)gate, gate_stride, (T*)out, total, heads, hd, dv, per_column)
+    if (dtype == BRAID_F32 && wide) HG_LAUNCH(float, 4);
+    else if (dtype == BRAID_F32) HG_LAUNCH(float, 1);
+    else if (wide) HG_LAUNCH(__nv_bfloat16, 8);
+    else HG_LAUNCH(__nv_bfloat16, 1);
+#undef HG_LAUNCH
     BRAID_LAUNCH_CHECK();
 }
 

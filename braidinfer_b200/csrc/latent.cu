@@ -32,6 +32,10 @@ struct LatentPrepArgs {
     float eps;
     int* error_flag;
     int adjacent;             // pairs are (2p, 2p + 1) instead of (p, p + rot_dims/2)
+    void* dq_out;             // [rows, dq_ld]: the RMS norm of the row's first q_rank numbers (low-rank queries), zeros up to
+    long long dq_ld;          // dq_ld; or null.  The row then holds no queries (heads = 0)
+    const void* dq_w;         // [q_rank]
+    int q_rank;
 };
 
 template <typename T>
@@ -68,6 +72,20 @@ latent_prep_kernel(LatentPrepArgs a) {
         ss = block_sum(ss, red);
     }
     const float scale = 1.f / sqrtf(ss / (float)a.rank + a.eps);
+    if (a.dq_out) {
+        float sq = 0.f;
+        for (int i = threadIdx.x; i < a.q_rank; i += blockDim.x) {
+            const float v = to_f32(src[i]);
+            sq = fmaf(v, v, sq);
+        }
+        __syncthreads();                                   // the sum before has been read
+        sq = block_sum(sq, red);
+        const float qs = 1.f / sqrtf(sq / (float)a.q_rank + a.eps);
+        T* o = (T*)a.dq_out + (size_t)row * a.dq_ld;
+        const T* w = (const T*)a.dq_w;
+        for (int i = threadIdx.x; i < a.dq_ld; i += blockDim.x)
+            o[i] = i < a.q_rank ? from_f32<T>(to_f32(src[i]) * qs * to_f32(w[i])) : from_f32<T>(0.f);
+    }
     if (dst) {
         const T* w = (const T*)a.norm_w;
         for (int i = threadIdx.x; i < a.rank; i += blockDim.x) dst[i] = from_f32<T>(to_f32(cin[i]) * scale * to_f32(w[i]));
@@ -98,14 +116,17 @@ latent_prep_kernel(LatentPrepArgs a) {
 extern "C" int braid_latent_prep(const void* proj, long long ld, int q_cols, const void* norm_w, const float* inv_freq,
                                  const int* positions, const int* token_seq, const int* page_table, void* cache,
                                  void* q_lat, int dtype, int rows, int heads, int dim, int rot, int rank, int rot_dims,
-                                 int page_size, int table_cols, int num_pages, float eps, int adjacent, int* error_flag, void* stream) {
+                                 int page_size, int table_cols, int num_pages, float eps, int adjacent, void* dq_out,
+                                 long long dq_ld, const void* dq_w, int q_rank, int* error_flag, void* stream) {
     if (rows <= 0) return BRAID_OK;
-    if (heads <= 0 || dim < 0 || rot < 0 || rank <= 0) BRAID_REFUSE("latent_prep: heads=%d dim=%d rot=%d rank=%d", heads, dim, rot, rank);
+    if (dq_out && (heads != 0 || q_rank <= 0 || q_rank > dq_ld || q_rank > q_cols || !dq_w))
+        BRAID_REFUSE("latent_prep: the low-rank part of %d numbers lies before column %d, in rows without queries, and fits %lld", q_rank, q_cols, dq_ld);
+    if ((heads <= 0 && !dq_out) || dim < 0 || rot < 0 || rank <= 0) BRAID_REFUSE("latent_prep: heads=%d dim=%d rot=%d rank=%d", heads, dim, rot, rank);
     if (rot_dims < 0 || rot_dims > rot || rot_dims % 2) BRAID_REFUSE("latent_prep: %d rotated dimensions must be even and within %d", rot_dims, rot);
     if (!error_flag) BRAID_REFUSE("latent_prep: error_flag is required");
     if (cache && (!page_table || table_cols <= 0 || num_pages <= 0 || page_size <= 0)) BRAID_REFUSE("latent_prep: the cache has no pages");
     LatentPrepArgs a{proj, ld, q_cols, norm_w, inv_freq, positions, token_seq, page_table, cache, q_lat,
-                     rows, heads, dim, rot, rank, rot_dims, page_size, table_cols, num_pages, eps, error_flag, adjacent};
+                     rows, heads, dim, rot, rank, rot_dims, page_size, table_cols, num_pages, eps, error_flag, adjacent, dq_out, dq_ld, dq_w, q_rank};
     cudaStream_t s = (cudaStream_t)stream;
     if (dtype == BRAID_F32) braid_launch(latent_prep_kernel<float>, dim3(rows), dim3(128), 0, s, a);
     else if (dtype == BRAID_BF16) braid_launch(latent_prep_kernel<__nv_bfloat16>, dim3(rows), dim3(128), 0, s, a);
@@ -288,6 +309,7 @@ struct AttnLatentArgs {
     int rows, heads, D, rank, page_size, table_cols, num_pages, window;
     float scale;
     int* error_flag;
+    const float* sinks;       // [heads] float32: a score a head that joins the denominator and has no value; or null
 };
 
 #define ATTN_LATENT_WARPS 4
@@ -357,7 +379,13 @@ attn_latent_simple_kernel(AttnLatentArgs a) {
         }
         __syncwarp();
     }
-    const float inv = 1.f / l;
+    float corr_end = 1.f;
+    if (a.sinks) {                                       // the sink joins as one more score, with no value
+        const float sink = a.sinks[head], m_new = fmaxf(m, sink);
+        corr_end = expf(m - m_new);
+        l = l * corr_end + expf(sink - m_new);
+    }
+    const float inv = corr_end / l;
 #pragma unroll
     for (int i = 0; i < NACC; ++i) {
         const int d = lane + 32 * i;
@@ -378,14 +406,15 @@ static cudaError_t launch_attn_latent_simple(const AttnLatentArgs& a, int blocks
 extern "C" int braid_attn_latent_simple(const void* q, void* out, int dtype, const void* cache, const int* page_table,
                                         const int* positions, const int* token_seq, long long ldq, long long ldo,
                                         int rows, int heads, int D, int rank, int page_size, int table_cols,
-                                        int num_pages, int window, float scale, int* error_flag, void* stream) {
+                                        int num_pages, int window, float scale, const float* sinks, int* error_flag,
+                                        void* stream) {
     if (rows <= 0) return BRAID_OK;
     if (!error_flag) BRAID_REFUSE("attn_latent_simple: error_flag is required");
     if (num_pages <= 0 || table_cols <= 0 || page_size <= 0) BRAID_REFUSE("attn_latent_simple: the cache has no pages");
     if (heads <= 0 || rank <= 0 || rank > D) BRAID_REFUSE("attn_latent_simple: heads=%d rank=%d D=%d", heads, rank, D);
     if (rank > 1024 || D > 2048) BRAID_REFUSE("attn_latent_simple: rank=%d (at most 1024), row size=%d (at most 2048)", rank, D);
     AttnLatentArgs a{q, out, cache, page_table, positions, token_seq, ldq, ldo, rows, heads, D, rank, page_size,
-                     table_cols, num_pages, window, scale, error_flag};
+                     table_cols, num_pages, window, scale, error_flag, sinks};
     const long long items = (long long)rows * heads;
     const long long blocks = (items + ATTN_LATENT_WARPS - 1) / ATTN_LATENT_WARPS;
     if (blocks > 0x7fffffffLL) BRAID_REFUSE("attn_latent_simple: %lld (token, head) pairs exceed one launch", items);

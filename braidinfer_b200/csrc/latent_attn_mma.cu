@@ -9,7 +9,7 @@
 // 32 at a time (half a page) through two cp.async stages; scores S = Q K^T with Q fragments read from shared
 // memory, the online softmax in registers, P reused as the A operand of O += P V with V fragments taken from
 // the same key tile by transposing loads.  With slices, unnormalised O and (max, sum) go to a workspace and a
-// second kernel merges them.  Key j is visible to position p iff j <= p and (no window or p - j < window).
+// second kernel merges them.  A sink a head (optional) joins the denominator where a row is finished.  Key j is visible to position p iff j <= p and (no window or p - j < window).
 #include "common.cuh"
 #include "mma_tile.cuh"
 #include "page.h"
@@ -41,7 +41,16 @@ struct LatAttnArgs {
     int heads, table_cols, num_pages, window, n_splits, total_pairs;
     float scale_log2;              // scale * log2(e)
     int* error_flag;
+    const float* sinks;            // [heads] float32: a score a head that joins the denominator and has no value; or null
 };
+
+// The denominator of a finished row with its head's sink in it (m, l in units of log2), as the factor on the accumulators.
+__device__ __forceinline__ float lat_finish(float m, float l, const float* sinks, long long pair, int heads) {
+    if (!sinks) return 1.f / l;
+    const float sk = sinks[pair % heads] * 1.4426950408889634f, mn = fmaxf(m, sk);
+    const float c = exp2f(m - mn);
+    return c / (l * c + exp2f(sk - mn));
+}
 
 __global__ void __launch_bounds__(128)
 latent_attn_mma_kernel(LatAttnArgs a) {
@@ -212,7 +221,7 @@ latent_attn_mma_kernel(LatAttnArgs a) {
         if (!live_row[h2]) continue;
         const long long pair = base_pair + warp * 16 + g + h2 * 8;
         if (a.partial == nullptr) {
-            const float inv = 1.f / l_run[h2];
+            const float inv = lat_finish(m_run[h2], l_run[h2], a.sinks, pair, a.heads);
             __nv_bfloat16* o = a.out + pair * R + vc0;
 #pragma unroll
             for (int i = 0; i < VC / 8; ++i)
@@ -408,7 +417,7 @@ latent_attn_few_kernel(LatAttnArgs a) {
         if (!live_row[h2]) continue;
         const long long pair = base_pair + g + h2 * 8;
         if (a.partial == nullptr) {
-            const float inv = 1.f / l_run[h2];
+            const float inv = lat_finish(m_run[h2], l_run[h2], a.sinks, pair, a.heads);
             __nv_bfloat16* o = a.out + pair * R + warp * VQ;
 #pragma unroll
             for (int i = 0; i < VQ / 8; ++i)
@@ -432,7 +441,7 @@ latent_attn_few_kernel(LatAttnArgs a) {
 #define LAT_MERGE_MAX_SPLITS 64
 __global__ void __launch_bounds__(128)
 latent_attn_merge_kernel(const float* __restrict__ partial, __nv_bfloat16* __restrict__ out, const int* __restrict__ token_seq,
-                         int heads, int total_pairs, int n_splits) {
+                         int heads, int total_pairs, int n_splits, const float* __restrict__ sinks) {
     pdl_trigger();
     pdl_wait();
     __shared__ float wgt[LAT_MERGE_MAX_SPLITS];
@@ -458,7 +467,7 @@ latent_attn_merge_kernel(const float* __restrict__ partial, __nv_bfloat16* __res
             d += w * l[i];
         }
         d = warp_sum(d);
-        if (threadIdx.x == 0) inv_s = d > 0.f ? 1.f / d : 0.f;
+        if (threadIdx.x == 0) inv_s = d > 0.f ? lat_finish(M, d, sinks, pair, heads) : 0.f;   // the sink: once, not once a slice
     }
     __syncthreads();
     const float inv = inv_s;
@@ -498,7 +507,7 @@ extern "C" int braid_latent_attn_mma(const void* q, void* out, float* partial, c
                                      const int* q_start, const int* q_len, const int* kv_before, const int* token_seq,
                                      int rows, int n_seqs,
                                      int max_q_len, int heads, int table_cols, int num_pages, int window, int n_splits,
-                                     float scale, int* error_flag, void* stream) {
+                                     float scale, const float* sinks, int* error_flag, void* stream) {
     if (rows <= 0 || n_seqs <= 0 || max_q_len <= 0) return BRAID_OK;
     if (!error_flag) BRAID_REFUSE("latent_attn_mma: error_flag is required");
     if (heads <= 0 || table_cols <= 0 || num_pages <= 0) BRAID_REFUSE("latent_attn_mma: heads=%d, table columns=%d, pages=%d", heads, table_cols, num_pages);
@@ -518,13 +527,13 @@ extern "C" int braid_latent_attn_mma(const void* q, void* out, float* partial, c
     }
     LatAttnArgs a{(const __nv_bfloat16*)q, (__nv_bfloat16*)out, n_splits > 1 ? partial : nullptr, (const __nv_bfloat16*)cache,
                   page_table, q_start, q_len, kv_before, heads, table_cols, num_pages, window, n_splits, rows * heads,
-                  scale * 1.4426950408889634f, error_flag};
+                  scale * 1.4426950408889634f, error_flag, sinks};
     cudaStream_t s = (cudaStream_t)stream;
     cudaError_t e = few
         ? braid_launch(latent_attn_few_kernel, dim3((unsigned)tiles, n_seqs, n_splits), dim3(128), (size_t)SMEM_FEW, s, a)
         : braid_launch(latent_attn_mma_kernel, dim3((unsigned)tiles, n_seqs, n_splits * VPARTS), dim3(128), (size_t)SMEM_BYTES, s, a);
     if (e == cudaSuccess && n_splits > 1)
         braid_launch(latent_attn_merge_kernel, dim3(rows * heads), dim3(128), 0, s, (const float*)partial, (__nv_bfloat16*)out,
-                     token_seq, heads, rows * heads, n_splits);
+                     token_seq, heads, rows * heads, n_splits, sinks);
     BRAID_LAUNCH_CHECK();
 }

@@ -4,5 +4,5 @@ from .base import (BLOCKS, CONNECTIONS, EMBEDDINGS, FEED_FORWARDS, HEADS, INJECT
                    Norm, Part, PositionEncoding, Registry, Streams)
 from .spec import CacheRequest, LayerSpec, ModelSpec, PartSpec, ScheduleEntry, TensorSpec
 from .runtime import Runtime
-from . import (attention, block, embedding, feedforward, hyper, injection, latent_attention, linear_attention,  # noqa: F401
-               mlstm, moe, norm, parallel, rope, ssm, token_input)                                       # (registration)
+from . import (attention, block, delta, embedding, feedforward, hyper, injection, latent_attention,  # noqa: F401
+               linear_attention, mlstm, moe, norm, parallel, rope, ssm, token_input)                                       # (registration)

@@ -37,6 +37,17 @@ Options that other designs use, each off unless named:
     distance_bias   {"slope", "rate"} (tensor names, num_heads numbers each, r1 and r2): r1 ln(1 + r2 (p - j)) comes off the
                     scaled score of key j at position p, float32 (the logarithmic kernel of Chi, Fan, Ramadge, Rudnicky:
                     "KERPLE: Kernelized Relative Positional Embedding for Length Extrapolation", 2022)
+    softcap         scores are capped: cap * tanh(score / cap), after the scale (float32)
+    column_gate     a gate a column on the result: the concatenated heads are multiplied by sigmoid(Wg x), Wg a stored
+                    [num_heads * value_dim, hidden] tensor whose rows ride in the stacked product
+    conv            a number of taps: every channel of q, k and v passes a causal convolution over time (weights stored under
+                    the projection's name with ".conv" added, [channels, taps], the last tap meets the current token; no bias
+                    of its own), after the projection and its bias, before norm and rotation.  The last taps - 1 projected
+                    rows of a sequence are its state (float32).  One kernel convolves, norms, rotates, pads to one head size
+                    and stores keys and values (csrc/conv_heads.cu)
+    shared_kv       the layer makes no keys and values: it reads those that an earlier layer cached (the schedule's
+                    `cache_of`), with its own queries, window and output; goes with `conv`
+    cache_window    how far back the cache keeps keys where readers see further than this layer's own window
 unit_qk_eps, q_temp, qkv_bias, proj_norm, unit_v_eps and value_dim without rotation are for heads that are not rotated (position encoding "none"): one kernel norms, scales and
 stores.  Keys, values and queries are then padded with zeros to one head size that the attention kernels take
 (max(head_dim, value_dim), rounded up to 16), which changes no score and no result.  Rotated heads whose value
@@ -61,7 +72,8 @@ class GQAAttention(Mixer):
     position_encoding (PartSpec), and tensor names q_proj, k_proj, v_proj, o_proj; optional qk_norm
     ({"eps", "q_name", "k_name"}), value_from_key (bool), scale, sink (a score), out_mult, sink_name, head_gate,
     unit_qk_eps, q_temp ({"coef", "every"}), value_dim, keep_first, head_scale (a tensor name), talk (a tensor name), qkv_bias,
-    proj_norm ({"eps", "q_name", "k_name"}), unit_v_eps, distance_bias ({"slope", "rate"})."""
+    proj_norm ({"eps", "q_name", "k_name"}), unit_v_eps, distance_bias ({"slope", "rate"}), softcap, column_gate (a tensor name),
+    conv (taps), shared_kv (bool), cache_window."""
 
     plain_output = True
 
@@ -90,29 +102,43 @@ class GQAAttention(Mixer):
         self.proj_norm = (float(pn["eps"]), prefix + pn["q_name"], prefix + pn["k_name"]) if pn else None
         self.unit_v_eps = float(p["unit_v_eps"]) if p.get("unit_v_eps") is not None else None
         # what the kernel that works on whole projections does (biases, norms over all heads, values of unit size)
-        self.whole_proj = bool(p.get("qkv_bias")) or self.proj_norm is not None or self.unit_v_eps is not None
+        self.taps = int(p.get("conv") or 0)
+        self.shared_kv = bool(p.get("shared_kv", False))
+        self.softcap = float(p["softcap"]) if p.get("softcap") is not None else None
+        if self.softcap is not None and not self.softcap > 0:
+            raise ValueError(f"gqa_attention: softcap must be positive, got {self.softcap}")
+        self.cache_window = p.get("cache_window") or self.window
+        if (self.cache_window is None) != (self.window is None) or (self.window and self.cache_window < self.window):
+            raise ValueError("gqa_attention: the cache must keep at least the layer's own window")
+        self.whole_proj = not self.taps and (bool(p.get("qkv_bias")) or self.proj_norm is not None or self.unit_v_eps is not None)
         if self.whole_proj and (self.unit_qk_eps is not None or self.q_temp):
             raise ValueError("gqa_attention: biases, norms of whole projections and unit values do not go with unit heads or a "
                              "query temperature")
         if self.proj_norm and self.unit_v_eps is not None and self.proj_norm[0] != self.unit_v_eps:
             raise ValueError("gqa_attention: the norms of whole projections and of values have one eps")
-        self.prep = (self.whole_proj or self.unit_qk_eps is not None or self.q_temp is not None or (self.vd != self.hd and pe.kind == "none")
-                     or (gated and pe.kind == "none"))
+        if self.taps and (gated or self.unit_qk_eps is not None or self.q_temp or self.proj_norm or self.unit_v_eps is not None
+                          or self.value_from_key or p.get("keep_first") or p.get("talk") is not None):
+            raise ValueError("gqa_attention: a convolution goes with projections (biased or not), weighted head norms, rotation, a "
+                             "value size of its own, a cap, a gate a column and shared keys and values")
+        if not self.taps and (self.shared_kv or p.get("column_gate") is not None):
+            raise ValueError("gqa_attention: keys and values of another layer and a gate a column go with a convolution")
+        self.prep = not self.taps and (self.whole_proj or self.unit_qk_eps is not None or self.q_temp is not None
+                                       or (self.vd != self.hd and pe.kind == "none") or (gated and pe.kind == "none"))
         if gated and not self.prep and not (p.get("qk_norm") is not None or self.value_from_key):
             raise ValueError("gqa_attention: a gate a head rides in the stacked product, which the plain rotation kernels "
                              "take without further columns; it goes with head norms or with heads that are not rotated")
-        self.hd_pad = -(-max(self.hd, self.vd) // 16) * 16 if self.prep else self.hd
+        self.hd_pad = -(-max(self.hd, self.vd) // 16) * 16 if self.prep or self.taps else self.hd
         self.keep_first = int(p.get("keep_first") or 0)
         self.head_scale_name = prefix + p["head_scale"] if p.get("head_scale") is not None else None
         self.talk_name = prefix + p["talk"] if p.get("talk") is not None else None
         self.head_scale = self.talk = None
         # rotated heads with a value size of their own, or of a size the tensor-core kernels do not take: rows of zeros in
         # the stacked projection pad every head to one size
-        self.pad_rows = (not self.prep and pe.kind != "none" and not self.value_from_key and p.get("qk_norm") is None
+        self.pad_rows = (not self.prep and not self.taps and pe.kind != "none" and not self.value_from_key and p.get("qk_norm") is None
                          and (self.vd != self.hd or (self.hd % 16 and (self.talk_name or self.keep_first))))
         if self.pad_rows:
             self.hd_pad = -(-max(self.hd, self.vd) // 16) * 16
-        if self.vd != self.hd and not (self.prep or self.pad_rows):
+        if self.vd != self.hd and not (self.prep or self.pad_rows or self.taps):
             raise ValueError("gqa_attention: a value size of its own goes with plainly rotated heads or with heads without rotation")
         if self.keep_first and not self.window:
             raise ValueError("gqa_attention: keep_first goes with a window")
@@ -131,14 +157,22 @@ class GQAAttention(Mixer):
         if not self.value_from_key:
             names.append(prefix + p.get("v_proj", "self_attn.v_proj.weight"))
             outs.append(self.nkh * self.vd)
+        if self.shared_kv:
+            names, outs = names[:1], outs[:1]
+        self.channels = sum(outs)            # what a convolution works on
+        self.conv_names = [n + ".conv" for n in names] if self.taps else None
+        self.bias_names = [n + ".b" for n in names] if p.get("qkv_bias") else None
+        self.bias_sizes = list(outs)
+        self.column_gate = p.get("column_gate") is not None
+        if self.column_gate:
+            names.append(prefix + p["column_gate"])
+            outs.append(self.nqh * self.vd)
         self.gate_col = None
         if p.get("head_gate") is not None:
             self.gate_col = sum(outs)
             names.append(prefix + p["head_gate"])
             outs.append(self.nqh)
         self.qkv = Linear(runtime, names, outs, self.hidden)
-        self.bias_names = [n + ".b" for n in names[:3]] if p.get("qkv_bias") else None
-        self.bias_sizes = outs[:3]
         db = p.get("distance_bias")
         self.distance_bias_names = (prefix + db["slope"], prefix + db["rate"]) if db else None
         self.biases = self.distance_bias = self.proj_norm_w = None
@@ -154,6 +188,7 @@ class GQAAttention(Mixer):
         if qn is not None:
             self.qk_norm = (float(qn["eps"]), prefix + qn["q_name"], prefix + qn["k_name"])
         self.q_norm_w = self.k_norm_w = None
+        self.conv_w = self.conv_b = None
         if (self.qk_norm or self.value_from_key) and not hasattr(self.pe, "norm_encode_and_store"):
             raise ValueError(f"position encoding '{pe.kind}' cannot norm heads or store a key as the value")
 
@@ -163,7 +198,10 @@ class GQAAttention(Mixer):
         d.update(self.pe.tensor_specs())
         if self.qk_norm:
             d[self.qk_norm[1]] = TensorSpec((self.hd,), init="one_plus_normal")
-            d[self.qk_norm[2]] = TensorSpec((self.hd,), init="one_plus_normal")
+            if not self.shared_kv:
+                d[self.qk_norm[2]] = TensorSpec((self.hd,), init="one_plus_normal")
+        if self.conv_names:
+            d.update({n: TensorSpec((size, self.taps), std=0.3) for n, size in zip(self.conv_names, self.bias_sizes)})
         if self.sink_name:
             d[self.sink_name] = TensorSpec((self.nqh,), std=1.0)
         if self.head_scale_name:
@@ -184,7 +222,7 @@ class GQAAttention(Mixer):
         self.qkv.load(tensors)
         w = self.qkv.weight
         pad = -w.shape[0] % 8            # rows of zeros, so that a row of the stacked result starts on 16 bytes
-        if pad and (self.qk_norm or self.value_from_key):     # (the plain rotation kernels take rows without padding)
+        if pad and (self.qk_norm or self.value_from_key or self.taps):     # (the plain rotation kernels take rows without padding)
             self.qkv.weight = torch.cat([w, torch.zeros((pad, w.shape[1]), dtype=w.dtype, device=w.device)]).contiguous()
         if self.pad_rows:
             # every head of q, k and v padded with rows of zeros to hd_pad: no score and no result changes
@@ -203,8 +241,12 @@ class GQAAttention(Mixer):
         if self.talk_name:
             self.talk = tensors[self.talk_name].contiguous()
         if self.qk_norm:
-            self.q_norm_w, self.k_norm_w = tensors[self.qk_norm[1]], tensors[self.qk_norm[2]]
-        if self.bias_names:
+            self.q_norm_w = tensors[self.qk_norm[1]]
+            self.k_norm_w = tensors[self.qk_norm[2]] if not self.shared_kv else None
+        if self.taps:
+            self.conv_w = torch.cat([tensors[n] for n in self.conv_names]).contiguous()
+            self.conv_b = torch.cat([tensors[n] for n in self.bias_names]).contiguous() if self.bias_names else None
+        elif self.bias_names:
             self.biases = tuple(tensors[n] for n in self.bias_names)
         if self.proj_norm:
             self.proj_norm_w = (tensors[self.proj_norm[1]], tensors[self.proj_norm[2]])
@@ -215,7 +257,10 @@ class GQAAttention(Mixer):
 
     def cache_request(self) -> Optional[CacheRequest]:
         kind = "window" if self.window else "full"
-        return CacheRequest(kind, self.nkh, self.hd_pad, self.window, keep_first=self.keep_first if self.window else 0)
+        return CacheRequest(kind, self.nkh, self.hd_pad, self.cache_window, keep_first=self.keep_first if self.window else 0)
+
+    def state_bytes(self) -> int:
+        return (self.taps - 1) * self.channels * 4 if self.taps > 1 else 0
 
     def takes_row_scale(self) -> bool:
         return self.qkv.takes_row_scale()
@@ -224,11 +269,13 @@ class GQAAttention(Mixer):
         if cache is None:
             raise RuntimeError("gqa_attention needs a cache view")
         rt = self.rt
-        fused = self.pe.accepts_deferred and not self.prep
+        fused = self.pe.accepts_deferred and not self.prep and not self.taps
         qkv = self.qkv.forward(x, defer_to=ctx if fused else None, in_scale=ctx.take_row_scale(x))
         gate = qkv[:, self.gate_col:self.gate_col + self.nqh] if self.gate_col is not None else None
         if self.prep:
             return self._forward_padded(qkv, gate, residual, ctx, cache)
+        if self.taps:
+            return self._forward_conv(qkv, residual, ctx, cache, state)
         if self.qk_norm or self.value_from_key:
             self.pe.norm_encode_and_store(qkv, self.nqh, self.nkh, ctx, cache, self.q_norm_w, self.k_norm_w,
                                           self.qk_norm[0] if self.qk_norm else 0.0, self.value_from_key)
@@ -281,6 +328,32 @@ class GQAAttention(Mixer):
             out = y
         return self._project(out, residual, ctx)
 
+    def _forward_conv(self, proj, residual, ctx, cache, state):
+        """Convolution, norm, rotation, padding and the cache write in one kernel, attention over the padded heads, then the
+        value columns alone, gated, go on to the output product."""
+        K = self.rt.kernels
+        rows, D = proj.shape[0], self.hd_pad
+        if self.shared_kv != cache.read_only:
+            raise RuntimeError("gqa_attention: a layer without keys and values reads another layer's cache (cache_of)")
+        q = self.rt.empty(rows, self.nqh * D)
+        eps = self.qk_norm[0] if self.qk_norm else 0.0
+        head = dict(rotate=True, pad=D, norm="rms" if self.qk_norm else None)
+        segments = [K.conv_segment(self.nqh, self.hd, weight=self.q_norm_w, out=q, **head)]
+        if not self.shared_kv:
+            segments += [K.conv_segment(self.nkh, self.hd, weight=self.k_norm_w, plane=0, **head),
+                         K.conv_segment(self.nkh, self.vd, plane=1, pad=D)]
+        K.conv_heads(proj[:, :self.channels], self.conv_w, self.conv_b, state, 0, ctx, segments, eps=eps,
+                     inv_freq=self.pe.inv_freq, adjacent=self.pe.pairing == "adjacent", amplitude=self.pe.amplitude,
+                     page_table=cache.page_table, cache=None if self.shared_kv else cache.storage)
+        out = self.rt.empty(rows, self.nqh * D)
+        self._attend(q, out, ctx, cache, D)
+        if self.column_gate or D != self.vd:
+            g = proj[:, self.channels:self.channels + self.nqh * self.vd] if self.column_gate else None
+            y = self.rt.empty(rows, self.nqh * self.vd)
+            K.head_gate(out, g, y, self.nqh, D, self.vd, per_column=self.column_gate)
+            out = y
+        return self._project(out, residual, ctx)
+
     def _attend(self, qkv, out, ctx, cache, hd, gate=None, value_heads: int = 1) -> None:
         """Pick the attention kernel for this step.  float32 runs, and runs that ask for
         the plain kernels, use the one-warp-per-query kernel for everything.  bfloat16
@@ -296,14 +369,14 @@ class GQAAttention(Mixer):
                           self.nqh, self.nkh, hd, cache.page_size, self.window, self.scale, sink=self.sink,
                           head_sinks=self.head_sinks, head_gate=gate, out_scale=self.out_mult,
                           keep_first=self.keep_first, head_scale=self.head_scale, value_heads=value_heads,
-                          distance_bias=self.distance_bias)
+                          distance_bias=self.distance_bias, softcap=self.softcap)
             return
         few = ctx.max_q_len <= 8
         if not few and self.rt.attention_backend == "auto" and K.attn_tc_supports(hd) and not extras:
             K.attn_tc(qkv, out, cache.storage, cache.page_table, ctx.q_start, ctx.q_len, ctx.kv_before,
                       ctx.n_seqs, ctx.max_q_len, self.nqh, self.nkh, hd, self.window, self.scale, sink=self.sink,
                       head_sinks=self.head_sinks, head_gate=gate, out_scale=self.out_mult,
-                      distance_bias=self.distance_bias)
+                      distance_bias=self.distance_bias, softcap=self.softcap)
             return
         n_splits = 1
         if few:
@@ -317,4 +390,4 @@ class GQAAttention(Mixer):
                    ctx.n_seqs, ctx.max_q_len, self.nqh, self.nkh, hd, self.window, self.scale,
                    n_splits=n_splits, few_tokens=few, sink=self.sink, head_sinks=self.head_sinks, head_gate=gate,
                    out_scale=self.out_mult, keep_first=self.keep_first, head_scale=self.head_scale,
-                   value_heads=value_heads, distance_bias=self.distance_bias)
+                   value_heads=value_heads, distance_bias=self.distance_bias, softcap=self.softcap)

@@ -10,7 +10,8 @@ crates/braidinfer-runtime/src/config.rs:552).  Reads the float32 residual stream
 the run's element type; the sum of squares and the scale are float32.  With `offset` the stored weight w is
 zero-centred and applied as offset + w (offset 1: y = x * rsqrt(mean(x^2) + eps) * (1 + w)), added in float32.
 With `scalar` the stored weight is one number that every column is multiplied by (it is spread over the columns when it
-is loaded, so every kernel that fuses the norm serves it).
+is loaded, so every kernel that fuses the norm serves it).  `gain` is a constant factor on the result (a factor on a
+model's logits, say, on the rows its head reads); it is multiplied into the weights, in float32, when they are loaded.
 `add_into(y, h)` norms a branch's float32 result y and adds it to the float32 stream h in one kernel, for
 layers that norm what a sublayer returns instead of what it reads."""
 from __future__ import annotations
@@ -27,7 +28,7 @@ from .spec import TensorSpec
 @NORMS.register("rmsnorm")
 class RMSNorm(Norm):
     """params: width, eps, name (tensor name under the prefix), offset (added to the stored weight; default 0), scalar (one
-    stored number instead of one a column; default False)."""
+    stored number instead of one a column; default False), gain (a constant factor on the result; default 1)."""
 
     accepts_deferred = True      # adds a deferred residual sum in the same kernel as the norm
 
@@ -38,6 +39,9 @@ class RMSNorm(Norm):
         self.name = prefix + params["name"]
         self.offset = float(params.get("offset", 0.0))
         self.scalar = bool(params.get("scalar", False))
+        self.gain = float(params.get("gain", 1.0))
+        if self.gain != 1.0 and self.offset:
+            raise ValueError("rmsnorm: a constant factor goes with plain weights")
         if self.offset:
             self.accepts_deferred = False        # the kernels that add up partial sums apply plain weights
         self.weight: Optional[torch.Tensor] = None
@@ -53,9 +57,16 @@ class RMSNorm(Norm):
     def load(self, tensors) -> None:
         w = tensors[self.name]
         self.weight = w.reshape(1).expand(self.width).contiguous() if self.scalar else w
+        if self.gain != 1.0:
+            self.weight = self.weight.float() * self.gain        # in 32 bits: no rounding beside the result's own
 
     def forward(self, x: torch.Tensor, ctx=None, row_index: Optional[torch.Tensor] = None,
-                rows: Optional[int] = None, reader_takes_row_scale: bool = False) -> torch.Tensor:
+                rows: Optional[int] = None, reader_takes_row_scale: bool = False, in_place: bool = False) -> torch.Tensor:
+        """`in_place`: x is not needed any more and the result stays float32 (an embedding's norm: its output is the stream)."""
+        if in_place:
+            out = torch.empty_like(x)
+            self.rt.kernels.rmsnorm(x, self.weight, out, self.eps, w_offset=self.offset)
+            return out
         n = rows if rows is not None else x.shape[0]
         out = self.rt.empty(n, self.width)
         if self.offset:

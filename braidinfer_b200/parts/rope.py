@@ -14,6 +14,11 @@ pair index that turns t times over the original length, lo = max(floor(d(fast)),
 rd - 1) and ramp_p = clamp((p - lo) / max(hi - lo, 0.001), 0, 1):
     f'_p = f_p / factor * ramp_p + f_p * (1 - ramp_p),     amplitude = 0.1 ln(factor) + 1 on sine and cosine.
 Fast pairs keep their frequency, slow pairs are divided by the factor, those between are blended.
+With `"kind": "bands"` the scaling is the other common one (Grattafiori and others: "The Llama 3 Herd of Models", 2024,
+whose 3.1 models use it), by wavelength: l_p = 2 pi / f_p, two bounds `high` > `low` on original / l_p, no amplitude:
+    f'_p = f_p                                      l_p < original / high
+    f'_p = f_p / factor                             l_p > original / low
+    f'_p = (1 - s) f_p / factor + s f_p             between, s = (original / l_p - low) / (high - low)
 """
 from __future__ import annotations
 
@@ -26,12 +31,24 @@ from .base import POSITION_ENCODINGS, PositionEncoding
 
 def rotary_frequencies(rope_dim: int, theta: float, scaling=None):
     """(inv_freq [rope_dim / 2] float64, amplitude) of a rotation, with the optional `scaling`
-    {"factor", "original", "fast", "slow"} described in this module's head."""
+    {"factor", "original", "fast", "slow"} or {"kind": "bands", "factor", "original", "low", "high"} described in this
+    module's head."""
     p = torch.arange(rope_dim // 2, dtype=torch.float64)
     inv = 1.0 / (theta ** (2.0 * p / rope_dim)) if rope_dim else p
     if not scaling:
         return inv, 1.0
     factor, original = float(scaling["factor"]), float(scaling["original"])
+    kind = scaling.get("kind", "yarn")
+    if kind == "bands":
+        low, high = float(scaling["low"]), float(scaling["high"])
+        if factor <= 0 or original <= 0 or low <= 0 or high <= low:
+            raise ValueError(f"rope scaling by bands wants positive factor, original and low < high, got {dict(scaling)}")
+        turns = original * inv / (2.0 * math.pi)                      # original / wavelength
+        s = (turns - low) / (high - low)
+        mixed = (1.0 - s) * inv / factor + s * inv
+        return torch.where(turns > high, inv, torch.where(turns < low, inv / factor, mixed)), 1.0
+    if kind != "yarn":
+        raise ValueError(f"rope scaling of kind {kind!r} is not built (yarn, bands)")
     fast, slow = float(scaling["fast"]), float(scaling["slow"])
     if factor <= 0 or original <= 0 or fast <= 0 or slow <= 0:
         raise ValueError(f"rope scaling wants positive factor, original, fast and slow, got {dict(scaling)}")
@@ -48,7 +65,7 @@ def rotary_frequencies(rope_dim: int, theta: float, scaling=None):
 @POSITION_ENCODINGS.register("rope")
 class RotaryEncoding(PositionEncoding):
     """params: head_dim, theta, rope_dim (default head_dim), pairing ("half" | "adjacent"), scaling (None, or
-    {"factor", "original", "fast", "slow"}: see the module's head)."""
+    {"factor", "original", "fast", "slow"}, or {"kind": "bands", ...}: see the module's head)."""
 
     accepts_deferred = True      # adds a deferred q/k/v product in the same kernel as the rotation
     # ... in steps of up to this many rows.  That kernel runs a small CTA per row and head, which saves a
