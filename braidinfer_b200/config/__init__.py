@@ -6,6 +6,7 @@ from .loduzen import LoduzenConfig
 from .birepel import BirepelConfig
 from .ludazen import LudazenConfig
 from .zisesun import ZisesunConfig
+from .megerax import MegeraxConfig
 from .presets import PRESETS, preset
 
 
