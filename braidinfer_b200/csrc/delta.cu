@@ -6,22 +6,22 @@
 // a decay a channel.)  q, k, v arrive as float32 rows (convolved, of unit length and scaled: conv_heads.cu), z as float32
 // logits, b in the run's type; everything here is float32 arithmetic on the ordinary pipes.
 //
-// Short steps are walked token by token (delta_walk_kernel).  Long ones are cut into chunks of 64 tokens.  With L_t the
-// running sum of log2 g inside a chunk (a channel), S_0 the state it starts from, and every product weighed by the decay
-// between its two tokens, the walk over a chunk is
-//     A_ts = sum_i k_t k_s 2^(L_t - L_s)  (s < t),     P_ts = sum_i q_t k_s 2^(L_t - L_s)  (s <= t)
-//     (I + diag(beta) A) [W | U0] = diag(beta) [k_t 2^(L_t) | v_t]                    (forward substitution)
+// Short steps are walked token by token (delta_walk_kernel).  Long ones are cut into chunks of 64 tokens.  With D(s, t) the product
+// of the decays of the tokens after s up to t (a channel; 0: the chunk's start) and S_0 the state a chunk starts from, the
+// walk over a chunk is
+//     A_ts = sum_i k_t k_s D(s, t)  (s < t),     P_ts = sum_i q_t k_s D(s, t)  (s <= t)
+//     (I + diag(beta) A) [W | U0] = diag(beta) [k_t D(0, t) | v_t]                    (forward substitution)
 //     U = U0 - W S_0
-//     O = (q_t 2^(L_t)) S_0 + P U
-//     S_64 = diag(2^(L_64)) S_0 + (k_t 2^(L_64 - L_t))^T U
+//     O = (q_t D(0, t)) S_0 + P U
+//     S_64 = diag(D(0, 64)) S_0 + (k_t D(t, 64))^T U
 // so all but the two products with S_0 that make U and the next S run for all chunks side by side:
 //     delta_intra_kernel   W, U0, P and the decayed q and k of every chunk
 //     delta_state_kernel   chunk after chunk, a tile of value columns a CTA: U, and the state every chunk starts from
 //     delta_out_kernel     O of every chunk
-// Every 2^x above has x <= 0 where it is taken: sub-chunks of 16 tokens are related through the running sum at their edges,
-// and inside a sub-chunk 2^(L_t - L_s) is taken as 2^(L_t - edge) 2^(edge - L_s) only while the second factor stays below
-// 2^60, pair by pair beyond.  log2 g is held at or above -32 (a token that forgets more than 32 binary digits of a channel
-// forgets all that float32 holds), which keeps the running sums' own rounding small.
+// No logarithm is taken: the decay between two tokens is a product of at most 16 decays at a time, which rounds like the walk
+// does.  Sub-chunks of 16 tokens are related through the products at their edges (never above one).  Inside a sub-chunk the
+// decay from s to t is taken as (edge to t) / (edge to s) for the channels whose decays over the sub-chunk multiply to 2^-60 or
+// more, and multiplied up pair by pair for the others.
 #include "common.cuh"
 #include "gated_norm.cuh"
 
@@ -33,8 +33,7 @@
 #define DELTA_NSUB (DELTA_C / DELTA_SUB)
 #define DELTA_DVT 32               // value columns a CTA of the chunk-after-chunk kernel
 #define DELTA_OUT_COLS 64          // value columns a CTA of the output kernel
-#define DELTA_LOG_MIN (-32.f)
-#define DELTA_SPREAD 60.f
+#define DELTA_SPREAD 8.6736174e-19f      // 2^-60
 
 struct DeltaArgs {
     const float* q; long long q_stride;          // [rows, groups * dk]
@@ -54,10 +53,9 @@ struct DeltaArgs {
     int dk4, dv4, max_chunks;
 };
 
-// log2 of a decay from its logit: -rate softplus(x) log2(e), held at DELTA_LOG_MIN
-__device__ __forceinline__ float delta_log_decay(float x, float rate) {
-    const float sp = fmaxf(x, 0.f) + log1pf(expf(-fabsf(x)));
-    return fmaxf(-rate * sp * 1.4426950408889634f, DELTA_LOG_MIN);
+// a decay from its logit: exp(-rate softplus(x))
+__device__ __forceinline__ float delta_decay(float x, float rate) {
+    return expf(-rate * (fmaxf(x, 0.f) + log1pf(expf(-fabsf(x)))));
 }
 __device__ __forceinline__ float delta_sigmoid(float x) { return 1.f / (1.f + expf(-x)); }
 
@@ -120,7 +118,7 @@ delta_walk_kernel(DeltaArgs a) {
             const int idx = tid + w * DELTA_WALK_THREADS, t = idx / DKP, i = idx - t * DKP;
             sq[idx] = pq[w];
             sk[idx] = pk[w];
-            if (t < nt) sa[idx] = i < dk ? exp2f(delta_log_decay(pz[w] + a.bias[(size_t)h * dk + i], rate)) : 0.f;
+            if (t < nt) sa[idx] = i < dk ? delta_decay(pz[w] + a.bias[(size_t)h * dk + i], rate) : 0.f;
         }
 #pragma unroll
         for (int w = 0; w < NV; ++w) sv[tid + w * DELTA_WALK_THREADS] = pv[w];
@@ -180,29 +178,35 @@ delta_walk_kernel(DeltaArgs a) {
 
 // ------------------------------------------------------------------ inside every chunk
 #define DELTA_INTRA_THREADS 256
+// A's rows take the place of q's once those have been used, where a row is wide enough
 template <int DKP> constexpr int delta_intra_smem() {
-    return (3 * DELTA_C * (DKP + 4) + DELTA_C * (DELTA_C + 4) + DELTA_C + (DELTA_NSUB + 1) * DKP) * 4;
+    return (3 * DELTA_C * (DKP + 4) + (DKP < DELTA_C ? DELTA_C * (DELTA_C + 4) : 0) + DELTA_C + 3 * DKP) * 4;
 }
 
 template <typename T, int DKP>
-__global__ void __launch_bounds__(DELTA_INTRA_THREADS)
+__global__ void __launch_bounds__(DELTA_INTRA_THREADS, DKP <= 128 ? 2 : 1)
 delta_intra_kernel(DeltaArgs a) {
-    constexpr int C = DELTA_C, LD = DKP + 4, LA = C + 4, NT = DELTA_INTRA_THREADS;
+    constexpr int C = DELTA_C, SUB = DELTA_SUB, LD = DKP + 4, NT = DELTA_INTRA_THREADS;
+    constexpr bool OWN_A = DKP < C;
+    constexpr int LA = OWN_A ? C + 4 : LD;
+    static_assert(DKP <= NT, "a thread a channel");
     extern __shared__ __align__(16) float sm[];
-    float* sK = sm;                          // k, then k 2^(edge - L) for the edge reached so far
-    float* sQ = sK + C * LD;                 // q, then q 2^(L - edge of its sub-chunk)
-    float* sL = sQ + C * LD;                 // L, then k 2^(L - edge), then k 2^L
-    float* sA = sL + C * LD;                 // beta_t A_ts
-    float* sB = sA + C * LA;                 // beta
-    float* sR = sB + C;                      // [5][DKP]: L at the edges of the sub-chunks
-    __shared__ int steep;                    // bit J: sub-chunk J decays by more than DELTA_SPREAD in some channel
+    float* sK = sm;                          // k, then k over the decays up to it, then k times the decays after it
+    float* sQ = sK + C * LD;                 // q, then q times the decays from its sub-chunk's edge
+    float* sG = sQ + C * LD;                 // g, then k times the decays from the edge, then from the chunk's start
+    float* sA = OWN_A ? sG + C * LD : sQ;    // beta_t A_ts
+    float* sB = sG + C * LD + (OWN_A ? C * LA : 0);      // beta
+    float* sT = sB + C;                      // the product of a sub-chunk's decays
+    float* sE = sT + DKP;                    // the product of all decays before the sub-chunk
+    int* steep = (int*)(sE + DKP);           // the channels whose factors cannot be split, their number in n_steep
+    __shared__ int n_steep;
     pdl_trigger();
     const int h = blockIdx.x, seq = blockIdx.y, c = blockIdx.z, tid = threadIdx.x;
     const int n = min(C, a.q_len[seq] - c * C), r0 = a.q_start[seq] + c * C;
     if (n <= 0) return;
     const int dk = a.dk, dv = a.dv, g = h / (a.heads / a.groups);
     const float rate = a.rate[h];
-    if (tid == 0) steep = 0;
+    if (tid == 0) n_steep = 0;
     pdl_wait();
     for (int idx = tid; idx < C * DKP; idx += NT) {
         const int t = idx / DKP, i = idx - t * DKP;
@@ -210,108 +214,136 @@ delta_intra_kernel(DeltaArgs a) {
         const bool in = t < n && i < dk;
         sK[t * LD + i] = in ? a.k[row * a.k_stride + (size_t)g * dk + i] : 0.f;
         sQ[t * LD + i] = in ? a.q[row * a.q_stride + (size_t)g * dk + i] : 0.f;
-        sL[t * LD + i] = in ? delta_log_decay(a.z[row * a.z_stride + (size_t)h * dk + i] + a.bias[(size_t)h * dk + i], rate) : 0.f;
+        sG[t * LD + i] = in ? delta_decay(a.z[row * a.z_stride + (size_t)h * dk + i] + a.bias[(size_t)h * dk + i], rate) : 1.f;
     }
     if (tid < C) sB[tid] = tid < n ? delta_sigmoid(to_f32(((const T*)a.b)[(size_t)(r0 + tid) * a.b_stride + h])) : 0.f;
+    if (tid < DKP) sE[tid] = 1.f;
     __syncthreads();
-    for (int i = tid; i < DKP; i += NT) {
-        float L = 0.f;
-        sR[i] = 0.f;
-#pragma unroll 1
-        for (int J = 0; J < DELTA_NSUB; ++J) {
-            const float edge = L;
-#pragma unroll
-            for (int t = 0; t < DELTA_SUB; ++t) {
-                float* p = sL + (J * DELTA_SUB + t) * LD + i;
-                L += *p;
-                *p = L;
-            }
-            sR[(J + 1) * DKP + i] = L;
-            if (edge - L > DELTA_SPREAD) atomicOr(&steep, 1 << J);
-        }
-    }
-    __syncthreads();
-    const int all_steep = steep;
     const int ty = tid >> 4, tx = tid & 15;
     const size_t hrow0 = (size_t)r0 * a.heads + h;                 // + t * heads: index of (row, head)
 #pragma unroll 1
     for (int J = 0; J < DELTA_NSUB; ++J) {
-        const bool direct = (all_steep >> J) & 1;
-        const float *edge = sR + J * DKP, *next = edge + DKP;
-        // this sub-chunk's rows; a steep one's pairs first, while k, q and L are there as they came
-        const int t = J * DELTA_SUB + ty;
-        float accA[DELTA_NSUB], accP[DELTA_NSUB];
+        const int row0 = J * SUB, t = row0 + ty;
+        // a thread a channel: the factors of this sub-chunk's rows
+        float e[SUB], kd[SUB];
+        bool split = true;
+        if (tid < DKP) {
+            float prod = 1.f;
 #pragma unroll
-        for (int I = 0; I < DELTA_NSUB; ++I) { accA[I] = 0.f; accP[I] = 0.f; }
-        float dA = 0.f, dP = 0.f;
-        if (direct) {
-            const int s = J * DELTA_SUB + tx;
+            for (int r = 0; r < SUB; ++r) {
+                prod *= sG[(row0 + r) * LD + tid];
+                e[r] = prod;
+            }
+            sT[tid] = prod;
+            split = prod >= DELTA_SPREAD;
+            if (split) {
+#pragma unroll
+                for (int r = 0; r < SUB; ++r) {
+                    const int at = (row0 + r) * LD + tid;
+                    const float kk = sK[at];
+                    sQ[at] *= e[r];
+                    sG[at] = kk * e[r];
+                    sK[at] = __fdividef(kk, e[r]);
+                }
+            } else {
+                steep[atomicAdd(&n_steep, 1)] = tid;
+                float after = 1.f;
+#pragma unroll
+                for (int r = SUB - 1; r >= 0; --r) {
+                    const int at = (row0 + r) * LD + tid;
+                    kd[r] = sK[at] * after;
+                    after *= sG[at];
+                }
+            }
+        }
+        __syncthreads();
+        float dA = 0.f, dP = 0.f;                                   // the diagonal block's sums over the steep channels
+        const int ns = n_steep;
+        if (ns > 0) {
             if (tx <= ty)
-                for (int i = 0; i < dk; ++i) {
-                    const float ks = sK[s * LD + i] * exp2f(sL[t * LD + i] - sL[s * LD + i]);
+                for (int w = 0; w < ns; ++w) {
+                    const int i = steep[w];
+                    float ks = sK[(row0 + tx) * LD + i];
+                    for (int r = tx + 1; r <= ty; ++r) ks *= sG[(row0 + r) * LD + i];
                     dA = fmaf(sK[t * LD + i], ks, dA);
                     dP = fmaf(sQ[t * LD + i], ks, dP);
                 }
             __syncthreads();
-        }
-        for (int idx = tid; idx < (J + 1) * DELTA_SUB * DKP; idx += NT) {
-            const int r = idx / DKP, i = idx - r * DKP;
-            if (r < J * DELTA_SUB) {
-                // an earlier row: on to this sub-chunk's edge (a steep sub-chunk's rows are there already when it is the last)
-                const int Jr = r / DELTA_SUB;
-                if (!(Jr == J - 1 && ((all_steep >> Jr) & 1))) sK[r * LD + i] *= exp2f(edge[i] - (edge - DKP)[i]);
-            } else {
-                const float L = sL[r * LD + i], kk = sK[r * LD + i], d = L - edge[i], e = exp2f(d);
-                sQ[r * LD + i] *= e;
-                sL[r * LD + i] = kk * e;
-                sK[r * LD + i] = kk * (direct ? exp2f(next[i] - L) : exp2f(-d));
+            if (!split) {
+#pragma unroll
+                for (int r = 0; r < SUB; ++r) {
+                    const int at = (row0 + r) * LD + tid;
+                    sQ[at] *= e[r];
+                    sG[at] = sK[at] * e[r];
+                    sK[at] = 0.f;
+                }
             }
+            if (tid == 0) n_steep = 0;
+            __syncthreads();
         }
-        __syncthreads();
+        float accA[DELTA_NSUB], accP[DELTA_NSUB];
+#pragma unroll
+        for (int I = 0; I < DELTA_NSUB; ++I) { accA[I] = 0.f; accP[I] = 0.f; }
         {
-            const float *ra = sL + t * LD, *rq = sQ + t * LD, *rk = sK + tx * LD;
-            const int last = direct ? J : J + 1;                    // the diagonal block is one of the products unless steep
-#pragma unroll 1
+            const float *ra = sG + t * LD, *rq = sQ + t * LD, *rk = sK + tx * LD;
+#pragma unroll 2
             for (int i = 0; i < DKP; i += 4) {
                 const float4 ka = *reinterpret_cast<const float4*>(ra + i), qa = *reinterpret_cast<const float4*>(rq + i);
 #pragma unroll
                 for (int I = 0; I < DELTA_NSUB; ++I)
-                    if (I < last) {
-                        const float4 kb = *reinterpret_cast<const float4*>(rk + I * DELTA_SUB * LD + i);
+                    if (I <= J) {
+                        const float4 kb = *reinterpret_cast<const float4*>(rk + I * SUB * LD + i);
                         accA[I] = fmaf(ka.x, kb.x, fmaf(ka.y, kb.y, fmaf(ka.z, kb.z, fmaf(ka.w, kb.w, accA[I]))));
                         accP[I] = fmaf(qa.x, kb.x, fmaf(qa.y, kb.y, fmaf(qa.z, kb.z, fmaf(qa.w, kb.w, accP[I]))));
                     }
             }
-            const float beta = sB[t];
+#pragma unroll
+            for (int I = 0; I < DELTA_NSUB; ++I)
+                if (I == J) { accA[I] += dA; accP[I] += dP; }
+        }
+        if (t < n) {
 #pragma unroll
             for (int I = 0; I < DELTA_NSUB; ++I)
                 if (I <= J) {
-                    const int s = I * DELTA_SUB + tx;
-                    const float A = (direct && I == J) ? dA : accA[I], P = (direct && I == J) ? dP : accP[I];
-                    sA[t * LA + s] = s < t ? beta * A : 0.f;
-                    if (t < n) a.p[(hrow0 + (size_t)t * a.heads) * C + s] = s <= t ? P : 0.f;
+                    const int s = I * SUB + tx;
+                    a.p[(hrow0 + (size_t)t * a.heads) * C + s] = s <= t ? accP[I] : 0.f;
                 }
         }
         __syncthreads();
-        // k 2^L stays for the substitution, q 2^L goes out
-        for (int idx = tid; idx < DELTA_SUB * DKP; idx += NT) {
-            const int r = J * DELTA_SUB + idx / DKP, i = idx % DKP;
-            const float e = exp2f(edge[i]);
-            sL[r * LD + i] *= e;
-            if (r < n && i < a.dk4) a.qd[(hrow0 + (size_t)r * a.heads) * a.dk4 + i] = sQ[r * LD + i] * e;
+        // k on to the sub-chunk's end; k and q from the chunk's start (q goes out)
+        for (int idx = tid; idx < (J + 1) * SUB * DKP; idx += NT) {
+            const int r = idx / DKP, i = idx - r * DKP, at = r * LD + i;
+            if (r < row0) sK[at] *= sT[i];
+            else {
+                const float E = sE[i];
+                sG[at] *= E;
+                if (r < n && i < a.dk4) a.qd[(hrow0 + (size_t)r * a.heads) * a.dk4 + i] = sQ[at] * E;
+            }
         }
-    }
-    __syncthreads();
-    {
-        const float *edge = sR + (DELTA_NSUB - 1) * DKP, *end = edge + DKP;
-        for (int idx = tid; idx < n * DKP; idx += NT) {
-            const int r = idx / DKP, i = idx - r * DKP;
-            const bool there = r / DELTA_SUB == DELTA_NSUB - 1 && ((all_steep >> (DELTA_NSUB - 1)) & 1);
-            if (i < a.dk4) a.kd[(hrow0 + (size_t)r * a.heads) * a.dk4 + i] = sK[r * LD + i] * (there ? 1.f : exp2f(end[i] - edge[i]));
+        if (tid < DKP) {
+#pragma unroll
+            for (int r = 0; r < SUB; ++r) {
+                float* at = sK + (row0 + r) * LD + tid;
+                *at = split ? *at * e[SUB - 1] : kd[r];
+            }
         }
-        float* gc = a.gc + ((size_t)(seq * a.max_chunks + c) * a.heads + h) * a.dk4;
-        for (int i = tid; i < a.dk4; i += NT) gc[i] = exp2f(end[i]);
+        __syncthreads();
+        if (tid < DKP) sE[tid] *= sT[tid];
+        const float beta = sB[t];
+#pragma unroll
+        for (int I = 0; I < DELTA_NSUB; ++I)
+            if (I <= J) {
+                const int s = I * SUB + tx;
+                sA[t * LA + s] = s < t ? beta * accA[I] : 0.f;
+            }
+        __syncthreads();
     }
+    for (int idx = tid; idx < n * DKP; idx += NT) {
+        const int r = idx / DKP, i = idx - r * DKP;
+        if (i < a.dk4) a.kd[(hrow0 + (size_t)r * a.heads) * a.dk4 + i] = sK[r * LD + i];
+    }
+    float* gc = a.gc + ((size_t)(seq * a.max_chunks + c) * a.heads + h) * a.dk4;
+    for (int i = tid; i < a.dk4; i += NT) gc[i] = sE[i];
     // forward substitution: a thread a column, its 64 numbers in registers
     for (int col = tid; col < a.dk4 + a.dv4; col += NT) {
         const bool is_w = col < a.dk4;
@@ -319,7 +351,7 @@ delta_intra_kernel(DeltaArgs a) {
         float x[C];
 #pragma unroll
         for (int t = 0; t < C; ++t)
-            x[t] = is_w ? sL[t * LD + col] : (t < n && vc < dv) ? a.v[(size_t)(r0 + t) * a.v_stride + (size_t)h * dv + vc] : 0.f;
+            x[t] = is_w ? sG[t * LD + col] : (t < n && vc < dv) ? a.v[(size_t)(r0 + t) * a.v_stride + (size_t)h * dv + vc] : 0.f;
 #pragma unroll
         for (int t = 0; t < C; ++t) {
             float acc = x[t] * sB[t];
@@ -453,7 +485,7 @@ delta_state_kernel(DeltaArgs a) {
         delta_cp_commit();
         delta_cp_wait<1>();                                // this chunk's k
         __syncthreads();
-        // S = diag(2^L) S + K^T U
+        // S = diag(D) S + K^T U
 #pragma unroll
         for (int e = 0; e < RI; ++e)
 #pragma unroll
