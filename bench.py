@@ -1841,6 +1841,247 @@ def zisesun_kernels(z, T, B, C, timed, frac):
     return res
 
 
+# ------------------------------------------------------------------ the Megerax decoder beside the Loduzen one
+# what `LODUZEN_SIZES` does not have: the latent layer's heads, sizes and ranks, and the delta layers' inner sizes
+MEGERAX_LATENT = {
+    "w2048": dict(heads=16, dim=128, rot=64, vdim=128, q_rank=1024, kv_rank=512, low=128),
+    "w4096": dict(heads=32, dim=128, rot=64, vdim=128, q_rank=1536, kv_rank=512, low=128),
+    "w1024": dict(heads=8, dim=64, rot=32, vdim=64, q_rank=512, kv_rank=256, low=64),
+}
+
+
+def megerax_config(name):
+    """Four layers at the sizes of `LODUZEN_SIZES`: a latent layer and a windowed attention layer with feed-forwards, a delta
+    layer without after each; the attention heads and the window of that model's attention, the delta heads of its linear
+    attention."""
+    z, y = LODUZEN_SIZES[name], MEGERAX_LATENT[name]
+    ff = {"kind": "dense", "ff": z["ff"]}
+    att = {"heads": z["heads"], "kv_heads": z["kv"], "dim": z["dim"], "vdim": z["dim"], "conv": 4, "scale": z["dim"] ** -0.5, "softcap": 50.0,
+           "mask": {"size": z["window"]},
+           "rot": {"base": 1e6, "dims": z["dim"] // 2, "scaling": {"factor": 4.0, "low": 1.0, "high": 4.0, "original": 4096}}}
+    delta = {"heads": z["lheads"], "kv_heads": z["lheads"], "dim": z["ldk"], "vdim": z["ldv"], "conv": 4, "decay_rank": y["low"],
+             "gate_rank": y["low"]}
+    lat = {"heads": y["heads"], "dim": y["dim"], "rot_dim": y["rot"], "vdim": y["vdim"], "q_rank": y["q_rank"], "kv_rank": y["kv_rank"],
+           "scale": (y["dim"] + y["rot"]) ** -0.5, "rot": {"base": 1e6, "dims": y["rot"]}}
+    d = {"type": "channel_delta", "mixer": delta, "mlp": None}
+    return {"architecture": "Megerax", "vocab": z["vocab"], "width": z["width"], "logit_scale": 0.5, "norm": {"eps": 1e-6},
+            "layers": [{"type": "latent_attention", "mixer": lat, "mlp": ff}, d, {"type": "attention", "mixer": att, "mlp": ff}, d]}
+
+
+def loduzen_pair_config(name):
+    """The Loduzen decoder with as many attentions, recurrences and feed-forwards as `megerax_config`: two layers of an attention
+    beside a gated linear attention, no token input."""
+    cfg = loduzen_config(LODUZEN_SIZES[name])
+    return {k: v for k, v in dict(cfg, layers=[cfg["layers"][0]] * 2).items() if k != "token_side"}
+
+
+def run_megerax(args):
+    """`--megerax`: prompt and decode throughput of the Megerax decoder at sizes like a real model's layers (random weights), beside
+    the Loduzen decoder of equal size (the closest model here: windowed attention with head norms beside linear attention with a
+    decay a channel, a gelu-gated feed-forward), and the new kernels one by one beside the like kernels of the models that have
+    them, with their fractions of the measured peaks.  Prints one JSON line of its own; the default run and its line are
+    untouched."""
+    import torch
+    from braidinfer_b200.engine import Engine
+    pk = peaks()
+    flush = torch.empty(256 << 20, dtype=torch.uint8, device="cuda")
+
+    def timed(fn, reps=5, warm=2, graph=False):
+        for _ in range(warm):
+            fn()
+        run = fn
+        if graph:
+            torch.cuda.synchronize()
+            gr = torch.cuda.CUDAGraph()
+            with torch.cuda.graph(gr):
+                fn()
+            run = gr.replay
+            run()
+        ts = []
+        for _ in range(reps):
+            flush.zero_()
+            torch.cuda.synchronize()
+            e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+            e0.record()
+            run()
+            e1.record()
+            torch.cuda.synchronize()
+            ts.append(e0.elapsed_time(e1) / 1e3)
+        return statistics.median(ts)
+
+    def frac(seconds, flops, nbytes):
+        return max(flops / (pk["bf16_tflops"] * 1e12), nbytes / (pk["hbm_gbs"] * 1e9)) / seconds
+
+    T, B, C = args.prompt_len, args.batch, args.context
+    sizes = [n for n in LODUZEN_SIZES if not args.sizes or n in args.sizes.split(",")]
+    out = {"metric": "megerax_beside_loduzen_decoder", "unit": "tokens/s", "dtype": "bf16", "data": "synthetic, random weights",
+           "prompt_len": T, "decode_batch": B, "decode_context": C, "peaks": pk, "l2": "flushed between timed calls", "sizes": {}}
+    with ClockSampler() as clocks:
+        for name in sizes:
+            row = {}
+            for label, cfg in (("megerax", megerax_config(name)), ("loduzen", loduzen_pair_config(name))):
+                eng = Engine.from_random(cfg, 1, dtype="bfloat16", on_device=True, max_tokens=max(B * (C + 192), T + 64),
+                                         max_slots=B, verbose=False)
+                g = torch.Generator().manual_seed(0)
+                prompt = torch.randint(0, cfg["vocab"], (T,), generator=g).tolist()
+
+                def prefill():
+                    s = eng.open()
+                    eng.step([(s, prompt)], want="last")
+                    eng.close(s)
+                tp = timed(prefill, reps=3, warm=2)
+                prompts = [torch.randint(0, cfg["vocab"], (C,), generator=g).tolist() for _ in range(B)]
+                secs, ctx0, launches = device_timed_decode(eng, eng.kernels, prompts, args.steps, max(args.warmup, 3))
+                eng.check()
+                row[label] = {"prefill_tokens_per_s": round(T / tp), "prefill_ms": round(tp * 1e3, 3),
+                              "decode_tokens_per_s": round(B * args.steps / secs), "decode_ms_per_step": round(secs / args.steps * 1e3, 4),
+                              "weight_gb": round(eng.weight_bytes / 1e9, 3), "state_mb_per_sequence": round(sum(
+                                  s.shape[1] for s in eng.cache.state if s is not None) / 1e6, 3),
+                              "launches_per_decode_step": launches // args.steps}
+                del eng
+                torch.cuda.empty_cache()
+            row["kernels"] = megerax_kernels(name, T, B, C, timed, frac)
+            out["sizes"][name] = row
+    out["clocks"] = clocks.summary()
+    print(json.dumps(out))
+    return 0
+
+
+def megerax_kernels(name, T, B, C, timed, frac):
+    """The new kernels and options alone, each beside another model's like kernel: seconds, and the fraction of the measured peak
+    that its algorithmic FLOPs or bytes (whichever bounds it) reach.  The recurrences' `frac` is of the copy bandwidth (the bytes
+    they must move); `tflops` says what a walk token by token computes."""
+    import torch
+    from types import SimpleNamespace
+    from braidinfer_b200.cache import PAGE_SIZE
+    from braidinfer_b200.csrc.api import get_kernels
+    K = get_kernels(verbose=False)
+    z, y = LODUZEN_SIZES[name], MEGERAX_LATENT[name]
+    dev, bf = "cuda", torch.bfloat16
+    i32 = lambda v: torch.tensor(v, dtype=torch.int32, device=dev)        # noqa: E731
+    rnd = lambda *s: torch.randn(*s, device=dev, dtype=bf)                # noqa: E731
+    H, nkh, hd, win = z["heads"], z["kv"], z["dim"], z["window"]
+    res = {}
+
+    def paged(n_seqs, length, planes, heads, dim):
+        blocks = -(-length // PAGE_SIZE)
+        return rnd(n_seqs * blocks, planes, heads, PAGE_SIZE, dim) * 0.5, \
+            torch.arange(n_seqs * blocks, dtype=torch.int32, device=dev).view(n_seqs, blocks)
+
+    def steps_of(n_seqs, each, before):
+        rows = n_seqs * each
+        return SimpleNamespace(rows=rows, n_tokens=rows, n_seqs=n_seqs, q_start=i32([i * each for i in range(n_seqs)]),
+                               q_len=i32([each] * n_seqs), kv_before=i32([before] * n_seqs), slot_ids=i32(list(range(n_seqs))), max_q_len=each,
+                               token_seq=torch.arange(n_seqs, dtype=torch.int32, device=dev).repeat_interleave(each),
+                               positions=(torch.arange(each, dtype=torch.int32, device=dev) + before).repeat(n_seqs))
+
+    def pair(what, new, old, **more):
+        """(seconds, flops, bytes) of the new kernel and of the other model's like kernel"""
+        res[what] = {"megerax_ms": round(new[0] * 1e3, 4), "megerax_frac": round(frac(*new), 4)}
+        if old:
+            res[what].update(like_ms=round(old[0] * 1e3, 4), like_frac=round(frac(*old), 4))
+        res[what].update(more)
+
+    st, sd = steps_of(1, T, 0), steps_of(B, 1, C - 1)
+    for what, stp, n_seqs, each, length in (("prompt", st, 1, T, T), ("decode", sd, B, 1, C)):
+        rows, few = stp.rows, each == 1
+        # ---- attention: capped scores beside Loduzen's sink, behind the same window
+        cache, table = paged(n_seqs, length, 2, nkh, hd)
+        q, o = rnd(rows, H * hd) * 0.3, torch.empty(rows, H * hd, device=dev, dtype=bf)
+        span = min(length, win)
+        fl = 4 * H * hd * sum(min(p + 1, win) for p in range(length - each, length)) * n_seqs
+        by = n_seqs * span * 2 * nkh * hd * 2 if few else 0
+        sp = max(1, min(K.attn_decode_slots(hd) // (B * nkh * -(-(H // nkh) // 16)), (span // 32) // 4, 64)) if few else 1
+        t = {}
+        for label, kw in (("new", dict(softcap=50.0)), ("old", dict(sink=0.0))):
+            mma = timed(lambda: K.attn_mma(q, o, cache, table, stp.q_start, stp.q_len, stp.kv_before, stp.token_seq, n_seqs, each, H, nkh, hd,
+                                           win, hd ** -0.5, n_splits=sp, few_tokens=few, **kw), reps=9, graph=True)
+            t[label] = (mma, 0 if few else fl, by)
+            if not few and K.attn_tc_supports(hd):
+                tc = timed(lambda: K.attn_tc(q, o, cache, table, stp.q_start, stp.q_len, stp.kv_before, 1, T, H, nkh, hd, win, hd ** -0.5, **kw),
+                           reps=9, graph=True)
+                t[label + "_tc"] = (tc, fl, 0)
+        pair(f"{what}_attention_mma", t["new"], t["old"])
+        if "new_tc" in t:
+            qs = q * 40.0                      # scores near the cap: the other form of the tanh
+            far = timed(lambda: K.attn_tc(qs, o, cache, table, stp.q_start, stp.q_len, stp.kv_before, 1, T, H, nkh, hd, win, hd ** -0.5, softcap=50.0),
+                        reps=9, graph=True)
+            pair(f"{what}_attention_tcgen05", t["new_tc"], t["old_tc"], scores_near_the_cap_ms=round(far * 1e3, 4))
+        # ---- the gate a column beside Birepel's gate a head
+        gate = rnd(rows, H * hd)
+        t1 = timed(lambda: K.head_gate(q, gate, o, H, hd, hd, per_column=True), reps=9, graph=True)
+        t2 = timed(lambda: K.head_gate(q, gate, o, H, hd, hd), reps=9, graph=True)
+        pair(f"{what}_column_gate", (t1, 0, rows * H * hd * 6), (t2, 0, rows * H * hd * 4))
+        # ---- convolution + norm + rotation + cache write beside Loduzen's two kernels (convolution; norm, rotation, cache write)
+        ch = (H + 2 * nkh) * hd
+        x, w, b, wn = rnd(rows, ch), rnd(ch, 4), rnd(ch), rnd(hd)
+        cst = torch.zeros(n_seqs, 3 * ch * 4, dtype=torch.uint8, device=dev)
+        inv = torch.rand(hd // 4, device=dev)
+        head = dict(rotate=True, norm="rms", weight=wn)
+        segs = [K.conv_segment(H, hd, out=o, **head), K.conv_segment(nkh, hd, plane=0, **head), K.conv_segment(nkh, hd, plane=1)]
+        t1 = timed(lambda: K.conv_heads(x, w, b, cst, 0, stp, segs, eps=1e-6, inv_freq=inv, page_table=table, cache=cache), reps=9, graph=True)
+        yb = torch.empty(rows, ch, device=dev, dtype=bf)
+
+        def two():
+            K.causal_conv(x, yb, w, b, cst, 0, stp, silu=False)
+            K.head_norm_rope_kv(yb, wn, wn, inv, stp.positions, stp.token_seq, table, cache, H, nkh, hd, hd // 2, True, False, PAGE_SIZE, 1e-6)
+        t2 = timed(two, reps=9, graph=True)
+        pair(f"{what}_convolved_heads", (t1, 0, rows * ch * 4 + n_seqs * 3 * ch * 8), (t2, 0, rows * (ch * 4 + (H + nkh) * hd * 4 + 2 * nkh * hd * 2) + n_seqs * 3 * ch * 8))
+        # ---- the delta layer: its convolution (silu, unit heads, float32 out) beside Mamba-2's, the recurrence and the read-out beside
+        # those of the gated linear attention
+        heads, dk, dv = z["lheads"], z["ldk"], z["ldv"]
+        ch = heads * (2 * dk + dv)
+        x, w = rnd(rows, ch), rnd(ch, 4)
+        cst = torch.zeros(n_seqs, 3 * ch * 4, dtype=torch.uint8, device=dev)
+        f32 = lambda n: torch.empty(rows, n, device=dev)                  # noqa: E731
+        fq, fk, fv, oo = f32(heads * dk), f32(heads * dk), f32(heads * dv), f32(heads * dv)
+        segs = [K.conv_segment(heads, dk, silu=True, norm="unit", factor=dk ** -0.5, out=fq), K.conv_segment(heads, dk, silu=True, norm="unit", out=fk),
+                K.conv_segment(heads, dv, silu=True, out=fv)]
+        t1 = timed(lambda: K.conv_heads(x, w, None, cst, 0, stp, segs, eps=1e-6), reps=9, graph=True)
+        yb, cb = torch.empty(rows, ch, device=dev, dtype=bf), rnd(ch)
+        t2 = timed(lambda: K.causal_conv(x, yb, w, cb, cst, 0, stp), reps=9, graph=True)
+        pair(f"{what}_convolved_unit_heads", (t1, 0, rows * ch * 6 + n_seqs * 3 * ch * 8), (t2, 0, rows * ch * 4 + n_seqs * 3 * ch * 8))
+        S = torch.zeros(n_seqs, heads * dk * dv * 4, dtype=torch.uint8, device=dev)
+        zl, bl = torch.randn(rows, heads * dk, device=dev) - 3.0, rnd(rows, heads)
+        bias, rate = torch.zeros(heads * dk, device=dev), torch.ones(heads, device=dev)
+        delta = lambda r: (lambda: K.delta_rule(fq, fk, fv, zl, bias, r, bl, oo, S, 0, stp, heads, heads, dk, dv, chunked=not few))      # noqa: E731
+        t1 = timed(delta(rate), graph=True)
+        steep = timed(delta(rate * 200.0), graph=True)
+        by1 = rows * heads * ((3 * dk + 2 * dv) * 4 + 2) + 2 * n_seqs * heads * dk * dv * 4
+        qq, kk, vv = rnd(rows, heads * dk) * 0.1, rnd(rows, heads * dk) * 0.1, rnd(rows, heads * dv)
+        gd, zb = torch.rand(rows, heads * dk, device=dev) * 0.1 + 0.9, torch.zeros(heads * dk, device=dev, dtype=bf)
+        t2 = timed(lambda: K.linear_scan(qq, kk, vv, gd, zb, oo, S, 0, stp, heads, heads, dk, dv, "channel", q_scale=dk ** -0.5, inv_tau=1 / 8,
+                                         gate_is_decay=not few), graph=True)
+        by2 = rows * heads * (2 * dk * 2 + dv * 2 + dv * 4 + dk * 4) + 2 * n_seqs * heads * dk * dv * 4
+        pair(f"{what}_recurrence", (t1, 0, by1), (t2, 0, by2), every_channel_steep_ms=round(steep * 1e3, 4),
+             megerax_tflops=round(6 * rows * heads * dk * dv / t1 / 1e12, 2), like_tflops=round(4 * rows * heads * dk * dv / t2 / 1e12, 2))
+        gl, gb, wv = torch.randn(rows, heads * dv, device=dev), rnd(rows, heads * dv), rnd(dv)
+        ob = torch.empty(rows, heads * dv, device=dev, dtype=bf)
+        t1 = timed(lambda: K.delta_gated_norm(oo, gl, wv, ob, stp.token_seq, dv, 1e-6), reps=9, graph=True)
+        t2 = timed(lambda: K.gated_norm(oo, gb, wv, ob, stp.token_seq, dv, False, 1e-6), reps=9, graph=True)
+        pair(f"{what}_read_out", (t1, 0, rows * heads * dv * 10), (t2, 0, rows * heads * dv * 8))
+        # ---- latent attention: a sink a head beside none; the low-rank rows beside Bidinex's rows
+        LH, R, rot = y["heads"], y["kv_rank"], y["rot"]
+        D = R + rot
+        cache, table = paged(n_seqs, length, 1, 1, D)
+        ql, ol, sinks = rnd(rows, LH, D) * 0.3, torch.empty(rows, LH, R, device=dev, dtype=bf), torch.randn(LH, device=dev)
+        sp = max(1, min(296 // K.attn_latent_ctas(R, rot, n_seqs, each, LH), (length // 32) // 4, 32)) if few else 1
+        fl, by = 2 * LH * (D + R) * sum(range(length - each + 1, length + 1)) * n_seqs, n_seqs * length * D * 2
+        lat = lambda **kw: timed(lambda: K.attn_latent_mma(ql, ol, cache, table, stp.q_start, stp.q_len, stp.kv_before, stp.token_seq, n_seqs, each,     # noqa: E731
+                                                           R, None, 0.1, n_splits=sp, **kw), reps=7, graph=True)
+        pair(f"{what}_latent_attention", (lat(sinks=sinks), fl, by), (lat(), fl, by))
+        QR, qc = y["q_rank"], LH * (y["dim"] + rot)
+        proj, cq, wq, wc, inv = rnd(rows, QR + D), torch.empty(rows, QR, device=dev, dtype=bf), rnd(QR), rnd(R), torch.rand(rot // 2, device=dev)
+        t1 = timed(lambda: K.latent_down(proj, QR, cq, wq, wc, inv, stp.positions, stp.token_seq, table, cache, rot, R, rot, PAGE_SIZE, 1e-6),
+                   reps=9, graph=True)
+        full = rnd(rows, qc + D)
+        t2 = timed(lambda: K.latent_prep(full, qc, wc, inv, stp.positions, stp.token_seq, table, cache, ql, LH, y["dim"], rot, R, rot, PAGE_SIZE, 1e-6),
+                   reps=9, graph=True)
+        pair(f"{what}_latent_rows", (t1, 0, rows * (QR + D) * 4), (t2, 0, rows * (D + LH * rot) * 4))
+    K.check_device_errors()
+    return res
+
+
 def run_reference(args):
     print(json.dumps({"impl": "reference", "unavailable":
                       "mcelrath/braidinfer is Rust + HIP for AMD RDNA3: pip finds neither setup.py nor pyproject.toml, "
@@ -1888,7 +2129,10 @@ def main() -> int:
     ap.add_argument("--zisesun", action="store_true",
                     help="another measurement: the Zisesun decoder at sizes like a real model's layers beside the Birepel "
                          "decoder of equal size, and its kernels one by one; prints its own line (see run_zisesun)")
-    ap.add_argument("--sizes", default="", help="with --bidinex / --loduzen / --birepel / --ludazen / --zisesun: names of the sizes, with commas (default: all)")
+    ap.add_argument("--megerax", action="store_true",
+                    help="another measurement: the Megerax decoder at sizes like a real model's layers beside the Loduzen "
+                         "decoder of equal size, and its kernels one by one; prints its own line (see run_megerax)")
+    ap.add_argument("--sizes", default="", help="with --bidinex / --loduzen / --birepel / --ludazen / --zisesun / --megerax: names of the sizes, with commas (default: all)")
     ap.add_argument("--prompt-len", type=int, default=2048, help="with --bidinex: tokens of the timed prompt")
     ap.add_argument("--context", type=int, default=2048, help="with --bidinex: context of the timed decode steps")
     args = ap.parse_args()
@@ -1907,6 +2151,8 @@ def main() -> int:
         return run_ludazen(args)
     if args.zisesun:
         return run_zisesun(args)
+    if args.megerax:
+        return run_megerax(args)
     if args.sweep:
         return run_sweep(args)
     if args.prompt_timeline:

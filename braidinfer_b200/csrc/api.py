@@ -723,7 +723,7 @@ class Kernels:
                                                 [c_int] * 7 + [c_void_p, c_longlong, c_void_p]
                 lib.braid_delta_gated_norm.argtypes = [c_void_p, c_void_p, c_longlong, c_void_p, c_int, c_void_p, c_longlong,
                                                        c_void_p] + [c_int] * 4 + [c_float, c_void_p]
-                lib.braid_delta_work_floats.argtypes = [c_int] * 6
+                lib.braid_delta_work_floats.argtypes = [c_int] * 5
                 lib.braid_delta_work_floats.restype = c_longlong
                 names = ("braid_delta_rule", "braid_delta_gated_norm")
             elif name == "streams":
@@ -1181,7 +1181,7 @@ class Kernels:
                 or bias.numel() != heads * dk or rate.numel() != heads or b.shape[1] < heads or out.shape[1] != heads * dv:
             raise KernelError("delta_rule: the rows do not hold the heads")
         rows = out.shape[0]
-        need = lib.braid_delta_work_floats(rows, ctx.n_seqs, int(ctx.max_q_len), heads, dk, dv) if chunked else 0
+        need = lib.braid_delta_work_floats(rows, ctx.n_seqs, heads, dk, dv) if chunked else 0
         work = torch.empty(need, dtype=torch.float32, device=out.device) if need > 0 else None
         self.launches += 3 if work is not None else 1
         self._check_lib(lib, lib.braid_delta_rule(

@@ -43,17 +43,16 @@ struct ConvHeadsArgs {
     const float* inv_freq;       // [rope_dim / 2]
     int rope_dim, adjacent;
     float amp, eps;
-    int rows, channels, taps, n_segs;
+    int rows, channels, taps, n_segs, turns;     // turns: some segment is rotated
     int* error_flag;
     ConvSegment seg[CONV_MAX_SEGS];
 };
 
 // Where head `h` of segment s and row `row` is stored (its first number), or null.
 template <typename T, typename TO>
-__device__ __forceinline__ TO* conv_dst(const ConvHeadsArgs& a, const ConvSegment& s, int h, int row, int seq, bool flag) {
+__device__ __forceinline__ TO* conv_dst(const ConvHeadsArgs& a, const ConvSegment& s, int h, int row, int seq, int pos, bool flag) {
     if (s.plane < 0) return (TO*)s.out + (size_t)row * s.out_stride + (size_t)h * s.pad;
     if (!a.cache) return nullptr;
-    const int pos = a.positions[row];
     const int block = pos / a.page_size, off = pos - block * a.page_size;
     const int page = (block < a.table_cols) ? a.page_table[(size_t)seq * a.table_cols + block] : -1;
     if (page < 0 || page >= a.num_pages) {
@@ -64,25 +63,57 @@ __device__ __forceinline__ TO* conv_dst(const ConvHeadsArgs& a, const ConvSegmen
 }
 
 // 16 bytes of neighbouring channels a thread, LPH lanes a head, RPT neighbouring rows a thread: for sizes, strides and taps
-// that allow it (neighbouring pairs in the rotation).  TO: the type of what is stored.
+// that allow it (neighbouring pairs in the rotation).  TO: the type of what is stored.  What the rows' tables say is asked for
+// in rounds over all RPT rows (one trip a round instead of one a row), and the CTA's heads share the sines and cosines.
+#define CONV_MAX_PAIRS 128
 template <typename T, typename TO, int TAPS, int LPH, int RPT>
-__global__ void __launch_bounds__(128)
+__global__ void __launch_bounds__(128, RPT > 1 ? 4 : 6)
 conv_heads_vec_kernel(ConvHeadsArgs a) {
     constexpr int VEC = 16 / sizeof(T), HPC = 128 / LPH, SPAN = RPT + TAPS - 1;
+    __shared__ float2 turn[RPT][CONV_MAX_PAIRS];           // (sine, cosine) of the rows' angles
     pdl_trigger();
     const int sub = threadIdx.x / LPH, l = threadIdx.x % LPH, i0 = l * VEC;
-    // which segment and head: the CTAs of a row walk the segments' groups of HPC heads
-    int g = blockIdx.x, si = 0, c_seg = 0;
-    for (; si < a.n_segs - 1; ++si) {
-        const int groups = (a.seg[si].heads + HPC - 1) / HPC;
-        if (g < groups) break;
-        g -= groups;
-        c_seg += a.seg[si].heads * a.seg[si].size;
-    }
-    const ConvSegment& s = a.seg[si];
-    const int head = g * HPC + sub;
+    // which segment and head: the segments' heads are counted through
+    int head = blockIdx.x * HPC + sub, c_seg = 0;
+    ConvSegment s = a.seg[0];
+#pragma unroll
+    for (int si = 1; si < CONV_MAX_SEGS; ++si)
+        if (si < a.n_segs && head >= s.heads) {
+            head -= s.heads;
+            c_seg += s.heads * s.size;
+            s = a.seg[si];
+        }
     const bool live = head < s.heads, in = live && i0 < s.size;
     const int c0 = c_seg + head * s.size + i0;
+    const int row0 = blockIdx.y * RPT;
+    // the step's tables are on the device before its first kernel: read before the wait
+    int seq[RPT], pos[RPT], o[RPT], slot[RPT], qlen[RPT];
+#pragma unroll
+    for (int r = 0; r < RPT; ++r) {
+        seq[r] = row0 + r < a.rows ? a.token_seq[row0 + r] : -1;
+        pos[r] = row0 + r < a.rows ? a.positions[row0 + r] : 0;
+    }
+#pragma unroll
+    for (int r = 0; r < RPT; ++r) {
+        const int q = max(seq[r], 0);
+        o[r] = row0 + r - a.q_start[q];
+        qlen[r] = a.q_len[q];
+        slot[r] = a.slot_ids[q];
+    }
+    TO* dst[RPT];
+#pragma unroll
+    for (int r = 0; r < RPT; ++r) dst[r] = live && seq[r] >= 0 ? conv_dst<T, TO>(a, s, head, row0 + r, seq[r], pos[r], l == 0) : nullptr;
+    if (a.turns) {
+        const int half = a.rope_dim / 2;
+        for (int idx = threadIdx.x; idx < RPT * half; idx += 128) {
+            const int r = idx / half, p = idx - r * half;
+            const int ps = row0 + r < a.rows ? a.positions[row0 + r] : 0;
+            float sn, cs;
+            sincosf((float)ps * a.inv_freq[p], &sn, &cs);
+            turn[r][p] = make_float2(sn * a.amp, cs * a.amp);
+        }
+        __syncthreads();
+    }
     float wl[VEC * TAPS], bl[VEC];
 #pragma unroll
     for (int e = 0; e < VEC; ++e) bl[e] = 0.f;
@@ -92,100 +123,120 @@ conv_heads_vec_kernel(ConvHeadsArgs a) {
         if (a.bias) load_run<T, VEC>((const T*)a.bias + c0, bl);
     }
     pdl_wait();
-    const int row0 = blockIdx.y * RPT;
-    float xin[SPAN][VEC];
+    __align__(16) T xin[SPAN][VEC];                        // as they came: the bias is added where a row is used
 #pragma unroll
     for (int u = 0; u < SPAN; ++u) {
         const int r = row0 - (TAPS - 1) + u;
-        if (in && r >= 0 && r < a.rows) {
-            load_run<T, VEC>((const T*)a.x + (size_t)r * a.x_stride + c0, xin[u]);
-#pragma unroll
-            for (int e = 0; e < VEC; ++e) xin[u][e] += bl[e];
-        } else {
-#pragma unroll
-            for (int e = 0; e < VEC; ++e) xin[u][e] = 0.f;
-        }
+        if (in && r >= 0 && r < a.rows) *reinterpret_cast<uint4*>(xin[u]) = *reinterpret_cast<const uint4*>((const T*)a.x + (size_t)r * a.x_stride + c0);
+        else *reinterpret_cast<uint4*>(xin[u]) = make_uint4(0, 0, 0, 0);
     }
-    float nw[VEC];
-    if (in && s.norm == CONV_NORM_RMS) load_run<T, VEC>((const T*)s.weight + i0, nw);
-#pragma unroll
-    for (int rr = 0; rr < RPT; ++rr) {
-        const int row = row0 + rr;
-        if (row >= a.rows) break;                          // the whole CTA: rows are the grid's
-        const int seq = a.token_seq[row];
-        if (seq < 0) continue;
-        const int o = row - a.q_start[seq];
-        float* st = a.state ? (float*)(a.state + (size_t)a.slot_ids[seq] * a.state_stride + a.state_offset) : nullptr;
-        float y[VEC];
-#pragma unroll
-        for (int e = 0; e < VEC; ++e) y[e] = 0.f;
-        if (in) {
-            float old[TAPS > 1 ? TAPS - 1 : 1][VEC];       // rows before the step that this row's taps reach
-#pragma unroll
-            for (int j = 0; j < TAPS; ++j) {
-                const int back = TAPS - 1 - j;
-                float xv[VEC];
-                if (o - back >= 0) {
-#pragma unroll
-                    for (int e = 0; e < VEC; ++e) xv[e] = xin[rr + j][e];
-                } else {
-                    const float* sp = st + (size_t)(TAPS - 1 + (o - back)) * a.channels + c0;
-#pragma unroll
-                    for (int e = 0; e < VEC; e += 4) load_run<float, 4>(sp + e, xv + e);
-                }
-                if (j < TAPS - 1) {
-#pragma unroll
-                    for (int e = 0; e < VEC; ++e) old[j][e] = xv[e];
-                }
-#pragma unroll
-                for (int e = 0; e < VEC; ++e) y[e] = fmaf(wl[e * TAPS + j], xv[e], y[e]);
-            }
-            if (TAPS > 1 && a.q_len[seq] == 1) {           // one token: nobody else reads these channels of the state
-#pragma unroll
-                for (int j = 0; j < TAPS - 1; ++j)
-#pragma unroll
-                    for (int e = 0; e < VEC; e += 4)
-                        store_run<float, 4>(st + (size_t)j * a.channels + c0 + e, (j < TAPS - 2 ? old[j + 1 < TAPS - 1 ? j + 1 : j] : xin[rr + TAPS - 1]) + e);
-            }
-        }
+    // silu, norm, rotation and store of one row's channels; the whole warp calls
+    auto finish = [&](int rr, float* y) {
         if (s.silu) {
 #pragma unroll
             for (int e = 0; e < VEC; ++e) y[e] = sizeof(T) == 2 ? glu_act_fast(y[e], BRAID_ACT_SILU) : silu_f32(y[e]);
         }
+        float ss = 0.f;
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) ss = fmaf(y[e], y[e], ss);
+#pragma unroll
+        for (int b = LPH / 2; b > 0; b >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, b);       // whatever the lanes' segments
         if (s.norm != CONV_NORM_NONE) {
-            float ss = 0.f;
-#pragma unroll
-            for (int e = 0; e < VEC; ++e) ss = fmaf(y[e], y[e], ss);
-#pragma unroll
-            for (int b = LPH / 2; b > 0; b >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, b);
             const float r = s.factor / sqrtf((s.norm == CONV_NORM_RMS ? ss / (float)s.size : ss) + a.eps);
 #pragma unroll
-            for (int e = 0; e < VEC; ++e) y[e] *= s.norm == CONV_NORM_RMS && in ? r * nw[e] : r;
-        } else {
+            for (int e = 0; e < VEC; ++e) y[e] *= r;
+            if (in && s.norm == CONV_NORM_RMS) {
+                float nw[VEC];
+                load_run<T, VEC>((const T*)s.weight + i0, nw);
+#pragma unroll
+                for (int e = 0; e < VEC; ++e) y[e] *= nw[e];
+            }
+        } else if (s.factor != 1.f) {
 #pragma unroll
             for (int e = 0; e < VEC; ++e) y[e] *= s.factor;
         }
-        if (!live || i0 >= s.pad) continue;
+        if (!dst[rr] || i0 >= s.pad) return;
         if (s.rotate && i0 < a.rope_dim) {
-            const float pos = (float)a.positions[row];
 #pragma unroll
             for (int e = 0; e < VEC; e += 2) {
                 const int p = (i0 + e) >> 1;
                 if (2 * p < a.rope_dim) {
-                    float sn, cs;
-                    sincosf(pos * a.inv_freq[p], &sn, &cs);
-                    sn *= a.amp; cs *= a.amp;
+                    const float2 t = turn[rr][p];
                     const float u = y[e], v = y[e + 1];
-                    y[e] = u * cs - v * sn;
-                    y[e + 1] = v * cs + u * sn;
+                    y[e] = u * t.y - v * t.x;
+                    y[e + 1] = v * t.y + u * t.x;
                 }
             }
         }
-        TO* dst = conv_dst<T, TO>(a, s, head, row, seq, l == 0);
-        if (!dst) continue;
         constexpr int VO = 16 / sizeof(TO) < VEC ? 16 / sizeof(TO) : VEC;
 #pragma unroll
-        for (int e = 0; e < VEC; e += VO) store_run<TO, VO>(dst + i0 + e, y + e);
+        for (int e = 0; e < VEC; e += VO) store_run<TO, VO>(dst[rr] + i0 + e, y + e);
+    };
+    if (RPT > 1 && seq[0] >= 0 && seq[0] == seq[RPT - 1] && o[0] >= TAPS - 1) {
+        // all rows and what their taps reach lie inside one sequence's step: every row is converted once, the bias comes
+        // through the sum of the taps
+        float win[TAPS][VEC], yb[VEC];
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) {
+            float sum = 0.f;
+#pragma unroll
+            for (int j = 0; j < TAPS; ++j) sum += wl[e * TAPS + j];
+            yb[e] = sum * bl[e];
+        }
+#pragma unroll
+        for (int u = 0; u < SPAN; ++u) {
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) win[u % TAPS][e] = to_f32(xin[u][e]);
+            if (u < TAPS - 1) continue;
+            float y[VEC];
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) {
+                y[e] = yb[e];
+#pragma unroll
+                for (int j = 0; j < TAPS; ++j) y[e] = fmaf(wl[e * TAPS + j], win[(u + 1 + j) % TAPS][e], y[e]);
+            }
+            finish(u - (TAPS - 1), y);
+        }
+        return;
+    }
+#pragma unroll
+    for (int rr = 0; rr < RPT; ++rr) {
+        if (seq[rr] < 0) continue;                         // the whole CTA: rows are the grid's
+        float* st = a.state ? (float*)(a.state + (size_t)slot[rr] * a.state_stride + a.state_offset) : nullptr;
+        float y[VEC];
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) y[e] = 0.f;
+        if (in) {
+            const bool alone = RPT == 1 && TAPS > 1 && qlen[rr] == 1;
+            float old[RPT == 1 && TAPS > 1 ? TAPS - 1 : 1][VEC];       // rows before the step that this row's taps reach
+#pragma unroll
+            for (int j = 0; j < TAPS; ++j) {
+                const int back = TAPS - 1 - j;
+                float xv[VEC];
+                if (o[rr] - back >= 0) {
+#pragma unroll
+                    for (int e = 0; e < VEC; ++e) xv[e] = to_f32(xin[rr + j][e]) + bl[e];
+                } else {
+                    const float* sp = st + (size_t)(TAPS - 1 + (o[rr] - back)) * a.channels + c0;
+#pragma unroll
+                    for (int e = 0; e < VEC; e += 4) load_run<float, 4>(sp + e, xv + e);
+                }
+                if (RPT == 1 && j < TAPS - 1) {
+#pragma unroll
+                    for (int e = 0; e < VEC; ++e) old[RPT == 1 ? j : 0][e] = xv[e];
+                }
+#pragma unroll
+                for (int e = 0; e < VEC; ++e) y[e] = fmaf(wl[e * TAPS + j], xv[e], y[e]);
+                if (alone && j == TAPS - 1) {              // one token: nobody else reads these channels of the state
+#pragma unroll
+                    for (int k = 0; k < TAPS - 1; ++k)
+#pragma unroll
+                        for (int e = 0; e < VEC; e += 4)
+                            store_run<float, 4>(st + (size_t)k * a.channels + c0 + e, (k < TAPS - 2 ? old[RPT == 1 && k < TAPS - 2 ? k + 1 : 0] : xv) + e);
+                }
+            }
+        }
+        finish(rr, y);
     }
 }
 
@@ -251,22 +302,22 @@ conv_heads_kernel(ConvHeadsArgs a) {
         }
         __syncwarp();
     }
-    TO* dst = conv_dst<T, TO>(a, s, h, row, seq, lane == 0);
+    TO* dst = conv_dst<T, TO>(a, s, h, row, seq, a.positions[row], lane == 0);
     if (!dst) return;
     for (int i = lane; i < s.pad; i += 32) dst[i] = from_f32<TO>(i < s.size ? y[i] : 0.f);
 }
 
-// The state after the step of every sequence that brings more than one token: its last taps - 1 rows.  One thread per
+// The state after the step of every sequence that brings at least `from` tokens: its last taps - 1 rows.  One thread per
 // (sequence, channel) reads what it needs of the old state before it writes, in rising order.
 template <typename T>
 __global__ void __launch_bounds__(256)
-conv_heads_state_kernel(ConvHeadsArgs a, int n_seqs) {
+conv_heads_state_kernel(ConvHeadsArgs a, int n_seqs, int from) {
     pdl_trigger();
     pdl_wait();
     const int c = blockIdx.x * blockDim.x + threadIdx.x, seq = blockIdx.y;
     if (c >= a.channels || seq >= n_seqs) return;
     const int n = a.q_len[seq], r0 = a.q_start[seq], keep = a.taps - 1;
-    if (n <= 1) return;
+    if (n < from) return;
     const float b = a.bias ? to_f32(((const T*)a.bias)[c]) : 0.f;
     float* st = (float*)(a.state + (size_t)a.slot_ids[seq] * a.state_stride + a.state_offset);
     for (int i = 0; i < keep; ++i) {
@@ -276,37 +327,41 @@ conv_heads_state_kernel(ConvHeadsArgs a, int n_seqs) {
     }
 }
 
+// Returns the tokens from which on a sequence's state is still to be moved on.
 template <typename T, typename TO, int TAPS, int LPH>
-static void launch_conv_vec(const ConvHeadsArgs& a, cudaStream_t s) {
+static int launch_conv_vec(const ConvHeadsArgs& a, cudaStream_t s) {
     constexpr int HPC = 128 / LPH;
-    int groups = 0;
-    for (int i = 0; i < a.n_segs; ++i) groups += (a.seg[i].heads + HPC - 1) / HPC;
+    int heads = 0;
+    for (int i = 0; i < a.n_segs; ++i) heads += a.seg[i].heads;
+    const int groups = (heads + HPC - 1) / HPC;
     // neighbouring rows a thread: four where the rows alone fill the machine
-    if ((long long)a.rows * groups >= 148 * 16)
+    if ((long long)a.rows * groups >= 148 * 16) {
         braid_launch(conv_heads_vec_kernel<T, TO, TAPS, LPH, 4>, dim3(groups, (a.rows + 3) / 4), dim3(128), 0, s, a);
-    else
-        braid_launch(conv_heads_vec_kernel<T, TO, TAPS, LPH, 1>, dim3(groups, a.rows), dim3(128), 0, s, a);
+        return 1;
+    }
+    braid_launch(conv_heads_vec_kernel<T, TO, TAPS, LPH, 1>, dim3(groups, a.rows), dim3(128), 0, s, a);
+    return 2;
 }
 
 template <typename T, typename TO>
-static void launch_conv(const ConvHeadsArgs& a, bool wide, int lanes, cudaStream_t s) {
+static int launch_conv(const ConvHeadsArgs& a, bool wide, int lanes, cudaStream_t s) {
     if (wide) {
 #define CONV_LPH(TAPS)                                                        \
     do {                                                                      \
-        if (lanes <= 4) launch_conv_vec<T, TO, TAPS, 4>(a, s);                \
-        else if (lanes <= 8) launch_conv_vec<T, TO, TAPS, 8>(a, s);           \
-        else if (lanes <= 16) launch_conv_vec<T, TO, TAPS, 16>(a, s);         \
-        else launch_conv_vec<T, TO, TAPS, 32>(a, s);                          \
+        if (lanes <= 4) return launch_conv_vec<T, TO, TAPS, 4>(a, s);                \
+        if (lanes <= 8) return launch_conv_vec<T, TO, TAPS, 8>(a, s);           \
+        if (lanes <= 16) return launch_conv_vec<T, TO, TAPS, 16>(a, s);         \
+        return launch_conv_vec<T, TO, TAPS, 32>(a, s);                          \
     } while (0)
         if (a.taps == 2) CONV_LPH(2);
         else if (a.taps == 3) CONV_LPH(3);
         else CONV_LPH(4);
 #undef CONV_LPH
-        return;
     }
     int heads = 0;
     for (int i = 0; i < a.n_segs; ++i) heads += a.seg[i].heads;
     braid_launch(conv_heads_kernel<T, TO>, dim3((heads + CONV_ANY_WARPS - 1) / CONV_ANY_WARPS, a.rows), dim3(CONV_ANY_WARPS * 32), 0, s, a);
+    return 2;
 }
 
 // `segs`: n_segs records of 7 ints {heads, size, pad, norm, silu, rotate, plane}; factors, weights, outs, out_strides: one
@@ -327,12 +382,12 @@ extern "C" int braid_conv_heads(const void* x, long long x_stride, const void* b
     if (rope_dim < 0 || (rope_dim & 1)) BRAID_REFUSE("conv_heads: rope_dim=%d must be even", rope_dim);
     ConvHeadsArgs a{x, x_stride, bias, w, (uint8_t*)(taps > 1 ? state : nullptr), state_stride, state_offset, token_seq, positions,
                     q_start, q_len, slot_ids, page_table, cache, page_size, table_cols, num_pages, inv_freq, rope_dim, adjacent,
-                    amp, eps, rows, 0, taps, n_segs, error_flag, {}};
+                    amp, eps, rows, 0, taps, n_segs, 0, error_flag, {}};
     const int vec = dtype == BRAID_F32 ? 4 : 8;
     bool wide = taps >= 2 && taps <= 4 && x_stride % vec == 0 && state_stride % 16 == 0 && state_offset % 16 == 0 &&
                 (((uintptr_t)x | (uintptr_t)bias | (uintptr_t)w | (uintptr_t)cache | (uintptr_t)state) & 15) == 0 && rows <= 65535;
     int widest = 0;
-    for (int i = 0; i < n_segs; ++i) {
+    for (int i = 0; i < n_segs; ++i) {                      // (inv_freq is read only where something turns)
         const int* g = segs + 7 * i;
         a.seg[i] = ConvSegment{g[0], g[1], g[2], g[3], g[4], g[5], g[6], factors[i], weights[i], outs[i], out_strides[i]};
         const ConvSegment& s = a.seg[i];
@@ -343,21 +398,37 @@ extern "C" int braid_conv_heads(const void* x, long long x_stride, const void* b
             BRAID_REFUSE("conv_heads: a segment goes to a buffer, or to a cache with pages in the run's type");
         if (s.plane > 1) BRAID_REFUSE("conv_heads: the cache has a key plane (0) and a value plane (1)");
         a.channels += s.heads * s.size;
+        if (s.rotate && rope_dim > 0) a.turns = 1;
         if (s.pad > widest) widest = s.pad;
         wide = wide && s.size % vec == 0 && s.pad % vec == 0 && (!s.rotate || adjacent || rope_dim == 0) &&
                (((uintptr_t)s.weight | (uintptr_t)s.out) & 15) == 0 && (s.plane >= 0 || s.out_stride % vec == 0);
     }
+    // heads of channels that nothing ties together are cut to the size of the others, so that no lane of those is idle
+    int tied = 0;
+    auto loose = [](const ConvSegment& s) { return s.norm == CONV_NORM_NONE && !s.rotate && s.plane < 0 && s.pad == s.size; };
+    for (int i = 0; i < n_segs; ++i)
+        if (!loose(a.seg[i]) && a.seg[i].pad > tied) tied = a.seg[i].pad;
+    if (tied > 0 && tied % vec == 0) {
+        widest = tied;
+        for (int i = 0; i < n_segs; ++i) {
+            ConvSegment& s = a.seg[i];
+            if (loose(s) && s.size > tied && s.size % tied == 0) {
+                s.heads *= s.size / tied;
+                s.size = s.pad = tied;
+            } else if (s.pad > widest) widest = s.pad;
+        }
+    }
     const int lanes = (widest + vec - 1) / vec;
-    wide = wide && lanes <= 32;
+    wide = wide && lanes <= 32 && rope_dim <= 2 * CONV_MAX_PAIRS;
     if (rows > 65535 || n_seqs > 65535) BRAID_REFUSE("conv_heads: %d rows exceed one launch", rows);
     cudaStream_t st = (cudaStream_t)stream;
-    if (dtype == BRAID_F32) launch_conv<float, float>(a, wide, lanes, st);
-    else if (out_f32) launch_conv<__nv_bfloat16, float>(a, wide, lanes, st);
-    else launch_conv<__nv_bfloat16, __nv_bfloat16>(a, wide, lanes, st);
-    if (taps > 1 && max_q_len > 1) {
+    const int from = dtype == BRAID_F32 ? launch_conv<float, float>(a, wide, lanes, st)
+                     : out_f32 ? launch_conv<__nv_bfloat16, float>(a, wide, lanes, st)
+                               : launch_conv<__nv_bfloat16, __nv_bfloat16>(a, wide, lanes, st);
+    if (taps > 1 && max_q_len >= from) {
         const dim3 grid((a.channels + 255) / 256, n_seqs);
-        if (dtype == BRAID_F32) braid_launch(conv_heads_state_kernel<float>, grid, dim3(256), 0, st, a, n_seqs);
-        else braid_launch(conv_heads_state_kernel<__nv_bfloat16>, grid, dim3(256), 0, st, a, n_seqs);
+        if (dtype == BRAID_F32) braid_launch(conv_heads_state_kernel<float>, grid, dim3(256), 0, st, a, n_seqs, from);
+        else braid_launch(conv_heads_state_kernel<__nv_bfloat16>, grid, dim3(256), 0, st, a, n_seqs, from);
     }
     BRAID_LAUNCH_CHECK();
 }

@@ -31,7 +31,7 @@
 #define DELTA_C 64                 // tokens a chunk
 #define DELTA_SUB 16               // tokens a sub-chunk
 #define DELTA_NSUB (DELTA_C / DELTA_SUB)
-#define DELTA_DVT 32               // value columns a CTA of the chunk-after-chunk kernel
+#define DELTA_DVT 16               // value columns a CTA of the chunk-after-chunk kernel
 #define DELTA_OUT_COLS 64          // value columns a CTA of the output kernel
 #define DELTA_SPREAD 8.6736174e-19f      // 2^-60
 
@@ -47,11 +47,17 @@ struct DeltaArgs {
     uint8_t* state; long long state_stride, state_offset;
     const int *q_start, *q_len, *slot_ids;
     int heads, groups, dk, dv;
-    // scratch of the chunked form; row-wise buffers are [rows][heads][n]
-    float *w, *u, *qd, *kd, *p;                  // n = dk4, dv4, dk4, dk4, 64
-    float *gc, *sc;                              // [seq][chunk][head][dk4], [seq][chunk][head][dk][dv4]
-    int dk4, dv4, max_chunks;
+    // scratch of the chunked form: blocks a (chunk, head), see delta_block
+    float *w, *u, *qd, *kd, *p;                  // [64][LD], [tiles][64][16], [64][LD], [64][LD], [64][64]
+    float *gc, *sc;                              // [DKP], [tiles][DKP][16]
+    int tiles, max_chunks;                       // tiles of 16 value columns
 };
+
+// The place of chunk c of sequence seq among all chunks of the step: a sequence's chunks lie one after the other, and two
+// sequences' never meet (a sequence of n rows takes ceil(n / 64) places, the next one starts at least so many further on).
+__device__ __forceinline__ size_t delta_block(const DeltaArgs& a, int seq, int c, int h) {
+    return (size_t)(a.q_start[seq] / DELTA_C + seq + c) * a.heads + h;
+}
 
 // a decay from its logit: exp(-rate softplus(x))
 __device__ __forceinline__ float delta_decay(float x, float rate) {
@@ -178,24 +184,21 @@ delta_walk_kernel(DeltaArgs a) {
 
 // ------------------------------------------------------------------ inside every chunk
 #define DELTA_INTRA_THREADS 256
-// A's rows take the place of q's once those have been used, where a row is wide enough
-template <int DKP> constexpr int delta_intra_smem() {
-    return (3 * DELTA_C * (DKP + 4) + (DKP < DELTA_C ? DELTA_C * (DELTA_C + 4) : 0) + DELTA_C + 3 * DKP) * 4;
-}
+template <int DKP> constexpr int delta_intra_smem() { return (3 * DELTA_C * (DKP + 4) + DELTA_C + 3 * DKP) * 4; }
 
 template <typename T, int DKP>
 __global__ void __launch_bounds__(DELTA_INTRA_THREADS, DKP <= 128 ? 2 : 1)
 delta_intra_kernel(DeltaArgs a) {
     constexpr int C = DELTA_C, SUB = DELTA_SUB, LD = DKP + 4, NT = DELTA_INTRA_THREADS;
-    constexpr bool OWN_A = DKP < C;
-    constexpr int LA = OWN_A ? C + 4 : LD;
+    static_assert(DKP >= C, "A's rows fit where q's were");
+    constexpr int LA = LD;
     static_assert(DKP <= NT, "a thread a channel");
     extern __shared__ __align__(16) float sm[];
     float* sK = sm;                          // k, then k over the decays up to it, then k times the decays after it
     float* sQ = sK + C * LD;                 // q, then q times the decays from its sub-chunk's edge
     float* sG = sQ + C * LD;                 // g, then k times the decays from the edge, then from the chunk's start
-    float* sA = OWN_A ? sG + C * LD : sQ;    // beta_t A_ts
-    float* sB = sG + C * LD + (OWN_A ? C * LA : 0);      // beta
+    float* sA = sQ;                          // beta_t A_ts, in the place of q's rows once those have been used
+    float* sB = sG + C * LD;                 // beta
     float* sT = sB + C;                      // the product of a sub-chunk's decays
     float* sE = sT + DKP;                    // the product of all decays before the sub-chunk
     int* steep = (int*)(sE + DKP);           // the channels whose factors cannot be split, their number in n_steep
@@ -208,6 +211,7 @@ delta_intra_kernel(DeltaArgs a) {
     const float rate = a.rate[h];
     if (tid == 0) n_steep = 0;
     pdl_wait();
+#pragma unroll 8
     for (int idx = tid; idx < C * DKP; idx += NT) {
         const int t = idx / DKP, i = idx - t * DKP;
         const size_t row = (size_t)(r0 + t);
@@ -220,7 +224,8 @@ delta_intra_kernel(DeltaArgs a) {
     if (tid < DKP) sE[tid] = 1.f;
     __syncthreads();
     const int ty = tid >> 4, tx = tid & 15;
-    const size_t hrow0 = (size_t)r0 * a.heads + h;                 // + t * heads: index of (row, head)
+    const size_t block = delta_block(a, seq, c, h);
+    float *gP = a.p + block * (C * C), *gQ = a.qd + block * (C * LD), *gK = a.kd + block * (C * LD);
 #pragma unroll 1
     for (int J = 0; J < DELTA_NSUB; ++J) {
         const int row0 = J * SUB, t = row0 + ty;
@@ -301,14 +306,12 @@ delta_intra_kernel(DeltaArgs a) {
             for (int I = 0; I < DELTA_NSUB; ++I)
                 if (I == J) { accA[I] += dA; accP[I] += dP; }
         }
-        if (t < n) {
 #pragma unroll
-            for (int I = 0; I < DELTA_NSUB; ++I)
-                if (I <= J) {
-                    const int s = I * SUB + tx;
-                    a.p[(hrow0 + (size_t)t * a.heads) * C + s] = s <= t ? accP[I] : 0.f;
-                }
-        }
+        for (int I = 0; I < DELTA_NSUB; ++I)
+            if (I <= J) {
+                const int s = I * SUB + tx;
+                gP[t * C + s] = s <= t ? accP[I] : 0.f;
+            }
         __syncthreads();
         // k on to the sub-chunk's end; k and q from the chunk's start (q goes out)
         for (int idx = tid; idx < (J + 1) * SUB * DKP; idx += NT) {
@@ -317,7 +320,7 @@ delta_intra_kernel(DeltaArgs a) {
             else {
                 const float E = sE[i];
                 sG[at] *= E;
-                if (r < n && i < a.dk4) a.qd[(hrow0 + (size_t)r * a.heads) * a.dk4 + i] = sQ[at] * E;
+                gQ[at] = sQ[at] * E;
             }
         }
         if (tid < DKP) {
@@ -338,16 +341,15 @@ delta_intra_kernel(DeltaArgs a) {
             }
         __syncthreads();
     }
-    for (int idx = tid; idx < n * DKP; idx += NT) {
-        const int r = idx / DKP, i = idx - r * DKP;
-        if (i < a.dk4) a.kd[(hrow0 + (size_t)r * a.heads) * a.dk4 + i] = sK[r * LD + i];
+    for (int idx = tid; idx < C * DKP; idx += NT) {
+        const int r = idx / DKP, at = r * LD + idx - r * DKP;
+        gK[at] = sK[at];
     }
-    float* gc = a.gc + ((size_t)(seq * a.max_chunks + c) * a.heads + h) * a.dk4;
-    for (int i = tid; i < a.dk4; i += NT) gc[i] = sE[i];
+    if (tid < DKP) a.gc[block * DKP + tid] = sE[tid];
     // forward substitution: a thread a column, its 64 numbers in registers
-    for (int col = tid; col < a.dk4 + a.dv4; col += NT) {
-        const bool is_w = col < a.dk4;
-        const int vc = col - a.dk4;
+    for (int col = tid; col < DKP + a.tiles * DELTA_DVT; col += NT) {
+        const bool is_w = col < DKP;
+        const int vc = col - DKP;
         float x[C];
 #pragma unroll
         for (int t = 0; t < C; ++t)
@@ -365,167 +367,190 @@ delta_intra_kernel(DeltaArgs a) {
             }
             x[t] = acc;
         }
-        float* dst = is_w ? a.w + hrow0 * a.dk4 + col : a.u + hrow0 * a.dv4 + vc;
-        const size_t step = (size_t)a.heads * (is_w ? a.dk4 : a.dv4);
+        float* dst = is_w ? a.w + block * (C * LD) + col
+                          : a.u + (block * a.tiles + vc / DELTA_DVT) * (C * DELTA_DVT) + vc % DELTA_DVT;
+        const int step = is_w ? LD : DELTA_DVT;
 #pragma unroll
-        for (int t = 0; t < C; ++t)
-            if (t < n) dst[t * step] = x[t];
+        for (int t = 0; t < C; ++t) dst[t * step] = x[t];
     }
 }
 
 // ------------------------------------------------------------------ chunk after chunk
-__device__ __forceinline__ void delta_cp16(void* smem, const void* gmem, bool in) {
-    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"((uint32_t)__cvta_generic_to_shared(smem)), "l"(gmem), "r"(in ? 16 : 0) : "memory");
+__device__ __forceinline__ void delta_cp16(void* smem, const void* gmem) {
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"((uint32_t)__cvta_generic_to_shared(smem)), "l"(gmem) : "memory");
 }
 __device__ __forceinline__ void delta_cp_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
 template <int N> __device__ __forceinline__ void delta_cp_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
+// N floats (a multiple of 4) that lie one after the other, by NT threads
+template <int N, int NT>
+__device__ __forceinline__ void delta_copy(float* dst, const float* src, int tid) {
+#pragma unroll
+    for (int u = 0; u < (N / 4 + NT - 1) / NT; ++u) {
+        const int at = (tid + u * NT) * 4;
+        if ((N / 4) % NT == 0 || at < N) delta_cp16(dst + at, src + at);
+    }
+}
 
+// A CTA owns (head, sequence, 16 value columns) and walks the chunks.  Both products of a chunk, W S [64 x 16] and K^T U
+// [DKP x 16], are cut along their inner dimension over the eight warps, so that a lane's tile is 8 x 4 (a smaller one would be
+// bound by the reads of shared memory); the warps' partial tiles meet in shared memory, where the thread that owns four numbers
+// of U or of S adds them up.
 #define DELTA_STATE_THREADS 256
-template <int DKP> constexpr int delta_state_smem() { return (DKP * (DELTA_DVT + 4) + 2 * DELTA_C * (DKP + 4) + DELTA_C * (DELTA_DVT + 4)) * 4; }
+template <int DKP> constexpr int delta_state_smem() {
+    return (2 * DELTA_C * (DKP + 4) + (DKP + DELTA_C) * DELTA_DVT + 8 * DELTA_C * DELTA_DVT) * 4;
+}
 
 template <int DKP>
-__global__ void __launch_bounds__(DELTA_STATE_THREADS)
+__global__ void __launch_bounds__(DELTA_STATE_THREADS, DKP <= 128 ? 2 : 1)
 delta_state_kernel(DeltaArgs a) {
-    constexpr int C = DELTA_C, LD = DKP + 4, LS = DELTA_DVT + 4, NT = DELTA_STATE_THREADS, RI = DKP / 32;
+    constexpr int C = DELTA_C, LD = DKP + 4, N = DELTA_DVT, NT = DELTA_STATE_THREADS;
+    constexpr int RB = DKP / 64, KS = 8 / RB;             // row blocks of S, and slices of the tokens a row block
+    constexpr int KU = DKP / 8;                            // W's columns a warp
+    static_assert(C * N == 4 * NT, "a thread owns four neighbouring numbers of U, and of every row block of S");
     extern __shared__ __align__(16) float sm[];
-    float* sS = sm;                          // [DKP][LS]
-    float* sW = sS + DKP * LS;               // [C][LD]
-    float* sK = sW + C * LD;
-    float* sU = sK + C * LD;                 // [C][LS]
-    pdl_trigger();
-    const int h = blockIdx.x, seq = blockIdx.y, col0 = blockIdx.z * DELTA_DVT, tid = threadIdx.x;
-    const int n_all = a.q_len[seq], r0 = a.q_start[seq];
+    float* sW = sm;                          // [C][LD]
+    float* sK = sW + C * LD;                 // [C][LD]
+    float* sS = sK + C * LD;                 // [DKP][16]
+    float* sU = sS + DKP * N;                // [C][16]
+    float* sP = sU + C * N;                  // [8 warps][64][16]
+    const int h = blockIdx.x, seq = blockIdx.y, tile = blockIdx.z, tid = threadIdx.x;
+    const int warp = tid >> 5, lr = (tid & 31) >> 2, lc = tid & 3;
+    const int n_all = a.q_len[seq];
     if (n_all <= 0) return;
     const int dk = a.dk, dv = a.dv, n_chunks = (n_all + C - 1) / C;
-    const int ty = tid >> 3, tx = tid & 7;   // 2 rows of U or RI rows of S, and 4 columns
-    const int j0 = col0 + tx * 4;
+    const int own = tid * 4, own_p = own / N, own_c = own % N, j0 = tile * N + own_c;
+    // the rows of S a thread owns: partial tiles hold row lr * 8 + e at place e * 8 + lr
+    const int own_i = (own_p & 7) * 8 + (own_p >> 3);
     float* S_area = (float*)(a.state + (size_t)a.slot_ids[seq] * a.state_stride + a.state_offset) + (size_t)h * dk * dv;
-    float s[RI][4];
+    float s[RB][4];
 #pragma unroll
-    for (int e = 0; e < RI; ++e)
+    for (int b = 0; b < RB; ++b) {
+        const int i = b * 64 + own_i;
 #pragma unroll
-        for (int x = 0; x < 4; ++x) {
-            const int i = ty * RI + e;
-            s[e][x] = (i < dk && j0 + x < dv) ? S_area[(size_t)i * dv + j0 + x] : 0.f;
-            sS[i * LS + tx * 4 + x] = s[e][x];
-        }
-    for (int idx = tid; idx < 2 * C * LD; idx += NT) sW[idx] = 0.f;      // columns that no copy touches stay zero
-    __syncthreads();
-    pdl_wait();
-    const int ch = a.dk4 / 4;
-    auto load = [&](float* dst, const float* src, int c) {
-        const int n = min(C, n_all - c * C);
-        for (int idx = tid; idx < C * ch; idx += NT) {
-            const int t = idx / ch, i = (idx - t * ch) * 4;
-            const bool in = t < n;
-            delta_cp16(dst + t * LD + i, src + ((size_t)(r0 + c * C + (in ? t : 0)) * a.heads + h) * a.dk4 + i, in);
-        }
-    };
-    float4 u0[2];
-    auto load_u = [&](int c) {
-        const int n = min(C, n_all - c * C);
-#pragma unroll
-        for (int r = 0; r < 2; ++r) {
-            const int t = ty * 2 + r;
-            u0[r] = (t < n && j0 < a.dv4) ? *reinterpret_cast<const float4*>(a.u + ((size_t)(r0 + c * C + t) * a.heads + h) * a.dv4 + j0)
-                                          : make_float4(0.f, 0.f, 0.f, 0.f);
-        }
-    };
-    float gn[RI];
-    auto load_g = [&](int c) {
-        const float* gc = a.gc + ((size_t)(seq * a.max_chunks + c) * a.heads + h) * a.dk4;
-#pragma unroll
-        for (int e = 0; e < RI; ++e) gn[e] = ty * RI + e < a.dk4 ? gc[ty * RI + e] : 0.f;
-    };
-    load(sW, a.w, 0);
-    delta_cp_commit();
-    load(sK, a.kd, 0);
-    delta_cp_commit();
-    load_u(0);
-    load_g(0);
-    for (int c = 0; c < n_chunks; ++c) {
-        const int n = min(C, n_all - c * C);
-        // the state that this chunk starts from, for the output kernel
-        float* sc = a.sc + ((size_t)(seq * a.max_chunks + c) * a.heads + h) * dk * a.dv4;
-#pragma unroll
-        for (int e = 0; e < RI; ++e)
-            if (ty * RI + e < dk && j0 < a.dv4)
-                *reinterpret_cast<float4*>(sc + (size_t)(ty * RI + e) * a.dv4 + j0) = make_float4(s[e][0], s[e][1], s[e][2], s[e][3]);
-        delta_cp_wait<1>();
-        __syncthreads();
-        // U = U0 - W S
-        float u[2][4];
-#pragma unroll
-        for (int r = 0; r < 2; ++r) { u[r][0] = u0[r].x; u[r][1] = u0[r].y; u[r][2] = u0[r].z; u[r][3] = u0[r].w; }
-        if (c + 1 < n_chunks) load_u(c + 1);
-        const float* w0 = sW + (ty * 2) * LD;
-#pragma unroll 4
-        for (int i = 0; i < DKP; i += 4) {
-            float wv[2][4], sv[4][4];
-#pragma unroll
-            for (int r = 0; r < 2; ++r) *reinterpret_cast<float4*>(wv[r]) = *reinterpret_cast<const float4*>(w0 + r * LD + i);
-#pragma unroll
-            for (int e = 0; e < 4; ++e) *reinterpret_cast<float4*>(sv[e]) = *reinterpret_cast<const float4*>(sS + (i + e) * LS + tx * 4);
-#pragma unroll
-            for (int e = 0; e < 4; ++e)
-#pragma unroll
-                for (int r = 0; r < 2; ++r)
-#pragma unroll
-                    for (int x = 0; x < 4; ++x) u[r][x] = fmaf(-wv[r][e], sv[e][x], u[r][x]);
-        }
-#pragma unroll
-        for (int r = 0; r < 2; ++r) {
-            const int t = ty * 2 + r;
-            const float4 uv = make_float4(u[r][0], u[r][1], u[r][2], u[r][3]);
-            *reinterpret_cast<float4*>(sU + t * LS + tx * 4) = uv;
-            if (t < n && j0 < a.dv4) *reinterpret_cast<float4*>(a.u + ((size_t)(r0 + c * C + t) * a.heads + h) * a.dv4 + j0) = uv;
-        }
-        __syncthreads();                                   // W has been read, U is there
-        if (c + 1 < n_chunks) load(sW, a.w, c + 1);
-        delta_cp_commit();
-        delta_cp_wait<1>();                                // this chunk's k
-        __syncthreads();
-        // S = diag(D) S + K^T U
-#pragma unroll
-        for (int e = 0; e < RI; ++e)
-#pragma unroll
-            for (int x = 0; x < 4; ++x) s[e][x] *= gn[e];
-        if (c + 1 < n_chunks) load_g(c + 1);
-#pragma unroll 4
-        for (int t = 0; t < C; ++t) {
-            float kv[RI], uv[4];
-            if (RI >= 4) {
-#pragma unroll
-                for (int e = 0; e < RI; e += 4) *reinterpret_cast<float4*>(kv + e) = *reinterpret_cast<const float4*>(sK + t * LD + ty * RI + e);
-            } else {
-#pragma unroll
-                for (int e = 0; e < RI; ++e) kv[e] = sK[t * LD + ty * RI + e];
-            }
-            *reinterpret_cast<float4*>(uv) = *reinterpret_cast<const float4*>(sU + t * LS + tx * 4);
-#pragma unroll
-            for (int e = 0; e < RI; ++e)
-#pragma unroll
-                for (int x = 0; x < 4; ++x) s[e][x] = fmaf(kv[e], uv[x], s[e][x]);
-        }
-#pragma unroll
-        for (int e = 0; e < RI; ++e)
-            *reinterpret_cast<float4*>(sS + (ty * RI + e) * LS + tx * 4) = make_float4(s[e][0], s[e][1], s[e][2], s[e][3]);
-        __syncthreads();                                   // k has been read, the new S is there
-        if (c + 1 < n_chunks) load(sK, a.kd, c + 1);
-        delta_cp_commit();
+        for (int x = 0; x < 4; ++x) s[b][x] = (i < dk && j0 + x < dv) ? S_area[(size_t)i * dv + j0 + x] : 0.f;
+        *reinterpret_cast<float4*>(sS + i * N + own_c) = make_float4(s[b][0], s[b][1], s[b][2], s[b][3]);
     }
+    pdl_wait();
+    const size_t block0 = delta_block(a, seq, 0, h), step = a.heads;      // block of chunk c: block0 + c * step
+    float4 u0;
+    float gn[RB];
+    auto ahead = [&](int c) {                               // what the owners need of chunk c
+        const size_t blk = block0 + c * step;
+        u0 = *reinterpret_cast<const float4*>(a.u + (blk * a.tiles + tile) * (C * N) + own);
+#pragma unroll
+        for (int b = 0; b < RB; ++b) gn[b] = a.gc[blk * DKP + b * 64 + own_i];
+    };
+    delta_copy<C * LD, NT>(sW, a.w + block0 * (C * LD), tid);
+    delta_cp_commit();
+    delta_copy<C * LD, NT>(sK, a.kd + block0 * (C * LD), tid);
+    delta_cp_commit();
+    ahead(0);
+    for (int c = 0; c < n_chunks; ++c) {
+        const size_t blk = block0 + c * step;
+        const bool more = c + 1 < n_chunks;
+        // the state that this chunk starts from, for the output kernel
+        float* sc = a.sc + (blk * a.tiles + tile) * (DKP * N);
+#pragma unroll
+        for (int b = 0; b < RB; ++b)
+            *reinterpret_cast<float4*>(sc + (b * 64 + own_i) * N + own_c) = make_float4(s[b][0], s[b][1], s[b][2], s[b][3]);
+        delta_cp_wait<1>();                                 // this chunk's W
+        __syncthreads();
+        {
+            float acc[8][4];
+#pragma unroll
+            for (int e = 0; e < 8; ++e)
+#pragma unroll
+                for (int x = 0; x < 4; ++x) acc[e][x] = 0.f;
+            const float *w0 = sW + lr * LD + warp * KU, *s0 = sS + warp * KU * N + lc * 4;
+#pragma unroll
+            for (int i = 0; i < KU; i += 4) {
+                float sv[4][4];
+#pragma unroll
+                for (int d = 0; d < 4; ++d) *reinterpret_cast<float4*>(sv[d]) = *reinterpret_cast<const float4*>(s0 + (i + d) * N);
+#pragma unroll
+                for (int e = 0; e < 8; ++e) {
+                    float wv[4];
+                    *reinterpret_cast<float4*>(wv) = *reinterpret_cast<const float4*>(w0 + e * 8 * LD + i);
+#pragma unroll
+                    for (int d = 0; d < 4; ++d)
+#pragma unroll
+                        for (int x = 0; x < 4; ++x) acc[e][x] = fmaf(wv[d], sv[d][x], acc[e][x]);
+                }
+            }
+            float* part = sP + warp * (C * N) + lr * N + lc * 4;
+#pragma unroll
+            for (int e = 0; e < 8; ++e) *reinterpret_cast<float4*>(part + e * 8 * N) = make_float4(acc[e][0], acc[e][1], acc[e][2], acc[e][3]);
+        }
+        __syncthreads();                                    // W and S have been read, the partial tiles are there
+        if (more) delta_copy<C * LD, NT>(sW, a.w + (blk + step) * (C * LD), tid);
+        delta_cp_commit();
+        {
+            float4 u = u0;
+#pragma unroll
+            for (int w = 0; w < 8; ++w) {
+                const float4 q = *reinterpret_cast<const float4*>(sP + w * (C * N) + own);
+                u.x -= q.x; u.y -= q.y; u.z -= q.z; u.w -= q.w;
+            }
+            *reinterpret_cast<float4*>(sU + own) = u;
+            *reinterpret_cast<float4*>(a.u + (blk * a.tiles + tile) * (C * N) + own) = u;
+        }
+#pragma unroll
+        for (int b = 0; b < RB; ++b)
+#pragma unroll
+            for (int x = 0; x < 4; ++x) s[b][x] *= gn[b];
+        if (more) ahead(c + 1);
+        delta_cp_wait<1>();                                 // this chunk's k
+        __syncthreads();
+        {
+            float acc[8][4];
+#pragma unroll
+            for (int e = 0; e < 8; ++e)
+#pragma unroll
+                for (int x = 0; x < 4; ++x) acc[e][x] = 0.f;
+            const int rb = warp % RB, ks = warp / RB;
+            const float *k0 = sK + (ks * (C / KS)) * LD + rb * 64 + lr * 8, *v0 = sU + (ks * (C / KS)) * N + lc * 4;
+#pragma unroll 4
+            for (int t = 0; t < C / KS; ++t) {
+                float kv[8], uv[4];
+                *reinterpret_cast<float4*>(kv) = *reinterpret_cast<const float4*>(k0 + t * LD);
+                *reinterpret_cast<float4*>(kv + 4) = *reinterpret_cast<const float4*>(k0 + t * LD + 4);
+                *reinterpret_cast<float4*>(uv) = *reinterpret_cast<const float4*>(v0 + t * N);
+#pragma unroll
+                for (int e = 0; e < 8; ++e)
+#pragma unroll
+                    for (int x = 0; x < 4; ++x) acc[e][x] = fmaf(kv[e], uv[x], acc[e][x]);
+            }
+            float* part = sP + (rb * KS + ks) * (64 * N) + lr * N + lc * 4;
+#pragma unroll
+            for (int e = 0; e < 8; ++e) *reinterpret_cast<float4*>(part + e * 8 * N) = make_float4(acc[e][0], acc[e][1], acc[e][2], acc[e][3]);
+        }
+        __syncthreads();                                    // k and U have been read, the partial tiles are there
+        if (more) delta_copy<C * LD, NT>(sK, a.kd + (blk + step) * (C * LD), tid);
+        delta_cp_commit();
+#pragma unroll
+        for (int b = 0; b < RB; ++b) {
+#pragma unroll
+            for (int w = 0; w < KS; ++w) {
+                const float4 q = *reinterpret_cast<const float4*>(sP + (b * KS + w) * (64 * N) + own);
+                s[b][0] += q.x; s[b][1] += q.y; s[b][2] += q.z; s[b][3] += q.w;
+            }
+            *reinterpret_cast<float4*>(sS + (b * 64 + own_i) * N + own_c) = make_float4(s[b][0], s[b][1], s[b][2], s[b][3]);
+        }
+    }
+    pdl_trigger();
     delta_cp_wait<0>();
 #pragma unroll
-    for (int e = 0; e < RI; ++e)
+    for (int b = 0; b < RB; ++b)
 #pragma unroll
         for (int x = 0; x < 4; ++x) {
-            const int i = ty * RI + e;
-            if (i < dk && j0 + x < dv) S_area[(size_t)i * dv + j0 + x] = s[e][x];
+            const int i = b * 64 + own_i;
+            if (i < dk && j0 + x < dv) S_area[(size_t)i * dv + j0 + x] = s[b][x];
         }
 }
 
 // ------------------------------------------------------------------ outputs of every chunk
-#define DELTA_OUT_THREADS 256
+// A CTA owns 64 tokens x 64 value columns of one (chunk, head); a lane's tile is 8 x 4.
+#define DELTA_OUT_THREADS 128
 template <int DKP> constexpr int delta_out_smem() {
     return (DELTA_C * (DKP + 4) + DKP * (DELTA_OUT_COLS + 4) + DELTA_C * (DELTA_C + 4) + DELTA_C * (DELTA_OUT_COLS + 4)) * 4;
 }
@@ -533,72 +558,79 @@ template <int DKP> constexpr int delta_out_smem() {
 template <int DKP>
 __global__ void __launch_bounds__(DELTA_OUT_THREADS)
 delta_out_kernel(DeltaArgs a) {
-    constexpr int C = DELTA_C, LD = DKP + 4, LS = DELTA_OUT_COLS + 4, LP = C + 4, NT = DELTA_OUT_THREADS;
+    constexpr int C = DELTA_C, LD = DKP + 4, LS = DELTA_OUT_COLS + 4, LP = C + 4, NT = DELTA_OUT_THREADS, N = DELTA_DVT;
     extern __shared__ __align__(16) float sm[];
     float* sQ = sm;                          // [C][LD]
     float* sS = sQ + C * LD;                 // [DKP][LS]
     float* sP = sS + DKP * LS;               // [C][LP]
     float* sU = sP + C * LP;                 // [C][LS]
     pdl_trigger();
-    const int tiles = (a.dv4 + DELTA_OUT_COLS - 1) / DELTA_OUT_COLS;
-    const int h = blockIdx.x, seq = blockIdx.y, c = blockIdx.z / tiles, col0 = (blockIdx.z - c * tiles) * DELTA_OUT_COLS, tid = threadIdx.x;
+    const int spans = (a.tiles * N + DELTA_OUT_COLS - 1) / DELTA_OUT_COLS;
+    const int h = blockIdx.x, seq = blockIdx.y, c = blockIdx.z / spans, col0 = (blockIdx.z - c * spans) * DELTA_OUT_COLS, tid = threadIdx.x;
     const int n = min(C, a.q_len[seq] - c * C), r0 = a.q_start[seq] + c * C;
     if (n <= 0) return;
-    const int dk = a.dk;
-    const size_t hrow0 = (size_t)r0 * a.heads + h;
+    const size_t block = delta_block(a, seq, c, h);
+    const int tile0 = col0 / N, tiles = min(DELTA_OUT_COLS / N, a.tiles - tile0);
     pdl_wait();
-    for (int idx = tid; idx < C * (DKP / 4); idx += NT) {
-        const int t = idx / (DKP / 4), i = (idx - t * (DKP / 4)) * 4;
-        const bool in = t < n && i < a.dk4;
-        delta_cp16(sQ + t * LD + i, in ? a.qd + (hrow0 + (size_t)t * a.heads) * a.dk4 + i : a.qd, in);
-    }
-    const float* sc = a.sc + ((size_t)(seq * a.max_chunks + c) * a.heads + h) * dk * a.dv4;
-    constexpr int CQ = DELTA_OUT_COLS / 4;
-    for (int idx = tid; idx < DKP * CQ; idx += NT) {
-        const int i = idx / CQ, j = col0 + (idx - i * CQ) * 4;
-        const bool in = i < dk && j < a.dv4;
-        delta_cp16(sS + i * LS + j - col0, in ? sc + (size_t)i * a.dv4 + j : a.sc, in);
+    delta_copy<C * LD, NT>(sQ, a.qd + block * (C * LD), tid);
+    const float *sc = a.sc + (block * a.tiles + tile0) * (DKP * N), *gu = a.u + (block * a.tiles + tile0) * (C * N), *gp = a.p + block * (C * C);
+    for (int w = 0; w < tiles; ++w) {
+#pragma unroll 4
+        for (int idx = tid; idx < DKP * (N / 4); idx += NT) delta_cp16(sS + (idx / (N / 4)) * LS + w * N + (idx % (N / 4)) * 4, sc + w * (DKP * N) + idx * 4);
+#pragma unroll
+        for (int idx = tid; idx < C * (N / 4); idx += NT) delta_cp16(sU + (idx / (N / 4)) * LS + w * N + (idx % (N / 4)) * 4, gu + w * (C * N) + idx * 4);
     }
     for (int idx = tid; idx < C * (C / 4); idx += NT) {
-        const int t = idx / (C / 4), s = (idx - t * (C / 4)) * 4;
-        const bool in = t < n && s / DELTA_SUB <= t / DELTA_SUB;       // the blocks beyond were not written
-        delta_cp16(sP + t * LP + s, in ? a.p + (hrow0 + (size_t)t * a.heads) * C + s : a.p, in);
-    }
-    for (int idx = tid; idx < C * CQ; idx += NT) {
-        const int t = idx / CQ, j = col0 + (idx - t * CQ) * 4;
-        const bool in = t < n && j < a.dv4;
-        delta_cp16(sU + t * LS + j - col0, in ? a.u + (hrow0 + (size_t)t * a.heads) * a.dv4 + j : a.u, in);
+        const int t = idx / (C / 4), s = (idx % (C / 4)) * 4;
+        if (s / DELTA_SUB <= t / DELTA_SUB) delta_cp16(sP + t * LP + s, gp + idx * 4);       // the blocks beyond were not written
     }
     delta_cp_commit();
     delta_cp_wait<0>();
     __syncthreads();
-    const int ty = tid >> 4, tx = tid & 15;
-    float o[4][4];
+    const int ty = tid >> 4, tx = tid & 15;                // rows r * 8 + ty, columns tx * 4 ...
+    float o[8][4];
 #pragma unroll
-    for (int r = 0; r < 4; ++r)
+    for (int r = 0; r < 8; ++r)
 #pragma unroll
         for (int x = 0; x < 4; ++x) o[r][x] = 0.f;
-    auto product = [&](const float* m, int ld, const float* rhs, int kk) {
+    if (tx * 4 < tiles * N) {
 #pragma unroll 2
-        for (int i = 0; i < kk; i += 4) {
-            float mv[4][4], sv[4][4];
+        for (int i = 0; i < DKP; i += 4) {
+            float sv[4][4];
 #pragma unroll
-            for (int r = 0; r < 4; ++r) *reinterpret_cast<float4*>(mv[r]) = *reinterpret_cast<const float4*>(m + (ty * 4 + r) * ld + i);
+            for (int e = 0; e < 4; ++e) *reinterpret_cast<float4*>(sv[e]) = *reinterpret_cast<const float4*>(sS + (i + e) * LS + tx * 4);
 #pragma unroll
-            for (int e = 0; e < 4; ++e) *reinterpret_cast<float4*>(sv[e]) = *reinterpret_cast<const float4*>(rhs + (i + e) * LS + tx * 4);
+            for (int r = 0; r < 8; ++r) {
+                float mv[4];
+                *reinterpret_cast<float4*>(mv) = *reinterpret_cast<const float4*>(sQ + (r * 8 + ty) * LD + i);
 #pragma unroll
-            for (int e = 0; e < 4; ++e)
+                for (int e = 0; e < 4; ++e)
 #pragma unroll
-                for (int r = 0; r < 4; ++r)
-#pragma unroll
-                    for (int x = 0; x < 4; ++x) o[r][x] = fmaf(mv[r][e], sv[e][x], o[r][x]);
+                    for (int x = 0; x < 4; ++x) o[r][x] = fmaf(mv[e], sv[e][x], o[r][x]);
+            }
         }
-    };
-    product(sQ, LD, sS, DKP);
-    product(sP, LP, sU, ty * 4 + 4);                       // P is lower triangular
+        // P is lower triangular: 16 keys at a time, the rows of earlier sub-chunks stay out
 #pragma unroll
-    for (int r = 0; r < 4; ++r) {
-        const int t = ty * 4 + r;
+        for (int I = 0; I < DELTA_NSUB; ++I)
+#pragma unroll 2
+            for (int s = I * DELTA_SUB; s < (I + 1) * DELTA_SUB; s += 4) {
+                float uv[4][4];
+#pragma unroll
+                for (int e = 0; e < 4; ++e) *reinterpret_cast<float4*>(uv[e]) = *reinterpret_cast<const float4*>(sU + (s + e) * LS + tx * 4);
+#pragma unroll
+                for (int r = 2 * I; r < 8; ++r) {
+                    float mv[4];
+                    *reinterpret_cast<float4*>(mv) = *reinterpret_cast<const float4*>(sP + (r * 8 + ty) * LP + s);
+#pragma unroll
+                    for (int e = 0; e < 4; ++e)
+#pragma unroll
+                        for (int x = 0; x < 4; ++x) o[r][x] = fmaf(mv[e], uv[e][x], o[r][x]);
+                }
+            }
+    }
+#pragma unroll
+    for (int r = 0; r < 8; ++r) {
+        const int t = r * 8 + ty;
         if (t >= n) continue;
         float* orow = a.out + (size_t)(r0 + t) * a.out_stride + (size_t)h * a.dv;
 #pragma unroll
@@ -608,12 +640,13 @@ delta_out_kernel(DeltaArgs a) {
 }
 
 // ------------------------------------------------------------------ host side
-static int delta_up4(int n) { return (n + 3) / 4 * 4; }
+static int delta_dkp(int dk) { return dk <= 64 ? 64 : dk <= 128 ? 128 : 256; }
+static long long delta_blocks(int rows, int n_seqs, int heads) { return ((long long)rows / DELTA_C + n_seqs + 1) * heads; }
 
-// Floats of scratch that the chunked form of a step needs: row-wise buffers, then the chunks' decays and states.
-extern "C" long long braid_delta_work_floats(int rows, int n_seqs, int max_q_len, int heads, int dk, int dv) {
-    const long long dk4 = delta_up4(dk), dv4 = delta_up4(dv), chunks = (max_q_len + DELTA_C - 1) / DELTA_C;
-    return (long long)rows * heads * (3 * dk4 + dv4 + DELTA_C) + n_seqs * chunks * heads * (dk4 + dk * dv4);
+// Floats of scratch that the chunked form of a step needs.
+extern "C" long long braid_delta_work_floats(int rows, int n_seqs, int heads, int dk, int dv) {
+    const long long dkp = delta_dkp(dk), dvp = (dv + DELTA_DVT - 1) / DELTA_DVT * DELTA_DVT;
+    return delta_blocks(rows, n_seqs, heads) * (3 * DELTA_C * (dkp + 4) + DELTA_C * dvp + DELTA_C * DELTA_C + dkp + dkp * dvp);
 }
 
 template <typename T, int DKP>
@@ -626,17 +659,16 @@ static int launch_delta_chunks(const DeltaArgs& a, int n_seqs, cudaStream_t s) {
         if (e != cudaSuccess) { braid_set_error("delta_rule: cannot reserve shared memory: %s", cudaGetErrorString(e)); return (int)e; }
         configured = true;
     }
-    const int tiles = (a.dv4 + DELTA_OUT_COLS - 1) / DELTA_OUT_COLS;
+    const int spans = (a.tiles * DELTA_DVT + DELTA_OUT_COLS - 1) / DELTA_OUT_COLS;
     braid_launch(delta_intra_kernel<T, DKP>, dim3(a.heads, n_seqs, a.max_chunks), dim3(DELTA_INTRA_THREADS), delta_intra_smem<DKP>(), s, a);
-    braid_launch(delta_state_kernel<DKP>, dim3(a.heads, n_seqs, (a.dv4 + DELTA_DVT - 1) / DELTA_DVT), dim3(DELTA_STATE_THREADS), delta_state_smem<DKP>(), s, a);
-    braid_launch(delta_out_kernel<DKP>, dim3(a.heads, n_seqs, a.max_chunks * tiles), dim3(DELTA_OUT_THREADS), delta_out_smem<DKP>(), s, a);
+    braid_launch(delta_state_kernel<DKP>, dim3(a.heads, n_seqs, a.tiles), dim3(DELTA_STATE_THREADS), delta_state_smem<DKP>(), s, a);
+    braid_launch(delta_out_kernel<DKP>, dim3(a.heads, n_seqs, a.max_chunks * spans), dim3(DELTA_OUT_THREADS), delta_out_smem<DKP>(), s, a);
     BRAID_LAUNCH_CHECK();
 }
 
 template <typename T>
 static int launch_delta(const DeltaArgs& a, int n_seqs, bool chunked, cudaStream_t s) {
     if (chunked) {
-        if (a.dk <= 32) return launch_delta_chunks<T, 32>(a, n_seqs, s);
         if (a.dk <= 64) return launch_delta_chunks<T, 64>(a, n_seqs, s);
         if (a.dk <= 128) return launch_delta_chunks<T, 128>(a, n_seqs, s);
         return launch_delta_chunks<T, 256>(a, n_seqs, s);
@@ -665,21 +697,21 @@ extern "C" int braid_delta_rule(const float* q, long long q_stride, const float*
     if (dtype != BRAID_F32 && dtype != BRAID_BF16) BRAID_REFUSE("delta_rule: unknown dtype code %d", dtype);
     DeltaArgs a{q, q_stride, k, k_stride, v, v_stride, z, z_stride, bias, rate, b, b_stride, out, out_stride, (uint8_t*)state,
                 state_stride, state_offset, q_start, q_len, slot_ids, heads, groups, dk, dv,
-                nullptr, nullptr, nullptr, nullptr, nullptr, nullptr, nullptr, delta_up4(dk), delta_up4(dv),
+                nullptr, nullptr, nullptr, nullptr, nullptr, nullptr, nullptr, (dv + DELTA_DVT - 1) / DELTA_DVT,
                 (max_q_len + DELTA_C - 1) / DELTA_C};
-    const long long tiles = (a.dv4 + DELTA_OUT_COLS - 1) / DELTA_OUT_COLS;
-    if (n_seqs > 65535 || (dv + 31) / 32 > 65535 || (work && a.max_chunks * tiles > 65535)) BRAID_REFUSE("delta_rule: the step exceeds the grid limits");
+    const long long spans = (a.tiles * DELTA_DVT + DELTA_OUT_COLS - 1) / DELTA_OUT_COLS;
+    if (n_seqs > 65535 || a.tiles > 65535 || (work && a.max_chunks * spans > 65535)) BRAID_REFUSE("delta_rule: the step exceeds the grid limits");
     if (work) {
-        const long long need = braid_delta_work_floats(rows, n_seqs, max_q_len, heads, dk, dv);
+        const long long need = braid_delta_work_floats(rows, n_seqs, heads, dk, dv);
         if (need > work_floats || ((uintptr_t)work & 15)) BRAID_REFUSE("delta_rule: the chunked form needs %lld floats of scratch on 16 bytes, it was given %lld", need, work_floats);
-        const long long rh = (long long)rows * heads;
+        const long long blocks = delta_blocks(rows, n_seqs, heads), dkp = delta_dkp(dk), wide = blocks * DELTA_C * (dkp + 4);
         a.w = work;
-        a.u = a.w + rh * a.dk4;
-        a.qd = a.u + rh * a.dv4;
-        a.kd = a.qd + rh * a.dk4;
-        a.p = a.kd + rh * a.dk4;
-        a.gc = a.p + rh * DELTA_C;
-        a.sc = a.gc + (long long)n_seqs * a.max_chunks * heads * a.dk4;
+        a.qd = a.w + wide;
+        a.kd = a.qd + wide;
+        a.u = a.kd + wide;
+        a.p = a.u + blocks * a.tiles * DELTA_C * DELTA_DVT;
+        a.gc = a.p + blocks * DELTA_C * DELTA_C;
+        a.sc = a.gc + blocks * dkp;
     }
     if (dtype == BRAID_F32) return launch_delta<float>(a, n_seqs, work != nullptr, (cudaStream_t)stream);
     return launch_delta<__nv_bfloat16>(a, n_seqs, work != nullptr, (cudaStream_t)stream);
