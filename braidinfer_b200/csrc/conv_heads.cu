@@ -24,6 +24,7 @@ struct ConvSegment {
     int norm, silu, rotate;
     int plane;                   // -1: to `out`; 0, 1: the cache's key or value plane
     float factor;
+    float inv_count;             // 1 / size for CONV_NORM_RMS, else 1
     const void* weight;          // CONV_NORM_RMS: [size] in the run's type
     void* out;                   // [rows, out_stride], head h at column h * pad
     long long out_stride;
@@ -62,181 +63,272 @@ __device__ __forceinline__ TO* conv_dst(const ConvHeadsArgs& a, const ConvSegmen
     return (TO*)a.cache + ((((size_t)page * 2 + s.plane) * s.heads + h) * a.page_size + off) * s.pad;
 }
 
-// 16 bytes of neighbouring channels a thread, LPH lanes a head, RPT neighbouring rows a thread: for sizes, strides and taps
-// that allow it (neighbouring pairs in the rotation).  TO: the type of what is stored.  What the rows' tables say is asked for
-// in rounds over all RPT rows (one trip a round instead of one a row), and the CTA's heads share the sines and cosines.
+// ---- 16 bytes of neighbouring channels a thread, LPH lanes a head: for sizes, strides and taps that allow it (neighbouring
+// pairs in the rotation).  TO: the type of what is stored.
 #define CONV_MAX_PAIRS 128
-template <typename T, typename TO, int TAPS, int LPH, int RPT>
-__global__ void __launch_bounds__(128, RPT > 1 ? 4 : 6)
-conv_heads_vec_kernel(ConvHeadsArgs a) {
-    constexpr int VEC = 16 / sizeof(T), HPC = 128 / LPH, SPAN = RPT + TAPS - 1;
-    __shared__ float2 turn[RPT][CONV_MAX_PAIRS];           // (sine, cosine) of the rows' angles
-    pdl_trigger();
-    const int sub = threadIdx.x / LPH, l = threadIdx.x % LPH, i0 = l * VEC;
-    // which segment and head: the segments' heads are counted through
-    int head = blockIdx.x * HPC + sub, c_seg = 0;
-    ConvSegment s = a.seg[0];
+
+// A thread's place among the segments' channels.
+struct ConvPlace {
+    ConvSegment s;
+    int head, c0, i0, l;         // head of the segment, first channel of all, of the head, lane of the head
+    bool live, in;               // a head at all; channels of one
+};
+template <typename T, int LPH>
+__device__ __forceinline__ ConvPlace conv_place(const ConvHeadsArgs& a) {
+    constexpr int VEC = 16 / sizeof(T), HPC = 128 / LPH;
+    ConvPlace p;
+    int c_seg = 0;
+    p.l = threadIdx.x % LPH;
+    p.i0 = p.l * VEC;
+    p.head = blockIdx.x * HPC + threadIdx.x / LPH;         // the segments' heads are counted through
+    p.s = a.seg[0];
 #pragma unroll
     for (int si = 1; si < CONV_MAX_SEGS; ++si)
-        if (si < a.n_segs && head >= s.heads) {
-            head -= s.heads;
-            c_seg += s.heads * s.size;
-            s = a.seg[si];
+        if (si < a.n_segs && p.head >= p.s.heads) {
+            p.head -= p.s.heads;
+            c_seg += p.s.heads * p.s.size;
+            p.s = a.seg[si];
         }
-    const bool live = head < s.heads, in = live && i0 < s.size;
-    const int c0 = c_seg + head * s.size + i0;
-    const int row0 = blockIdx.y * RPT;
-    // the step's tables are on the device before its first kernel: read before the wait
-    int seq[RPT], pos[RPT], o[RPT], slot[RPT], qlen[RPT];
-#pragma unroll
-    for (int r = 0; r < RPT; ++r) {
-        seq[r] = row0 + r < a.rows ? a.token_seq[row0 + r] : -1;
-        pos[r] = row0 + r < a.rows ? a.positions[row0 + r] : 0;
-    }
-#pragma unroll
-    for (int r = 0; r < RPT; ++r) {
-        const int q = max(seq[r], 0);
-        o[r] = row0 + r - a.q_start[q];
-        qlen[r] = a.q_len[q];
-        slot[r] = a.slot_ids[q];
-    }
-    TO* dst[RPT];
-#pragma unroll
-    for (int r = 0; r < RPT; ++r) dst[r] = live && seq[r] >= 0 ? conv_dst<T, TO>(a, s, head, row0 + r, seq[r], pos[r], l == 0) : nullptr;
-    if (a.turns) {
-        const int half = a.rope_dim / 2;
-        for (int idx = threadIdx.x; idx < RPT * half; idx += 128) {
-            const int r = idx / half, p = idx - r * half;
-            const int ps = row0 + r < a.rows ? a.positions[row0 + r] : 0;
-            float sn, cs;
-            sincosf((float)ps * a.inv_freq[p], &sn, &cs);
-            turn[r][p] = make_float2(sn * a.amp, cs * a.amp);
-        }
-        __syncthreads();
-    }
-    float wl[VEC * TAPS], bl[VEC];
+    p.live = p.head < p.s.heads;
+    p.in = p.live && p.i0 < p.s.size;
+    p.c0 = c_seg + p.head * p.s.size + p.i0;
+    return p;
+}
+
+// The taps and biases of a thread's channels.
+template <typename T, int TAPS, int VEC>
+__device__ __forceinline__ void conv_weights(const ConvHeadsArgs& a, const ConvPlace& p, float* wl, float* bl) {
 #pragma unroll
     for (int e = 0; e < VEC; ++e) bl[e] = 0.f;
-    if (in) {
 #pragma unroll
-        for (int u = 0; u < TAPS; ++u) load_run<T, VEC>((const T*)a.w + (size_t)c0 * TAPS + u * VEC, wl + u * VEC);
-        if (a.bias) load_run<T, VEC>((const T*)a.bias + c0, bl);
+    for (int e = 0; e < VEC * TAPS; ++e) wl[e] = 0.f;
+    if (!p.in) return;
+#pragma unroll
+    for (int u = 0; u < TAPS; ++u) load_run<T, VEC>((const T*)a.w + (size_t)p.c0 * TAPS + u * VEC, wl + u * VEC);
+    if (a.bias) load_run<T, VEC>((const T*)a.bias + p.c0, bl);
+}
+
+// silu, norm, rotation and store of one row's channels; the whole warp calls.  `turn`: the row's sines and cosines.
+template <typename T, typename TO, int LPH, int VEC>
+__device__ __forceinline__ void conv_finish(const ConvHeadsArgs& a, const ConvPlace& p, float* y, const float2* turn, TO* dst) {
+    if (p.s.silu) {
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) y[e] = sizeof(T) == 2 ? glu_act_fast(y[e], BRAID_ACT_SILU) : silu_f32(y[e]);
     }
+    float ss = 0.f;
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) ss = fmaf(y[e], y[e], ss);
+#pragma unroll
+    for (int b = LPH / 2; b > 0; b >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, b);       // whatever the lanes' segments
+    if (p.s.norm != CONV_NORM_NONE) {
+        const float m = ss * p.s.inv_count + a.eps;
+        const float r = p.s.factor * (sizeof(T) == 2 ? rsqrtf(m) : 1.f / sqrtf(m));
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) y[e] *= r;
+        if (p.in && p.s.norm == CONV_NORM_RMS) {
+            float nw[VEC];
+            load_run<T, VEC>((const T*)p.s.weight + p.i0, nw);
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) y[e] *= nw[e];
+        }
+    } else if (p.s.factor != 1.f) {
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) y[e] *= p.s.factor;
+    }
+    if (!dst || p.i0 >= p.s.pad) return;
+    if (p.s.rotate && p.i0 < a.rope_dim) {
+#pragma unroll
+        for (int e = 0; e < VEC; e += 2) {
+            const int k = (p.i0 + e) >> 1;
+            if (2 * k < a.rope_dim) {
+                const float2 t = turn[k];
+                const float u = y[e], v = y[e + 1];
+                y[e] = u * t.y - v * t.x;
+                y[e + 1] = v * t.y + u * t.x;
+            }
+        }
+    }
+    constexpr int VO = 16 / sizeof(TO) < VEC ? 16 / sizeof(TO) : VEC;
+#pragma unroll
+    for (int e = 0; e < VEC; e += VO) store_run<TO, VO>(dst + p.i0 + e, y + e);
+}
+
+// One row whose taps may reach before the step: every tap's row is looked up, in the step or in the state.  `st` is the row's
+// sequence's state; with `move` (a sequence of one token, whose channels nobody else reads) it takes the new row.
+template <typename T, int TAPS, int VEC>
+__device__ __forceinline__ void conv_row(const ConvHeadsArgs& a, const ConvPlace& p, const float* wl, const float* bl, int row, int o, float* st,
+                                         bool move, float* y) {
+    float u[TAPS][VEC];
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j) {
+        const int back = TAPS - 1 - j;
+        if (o - back >= 0) {
+            load_run<T, VEC>((const T*)a.x + (size_t)(row - back) * a.x_stride + p.c0, u[j]);
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) u[j][e] += bl[e];
+        } else {
+            const float* sp = st + (size_t)(TAPS - 1 + (o - back)) * a.channels + p.c0;
+#pragma unroll
+            for (int e = 0; e < VEC; e += 4) load_run<float, 4>(sp + e, u[j] + e);
+        }
+    }
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j)
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) y[e] = fmaf(wl[e * TAPS + j], u[j][e], y[e]);
+    if (move) {
+#pragma unroll
+        for (int k = 0; k < TAPS - 1; ++k)
+#pragma unroll
+            for (int e = 0; e < VEC; e += 4) store_run<float, 4>(st + (size_t)k * a.channels + p.c0 + e, u[k + 1] + e);
+    }
+}
+
+// Sines and cosines of rows row0 .. row0 + n - 1, by the whole CTA; their positions are pos0 and on, or (pos0 < 0) looked up.
+__device__ __forceinline__ void conv_turns(const ConvHeadsArgs& a, int row0, int n, int pos0, float2 (*turn)[CONV_MAX_PAIRS]) {
+    const int half = a.rope_dim / 2;
+    for (int idx = threadIdx.x; idx < n * half; idx += 128) {
+        const int r = idx / half, k = idx - r * half;
+        const int ps = pos0 >= 0 ? pos0 + r : row0 + r < a.rows ? a.positions[row0 + r] : 0;
+        float sn, cs;
+        sincosf((float)ps * a.inv_freq[k], &sn, &cs);
+        turn[r][k] = make_float2(sn * a.amp, cs * a.amp);
+    }
+}
+
+// Few rows: one a CTA.
+template <typename T, typename TO, int TAPS, int LPH>
+__global__ void __launch_bounds__(128)
+conv_heads_row_kernel(ConvHeadsArgs a) {
+    constexpr int VEC = 16 / sizeof(T);
+    __shared__ float2 turn[1][CONV_MAX_PAIRS];
+    pdl_trigger();
+    const ConvPlace p = conv_place<T, LPH>(a);
+    const int row = blockIdx.y;
+    // the step's tables are on the device before its first kernel: read before the wait
+    const int seq = a.token_seq[row];
+    if (seq < 0) return;
+    const int o = row - a.q_start[seq];
+    const bool move = TAPS > 1 && a.q_len[seq] == 1;
+    float* st = a.state ? (float*)(a.state + (size_t)a.slot_ids[seq] * a.state_stride + a.state_offset) : nullptr;
+    TO* dst = p.live ? conv_dst<T, TO>(a, p.s, p.head, row, seq, a.positions[row], p.l == 0) : nullptr;
+    if (a.turns) {
+        conv_turns(a, row, 1, -1, turn);
+        __syncthreads();
+    }
+    float wl[VEC * TAPS], bl[VEC], y[VEC];
+    conv_weights<T, TAPS, VEC>(a, p, wl, bl);
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) y[e] = 0.f;
     pdl_wait();
-    __align__(16) T xin[SPAN][VEC];                        // as they came: the bias is added where a row is used
+    if (p.in) conv_row<T, TAPS, VEC>(a, p, wl, bl, row, o, st, move, y);
+    conv_finish<T, TO, LPH, VEC>(a, p, y, turn[0], dst);
+}
+
+// Many rows: a CTA walks `span` neighbouring rows, four at a time, the next four on their way.  Where four rows and what their
+// taps reach lie inside one sequence's step (nearly everywhere), every row is loaded and converted once, the window of rows
+// moves along, and the bias comes through the sum of the taps.
+#define CONV_RPT 4
+template <typename T, typename TO, int TAPS, int LPH>
+__global__ void __launch_bounds__(128, 3)
+conv_heads_span_kernel(ConvHeadsArgs a, int span) {
+    constexpr int VEC = 16 / sizeof(T), R = CONV_RPT;
+    __shared__ float2 turn[2][R][CONV_MAX_PAIRS];
+    pdl_trigger();
+    const ConvPlace p = conv_place<T, LPH>(a);
+    const int begin = blockIdx.y * span, end = min(a.rows, begin + span);
+    float wl[VEC * TAPS], bl[VEC], yb[VEC];
+    conv_weights<T, TAPS, VEC>(a, p, wl, bl);
 #pragma unroll
-    for (int u = 0; u < SPAN; ++u) {
-        const int r = row0 - (TAPS - 1) + u;
-        if (in && r >= 0 && r < a.rows) *reinterpret_cast<uint4*>(xin[u]) = *reinterpret_cast<const uint4*>((const T*)a.x + (size_t)r * a.x_stride + c0);
-        else *reinterpret_cast<uint4*>(xin[u]) = make_uint4(0, 0, 0, 0);
+    for (int e = 0; e < VEC; ++e) {
+        float sum = 0.f;
+#pragma unroll
+        for (int j = 0; j < TAPS; ++j) sum += wl[e * TAPS + j];
+        yb[e] = sum * bl[e];
     }
-    // silu, norm, rotation and store of one row's channels; the whole warp calls
-    auto finish = [&](int rr, float* y) {
-        if (s.silu) {
+    int first = a.token_seq[begin], last = a.token_seq[min(begin + R, end) - 1], known = -1, q0 = 0, p0 = 0;
+    pdl_wait();
+    const T* x = (const T*)a.x + p.c0;
+    uint4 next[R];
+    auto ask = [&](int row0) {
 #pragma unroll
-            for (int e = 0; e < VEC; ++e) y[e] = sizeof(T) == 2 ? glu_act_fast(y[e], BRAID_ACT_SILU) : silu_f32(y[e]);
-        }
-        float ss = 0.f;
-#pragma unroll
-        for (int e = 0; e < VEC; ++e) ss = fmaf(y[e], y[e], ss);
-#pragma unroll
-        for (int b = LPH / 2; b > 0; b >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, b);       // whatever the lanes' segments
-        if (s.norm != CONV_NORM_NONE) {
-            const float r = s.factor / sqrtf((s.norm == CONV_NORM_RMS ? ss / (float)s.size : ss) + a.eps);
-#pragma unroll
-            for (int e = 0; e < VEC; ++e) y[e] *= r;
-            if (in && s.norm == CONV_NORM_RMS) {
-                float nw[VEC];
-                load_run<T, VEC>((const T*)s.weight + i0, nw);
-#pragma unroll
-                for (int e = 0; e < VEC; ++e) y[e] *= nw[e];
-            }
-        } else if (s.factor != 1.f) {
-#pragma unroll
-            for (int e = 0; e < VEC; ++e) y[e] *= s.factor;
-        }
-        if (!dst[rr] || i0 >= s.pad) return;
-        if (s.rotate && i0 < a.rope_dim) {
-#pragma unroll
-            for (int e = 0; e < VEC; e += 2) {
-                const int p = (i0 + e) >> 1;
-                if (2 * p < a.rope_dim) {
-                    const float2 t = turn[rr][p];
-                    const float u = y[e], v = y[e + 1];
-                    y[e] = u * t.y - v * t.x;
-                    y[e + 1] = v * t.y + u * t.x;
-                }
-            }
-        }
-        constexpr int VO = 16 / sizeof(TO) < VEC ? 16 / sizeof(TO) : VEC;
-#pragma unroll
-        for (int e = 0; e < VEC; e += VO) store_run<TO, VO>(dst[rr] + i0 + e, y + e);
+        for (int r = 0; r < R; ++r)
+            next[r] = p.in && row0 + r < end ? *reinterpret_cast<const uint4*>(x + (size_t)(row0 + r) * a.x_stride) : make_uint4(0, 0, 0, 0);
     };
-    if (RPT > 1 && seq[0] >= 0 && seq[0] == seq[RPT - 1] && o[0] >= TAPS - 1) {
-        // all rows and what their taps reach lie inside one sequence's step: every row is converted once, the bias comes
-        // through the sum of the taps
-        float win[TAPS][VEC], yb[VEC];
+    ask(begin);
+    float win[TAPS][VEC];                                  // row begin - (TAPS - 1) + u at place u % TAPS
+    bool fresh = true;                                     // the window is still to be filled from the rows before
+    int buf = 0;
+    for (int row0 = begin; row0 < end; row0 += R) {
+        uint4 cur[R];
 #pragma unroll
-        for (int e = 0; e < VEC; ++e) {
-            float sum = 0.f;
-#pragma unroll
-            for (int j = 0; j < TAPS; ++j) sum += wl[e * TAPS + j];
-            yb[e] = sum * bl[e];
+        for (int r = 0; r < R; ++r) cur[r] = next[r];
+        const int seq = first;
+        const bool one = seq >= 0 && seq == last && row0 + R <= end;
+        if (row0 + R < end) {
+            ask(row0 + R);
+            first = a.token_seq[row0 + R];
+            last = a.token_seq[min(row0 + 2 * R, end) - 1];
         }
+        if (one && seq != known) {                         // where the sequence's rows start, and its position there
+            known = seq;
+            q0 = a.q_start[seq];
+            p0 = a.positions[q0];
+        }
+        const bool inner = one && row0 - q0 >= TAPS - 1;
+        const int pos0 = p0 + row0 - q0;
+        if (a.turns) {
+            conv_turns(a, row0, R, inner ? pos0 : -1, turn[buf]);
+            __syncthreads();                               // two tables take turns: one barrier a round is enough
+        }
+        if (inner) {
+            TO* dst[R];
 #pragma unroll
-        for (int u = 0; u < SPAN; ++u) {
+            for (int r = 0; r < R; ++r) dst[r] = p.live ? conv_dst<T, TO>(a, p.s, p.head, row0 + r, seq, pos0 + r, p.l == 0) : nullptr;
+            if (fresh) {
 #pragma unroll
-            for (int e = 0; e < VEC; ++e) win[u % TAPS][e] = to_f32(xin[u][e]);
-            if (u < TAPS - 1) continue;
-            float y[VEC];
+                for (int u = 0; u < TAPS - 1; ++u) {
+                    if (p.in) load_run<T, VEC>(x + (size_t)(row0 - (TAPS - 1) + u) * a.x_stride, win[u]);
+                    else
 #pragma unroll
-            for (int e = 0; e < VEC; ++e) {
-                y[e] = yb[e];
-#pragma unroll
-                for (int j = 0; j < TAPS; ++j) y[e] = fmaf(wl[e * TAPS + j], win[(u + 1 + j) % TAPS][e], y[e]);
+                        for (int e = 0; e < VEC; ++e) win[u][e] = 0.f;
+                }
+                fresh = false;
             }
-            finish(u - (TAPS - 1), y);
-        }
-        return;
-    }
 #pragma unroll
-    for (int rr = 0; rr < RPT; ++rr) {
-        if (seq[rr] < 0) continue;                         // the whole CTA: rows are the grid's
-        float* st = a.state ? (float*)(a.state + (size_t)slot[rr] * a.state_stride + a.state_offset) : nullptr;
-        float y[VEC];
+            for (int r = 0; r < R; ++r) {
+                const T* c = reinterpret_cast<const T*>(&cur[r]);
 #pragma unroll
-        for (int e = 0; e < VEC; ++e) y[e] = 0.f;
-        if (in) {
-            const bool alone = RPT == 1 && TAPS > 1 && qlen[rr] == 1;
-            float old[RPT == 1 && TAPS > 1 ? TAPS - 1 : 1][VEC];       // rows before the step that this row's taps reach
+                for (int e = 0; e < VEC; ++e) win[TAPS - 1][e] = to_f32(c[e]);
+                float y[VEC];
 #pragma unroll
-            for (int j = 0; j < TAPS; ++j) {
-                const int back = TAPS - 1 - j;
-                float xv[VEC];
-                if (o[rr] - back >= 0) {
+                for (int e = 0; e < VEC; ++e) {
+                    y[e] = yb[e];
 #pragma unroll
-                    for (int e = 0; e < VEC; ++e) xv[e] = to_f32(xin[rr + j][e]) + bl[e];
-                } else {
-                    const float* sp = st + (size_t)(TAPS - 1 + (o[rr] - back)) * a.channels + c0;
-#pragma unroll
-                    for (int e = 0; e < VEC; e += 4) load_run<float, 4>(sp + e, xv + e);
+                    for (int j = 0; j < TAPS; ++j) y[e] = fmaf(wl[e * TAPS + j], win[j][e], y[e]);
                 }
-                if (RPT == 1 && j < TAPS - 1) {
+                conv_finish<T, TO, LPH, VEC>(a, p, y, turn[buf][r], dst[r]);
 #pragma unroll
-                    for (int e = 0; e < VEC; ++e) old[RPT == 1 ? j : 0][e] = xv[e];
-                }
+                for (int j = 0; j < TAPS - 1; ++j)
 #pragma unroll
-                for (int e = 0; e < VEC; ++e) y[e] = fmaf(wl[e * TAPS + j], xv[e], y[e]);
-                if (alone && j == TAPS - 1) {              // one token: nobody else reads these channels of the state
+                    for (int e = 0; e < VEC; ++e) win[j][e] = win[j + 1][e];
+            }
+        } else {
+            fresh = true;
+#pragma unroll 1
+            for (int r = 0; r < R && row0 + r < end; ++r) {
+                const int row = row0 + r, sq = a.token_seq[row];
+                if (sq < 0) continue;
+                float* st = a.state ? (float*)(a.state + (size_t)a.slot_ids[sq] * a.state_stride + a.state_offset) : nullptr;
+                TO* dst = p.live ? conv_dst<T, TO>(a, p.s, p.head, row, sq, a.positions[row], p.l == 0) : nullptr;
+                float y[VEC];
 #pragma unroll
-                    for (int k = 0; k < TAPS - 1; ++k)
-#pragma unroll
-                        for (int e = 0; e < VEC; e += 4)
-                            store_run<float, 4>(st + (size_t)k * a.channels + c0 + e, (k < TAPS - 2 ? old[RPT == 1 && k < TAPS - 2 ? k + 1 : 0] : xv) + e);
-                }
+                for (int e = 0; e < VEC; ++e) y[e] = 0.f;
+                if (p.in) conv_row<T, TAPS, VEC>(a, p, wl, bl, row, row - a.q_start[sq], st, false, y);
+                conv_finish<T, TO, LPH, VEC>(a, p, y, turn[buf][r], dst);
             }
         }
-        finish(rr, y);
+        buf ^= 1;
     }
 }
 
@@ -283,7 +375,7 @@ conv_heads_kernel(ConvHeadsArgs a) {
     float r = s.factor;
     if (s.norm != CONV_NORM_NONE) {
         ss = warp_sum(ss);
-        r = s.factor / sqrtf((s.norm == CONV_NORM_RMS ? ss / (float)s.size : ss) + a.eps);
+        r = s.factor / sqrtf(ss * s.inv_count + a.eps);
     }
     __syncwarp();
     for (int i = lane; i < s.size; i += 32) y[i] *= s.norm == CONV_NORM_RMS ? r * to_f32(((const T*)s.weight)[i]) : r;
@@ -334,13 +426,15 @@ static int launch_conv_vec(const ConvHeadsArgs& a, cudaStream_t s) {
     int heads = 0;
     for (int i = 0; i < a.n_segs; ++i) heads += a.seg[i].heads;
     const int groups = (heads + HPC - 1) / HPC;
-    // neighbouring rows a thread: four where the rows alone fill the machine
-    if ((long long)a.rows * groups >= 148 * 16) {
-        braid_launch(conv_heads_vec_kernel<T, TO, TAPS, LPH, 4>, dim3(groups, (a.rows + 3) / 4), dim3(128), 0, s, a);
-        return 1;
+    if ((long long)a.rows * groups < 148 * 16) {
+        braid_launch(conv_heads_row_kernel<T, TO, TAPS, LPH>, dim3(groups, a.rows), dim3(128), 0, s, a);
+        return 2;
     }
-    braid_launch(conv_heads_vec_kernel<T, TO, TAPS, LPH, 1>, dim3(groups, a.rows), dim3(128), 0, s, a);
-    return 2;
+    // spans so long that one wave of CTAs (three an SM) covers the rows, in whole rounds
+    long long span = ((long long)a.rows * groups + 148 * 3 - 1) / (148 * 3);
+    span = (span + CONV_RPT - 1) / CONV_RPT * CONV_RPT;
+    braid_launch(conv_heads_span_kernel<T, TO, TAPS, LPH>, dim3(groups, (unsigned)((a.rows + span - 1) / span)), dim3(128), 0, s, a, (int)span);
+    return 1;
 }
 
 template <typename T, typename TO>
@@ -389,7 +483,8 @@ extern "C" int braid_conv_heads(const void* x, long long x_stride, const void* b
     int widest = 0;
     for (int i = 0; i < n_segs; ++i) {                      // (inv_freq is read only where something turns)
         const int* g = segs + 7 * i;
-        a.seg[i] = ConvSegment{g[0], g[1], g[2], g[3], g[4], g[5], g[6], factors[i], weights[i], outs[i], out_strides[i]};
+        a.seg[i] = ConvSegment{g[0], g[1], g[2], g[3], g[4], g[5], g[6], factors[i],
+                               g[3] == CONV_NORM_RMS ? 1.f / (float)g[1] : 1.f, weights[i], outs[i], out_strides[i]};
         const ConvSegment& s = a.seg[i];
         if (s.heads <= 0 || s.size <= 0 || s.pad < s.size || s.pad > CONV_MAX_SIZE || (s.rotate && rope_dim > s.size))
             BRAID_REFUSE("conv_heads: heads of %d in %d numbers (at most %d), %d of them rotated", s.size, s.pad, CONV_MAX_SIZE, rope_dim);
