@@ -2026,7 +2026,8 @@ def megerax_kernels(name, T, B, C, timed, frac):
             K.causal_conv(x, yb, w, b, cst, 0, stp, silu=False)
             K.head_norm_rope_kv(yb, wn, wn, inv, stp.positions, stp.token_seq, table, cache, H, nkh, hd, hd // 2, True, False, PAGE_SIZE, 1e-6)
         t2 = timed(two, reps=9, graph=True)
-        pair(f"{what}_convolved_heads", (t1, 0, rows * ch * 4 + n_seqs * 3 * ch * 8), (t2, 0, rows * (ch * 4 + (H + nkh) * hd * 4 + 2 * nkh * hd * 2) + n_seqs * 3 * ch * 8))
+        by = rows * ch * 4 + n_seqs * 3 * ch * 8               # what the job must move, in one kernel or in two
+        pair(f"{what}_convolved_heads", (t1, 0, by), (t2, 0, by))
         # ---- the delta layer: its convolution (silu, unit heads, float32 out) beside Mamba-2's, the recurrence and the read-out beside
         # those of the gated linear attention
         heads, dk, dv = z["lheads"], z["ldk"], z["ldv"]
