@@ -143,6 +143,73 @@ def test_convolution_with_silu_and_unit_heads_in_32_bits(K, dtype, H, G, dk, dv,
     K.check_device_errors()
 
 
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("nqh, nkh, hd, taps, rot", [(3, 1, 16, 4, 8), (4, 2, 64, 3, 64), (2, 2, 128, 2, 32), (5, 1, 48, 4, 16)])
+def test_convolved_heads_of_many_rows_and_sequences(K, dtype, nqh, nkh, hd, taps, rot):
+    """Steps of so many rows that a CTA walks a span of them: long sequences, short ones that begin and end anywhere in a span,
+    hundreds of one token, over three steps with the inputs between them in the slots; rows of padding in the middle of nothing."""
+    g = torch.Generator().manual_seed(hd)
+    page, eps, ch = 64, 1e-5, (nqh + 2 * nkh) * hd
+    first = [2111, 1, 2, 5, 700, 3] + [1] * 300
+    steps = [first, [40, 1, 7, 1, 1500, 2] + [1] * 900, [1] * 2600]
+    n_seqs = max(len(c) for c in steps)
+    total = [sum(c[i] for c in steps if i < len(c)) for i in range(n_seqs)]
+    xs = [dev(torch.randn(n, ch, generator=g), dtype) for n in total]
+    b, w = dev(torch.randn(ch, generator=g), dtype), dev(torch.randn(ch, taps, generator=g) * 0.5, dtype)
+    qw, kw = (dev(1 + 0.3 * torch.randn(hd, generator=g), dtype) for _ in range(2))
+    r = {"base": 500.0, "dims": rot}
+    inv = P.frequencies(r).float().cuda()
+    # the plain result, all sequences as one batch with zeros before each start
+    flat = torch.cat([torch.cat([torch.zeros(taps - 1, ch, dtype=D), back(x) + back(b)]) for x in xs])
+    y = P.causal_conv(flat, back(w))
+    keep = torch.cat([torch.arange(n) + taps - 1 + at for n, at in zip(total, torch.tensor([0] + [n + taps - 1 for n in total[:-1]]).cumsum(0).tolist())])
+    y, pos = y[keep], torch.cat([torch.arange(n) for n in total])
+    starts = torch.tensor([0] + total[:-1]).cumsum(0).tolist()
+    q = P.rotate(P.norm(y[:, :nqh * hd].view(-1, nqh, hd), back(qw), eps), pos, r, "pairs")
+    k = P.rotate(P.norm(y[:, nqh * hd:(nqh + nkh) * hd].view(-1, nkh, hd), back(kw), eps), pos, r, "pairs")
+    v = y[:, (nqh + nkh) * hd:].view(-1, nkh, hd)
+    table, cache = paged(total, nkh, page, hd, dtype, g)
+    state, at = torch.zeros(n_seqs, (taps - 1) * ch * 4, dtype=torch.uint8, device="cuda"), [0] * n_seqs
+    tol = 3e-4 if dtype == "float32" else 1.2e-2                                # (angles of thousands of radians in float32)
+    for counts in steps:
+        m = len(counts)
+        t = step_tables(counts, at[:m], pad=3)
+        rows = torch.cat([xs[i][at[i]:at[i] + n] for i, n in enumerate(counts)] + [torch.full((3, ch), 9.0, dtype=TORCH[dtype], device="cuda")])
+        q_out = torch.full((t.rows, nqh * hd), 3.0, dtype=TORCH[dtype], device="cuda")
+        head = dict(norm="rms", rotate=True)
+        K.conv_heads(rows, w, b, state, 0, t, [K.conv_segment(nqh, hd, weight=qw, out=q_out, **head), K.conv_segment(nkh, hd, weight=kw, plane=0, **head),
+                                              K.conv_segment(nkh, hd, plane=1)], eps=eps, inv_freq=inv, page_table=table[:m].contiguous().cuda(), cache=cache)
+        K.check_device_errors()
+        where = torch.cat([torch.arange(at[i], at[i] + n) + starts[i] for i, n in enumerate(counts)])
+        assert rel(q_out[:t.n_tokens], q[where].reshape(len(where), -1)) < tol and (q_out[t.n_tokens:] == 3.0).all()
+        at = [x + (counts[i] if i < m else 0) for i, x in enumerate(at)]
+    seq = torch.repeat_interleave(torch.arange(n_seqs), torch.tensor(total))
+    pg = table[seq, pos // page].long().cuda()
+    assert rel(cache[pg, 0, :, (pos % page).cuda()], k) < tol and rel(cache[pg, 1, :, (pos % page).cuda()], v) < (1e-5 if dtype == "float32" else 1e-2)
+    for i in (0, 1, 2, 4, 5, 200, 1100, 2599):
+        u = torch.cat([torch.zeros(taps - 1, ch), xs[i].float().cpu() + b.float().cpu()])[-(taps - 1):]
+        assert torch.allclose(state[i].view(torch.float32).view(taps - 1, ch).cpu(), u, atol=1e-6)
+    # the delta layer's form on the same rows: silu, unit heads, float32 results, values in heads twice as wide
+    t = step_tables(first, [0] * len(first))
+    rows = torch.cat([xs[i][:n] for i, n in enumerate(first)])
+    wide = nqh + 2 * nkh
+    G, rest = (wide // 4, wide - 2 * (wide // 4)) if wide >= 4 else (1, wide - 2)
+    if rest % 2:
+        return
+    outs = [torch.zeros(t.rows, n, dtype=torch.float32, device="cuda") for n in (G * hd, G * hd, rest * hd)]
+    st2 = torch.zeros(len(first), (taps - 1) * ch * 4, dtype=torch.uint8, device="cuda")
+    K.conv_heads(rows, w, None, st2, 0, t, [K.conv_segment(G, hd, silu=True, norm="unit", factor=0.25, out=outs[0]),
+                                            K.conv_segment(G, hd, silu=True, norm="unit", out=outs[1]),
+                                            K.conv_segment(rest // 2, 2 * hd, silu=True, out=outs[2])], eps=1e-6)
+    r0 = 0
+    for i, n in enumerate(first[:30]):
+        z = P.silu(P.causal_conv(back(xs[i][:n]), back(w)))
+        assert rel(outs[0][r0:r0 + n], (P.unit_heads(z[:, :G * hd].view(n, G, hd)) * 0.25).reshape(n, -1)) < 5e-6
+        assert rel(outs[1][r0:r0 + n], P.unit_heads(z[:, G * hd:2 * G * hd].view(n, G, hd)).reshape(n, -1)) < 5e-6
+        assert rel(outs[2][r0:r0 + n], z[:, 2 * G * hd:]) < 5e-6
+        r0 += n
+
+
 def delta_inputs(g, n, H, G, dk, dv, dtype, spread=2.0, shift=-4.0):
     unit = lambda x: x / x.norm(dim=-1, keepdim=True)                           # noqa: E731
     q, k = (unit(torch.randn(n, G, dk, generator=g)) for _ in range(2))
@@ -201,6 +268,23 @@ def test_delta_rule_token_by_token_in_portions_and_over_chunks(K, dtype, H, G, d
             S = back(state[[3, 0, 2][i], off:].view(torch.float32)).view(H, dk, dv)
             assert rel(torch.cat(got[i]), want[i][0]) < 1e-5 and rel(S, want[i][1]) < 1e-5, (plan, i)
         assert state[1].abs().max() == 0 and state[4].abs().max() == 0
+
+
+def test_delta_rule_over_chunks_of_many_sequences_of_unequal_lengths(K):
+    """Chunks are packed one after the other: sequences that end anywhere, some of one token, in two steps."""
+    g = torch.Generator().manual_seed(8)
+    H, G, dk, dv = 2, 1, 20, 18
+    lens = [1, 64, 65, 130, 63, 2, 128, 1, 127, 200, 3, 61]
+    seqs = [delta_inputs(g, n, H, G, dk, dv, "float32") for n in lens]
+    bias, rate = torch.randn(H * dk, generator=g), torch.rand(H, generator=g) + 0.1
+    state = torch.zeros(len(lens), H * dk * dv * 4, dtype=torch.uint8, device="cuda")
+    cut = [(n + 1) // 2 for n in lens]
+    a = run_delta(K, seqs, [slice(0, c) for c in cut], list(range(len(lens))), state, bias, rate, H, G, dk, dv, True)
+    b = run_delta(K, seqs, [slice(c, n) for c, n in zip(cut, lens)], list(range(len(lens))), state, bias, rate, H, G, dk, dv, True)
+    for i, s in enumerate(seqs):
+        want, S = plain_delta(s, bias, rate, H, G)
+        assert rel(torch.cat([a[i]] + ([b[i]] if i in b else [])), want) < 1e-5, i
+        assert rel(back(state[i].view(torch.float32)).view(H, dk, dv), S) < 1e-5, i
 
 
 @pytest.mark.parametrize("dk", [32, 64, 128, 256])
