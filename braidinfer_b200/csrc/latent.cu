@@ -38,13 +38,15 @@ struct LatentPrepArgs {
     int q_rank;
 };
 
-template <typename T>
-__global__ void __launch_bounds__(128)
+// A CTA a row.  V neighbouring numbers a thread and turn (16 bytes, or one number where a size or stride does not allow it); the
+// first two runs of a thread stay in registers between the sums of squares and the results, and both norms' sums meet in one round.
+template <typename T, int V, int NT>
+__global__ void __launch_bounds__(NT)
 latent_prep_kernel(LatentPrepArgs a) {
     pdl_trigger();
-    pdl_wait();
-    __shared__ float red[32];
-    const int row = blockIdx.x;
+    __shared__ float2 red[NT / 32];
+    const int row = blockIdx.x, tid = threadIdx.x;
+    // the step's tables are on the device before its first kernel: read before the wait
     const int seq = a.token_seq[row];
     const int pos = seq < 0 ? 0 : a.positions[row];
     const int D = a.rank + a.rot;
@@ -56,39 +58,63 @@ latent_prep_kernel(LatentPrepArgs a) {
         const int block = pos / a.page_size, off = pos - block * a.page_size;
         int page = (block < a.table_cols) ? a.page_table[(size_t)seq * a.table_cols + block] : -1;
         if (page < 0 || page >= a.num_pages) {
-            if (threadIdx.x == 0) atomicExch(a.error_flag, 1);
+            if (tid == 0) atomicExch(a.error_flag, 1);
         } else {
             dst = (T*)a.cache + ((size_t)page * a.page_size + off) * D;
         }
     }
-    // c = x / sqrt(mean(x^2) + eps) * w  (only where there is a cache to write: a layer that reads another layer's
-    // latent has no c and no kr in its rows)
-    float ss = 0.f;
-    if (a.cache) {
-        for (int i = threadIdx.x; i < a.rank; i += blockDim.x) {
-            const float v = to_f32(cin[i]);
-            ss = fmaf(v, v, ss);
+    // c = x / sqrt(mean(x^2) + eps) * w where there is a cache to write (a layer that reads another layer's latent has no c and
+    // no kr in its rows), and the same for the queries' low-rank part where the rows have one: runs [0, nq) and [nq, nq + nc)
+    const int nq = a.dq_out ? a.q_rank / V : 0, nc = a.cache ? a.rank / V : 0;
+    constexpr int KEEP = 2;
+    float v[KEEP][V];
+    pdl_wait();
+    if (nq + nc > 0) {
+        float2 ss = make_float2(0.f, 0.f);
+        auto take = [&](int run, float* x) {
+            load_run<T, V>(run < nq ? src + (size_t)run * V : cin + (size_t)(run - nq) * V, x);
+            float t = 0.f;
+#pragma unroll
+            for (int e = 0; e < V; ++e) t = fmaf(x[e], x[e], t);
+            if (run < nq) ss.x += t;
+            else ss.y += t;
+        };
+#pragma unroll
+        for (int k = 0; k < KEEP; ++k)
+            if (tid + k * NT < nq + nc) take(tid + k * NT, v[k]);
+        for (int run = tid + KEEP * NT; run < nq + nc; run += NT) {
+            float x[V];
+            take(run, x);
         }
-        ss = block_sum(ss, red);
-    }
-    const float scale = 1.f / sqrtf(ss / (float)a.rank + a.eps);
-    if (a.dq_out) {
-        float sq = 0.f;
-        for (int i = threadIdx.x; i < a.q_rank; i += blockDim.x) {
-            const float v = to_f32(src[i]);
-            sq = fmaf(v, v, sq);
+        ss.x = warp_sum(ss.x);
+        ss.y = warp_sum(ss.y);
+        if ((tid & 31) == 0) red[tid >> 5] = ss;
+        __syncthreads();
+        float sq = 0.f, sc = 0.f;
+#pragma unroll
+        for (int w = 0; w < NT / 32; ++w) { sq += red[w].x; sc += red[w].y; }
+        const float rq = 1.f / sqrtf(sq / (float)max(a.q_rank, 1) + a.eps), rc = 1.f / sqrtf(sc / (float)a.rank + a.eps);
+        auto give = [&](int run, const float* x) {
+            const bool q = run < nq;
+            const int i = (q ? run : run - nq) * V;
+            T* out = q ? (T*)a.dq_out + (size_t)row * a.dq_ld : dst;
+            if (!out) return;
+            float w[V], y[V];
+            load_run<T, V>((const T*)(q ? a.dq_w : a.norm_w) + i, w);
+#pragma unroll
+            for (int e = 0; e < V; ++e) y[e] = x[e] * (q ? rq : rc) * w[e];
+            store_run<T, V>(out + i, y);
+        };
+#pragma unroll
+        for (int k = 0; k < KEEP; ++k)
+            if (tid + k * NT < nq + nc) give(tid + k * NT, v[k]);
+        for (int run = tid + KEEP * NT; run < nq + nc; run += NT) {
+            float x[V];
+            load_run<T, V>(run < nq ? src + (size_t)run * V : cin + (size_t)(run - nq) * V, x);
+            give(run, x);
         }
-        __syncthreads();                                   // the sum before has been read
-        sq = block_sum(sq, red);
-        const float qs = 1.f / sqrtf(sq / (float)a.q_rank + a.eps);
-        T* o = (T*)a.dq_out + (size_t)row * a.dq_ld;
-        const T* w = (const T*)a.dq_w;
-        for (int i = threadIdx.x; i < a.dq_ld; i += blockDim.x)
-            o[i] = i < a.q_rank ? from_f32<T>(to_f32(src[i]) * qs * to_f32(w[i])) : from_f32<T>(0.f);
-    }
-    if (dst) {
-        const T* w = (const T*)a.norm_w;
-        for (int i = threadIdx.x; i < a.rank; i += blockDim.x) dst[i] = from_f32<T>(to_f32(cin[i]) * scale * to_f32(w[i]));
+        if (a.dq_out)                                          // what the low-rank rows are padded with
+            for (int i = a.q_rank + tid; i < a.dq_ld; i += NT) ((T*)a.dq_out)[(size_t)row * a.dq_ld + i] = from_f32<T>(0.f);
     }
     // rotation: element i pairs with i + rot_dims/2 (or, `adjacent`, 2i with 2i + 1); vector 0 is the shared key
     // part, 1.. are the heads' queries
@@ -128,9 +154,22 @@ extern "C" int braid_latent_prep(const void* proj, long long ld, int q_cols, con
     LatentPrepArgs a{proj, ld, q_cols, norm_w, inv_freq, positions, token_seq, page_table, cache, q_lat,
                      rows, heads, dim, rot, rank, rot_dims, page_size, table_cols, num_pages, eps, error_flag, adjacent, dq_out, dq_ld, dq_w, q_rank};
     cudaStream_t s = (cudaStream_t)stream;
-    if (dtype == BRAID_F32) braid_launch(latent_prep_kernel<float>, dim3(rows), dim3(128), 0, s, a);
-    else if (dtype == BRAID_BF16) braid_launch(latent_prep_kernel<__nv_bfloat16>, dim3(rows), dim3(128), 0, s, a);
+    const int vec = dtype == BRAID_F32 ? 4 : 8;
+    const bool wide = ld % vec == 0 && q_cols % vec == 0 && rank % vec == 0 && (rank + rot) % vec == 0 && q_rank % vec == 0 && dq_ld % vec == 0 &&
+                      (((uintptr_t)proj | (uintptr_t)norm_w | (uintptr_t)cache | (uintptr_t)dq_out | (uintptr_t)dq_w) & 15) == 0;
+    // 256 threads a row where the norms have that much to do, or where rows are few and a row's way is what counts
+    const bool big = rows <= 64 || (dq_out ? q_rank : 0) + rank > 128 * vec;
+#define LP_LAUNCH(T, V)                                                                                     \
+    do {                                                                                                    \
+        if (big) braid_launch(latent_prep_kernel<T, V, 256>, dim3(rows), dim3(256), 0, s, a);               \
+        else braid_launch(latent_prep_kernel<T, V, 128>, dim3(rows), dim3(128), 0, s, a);                   \
+    } while (0)
+    if (dtype == BRAID_F32 && wide) LP_LAUNCH(float, 4);
+    else if (dtype == BRAID_F32) LP_LAUNCH(float, 1);
+    else if (dtype == BRAID_BF16 && wide) LP_LAUNCH(__nv_bfloat16, 8);
+    else if (dtype == BRAID_BF16) LP_LAUNCH(__nv_bfloat16, 1);
     else BRAID_REFUSE("latent_prep: unknown dtype code %d", dtype);
+#undef LP_LAUNCH
     BRAID_LAUNCH_CHECK();
 }
 
