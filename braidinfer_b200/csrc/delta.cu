@@ -203,7 +203,6 @@ delta_intra_kernel(DeltaArgs a) {
     float* sE = sT + DKP;                    // the product of all decays before the sub-chunk
     int* steep = (int*)(sE + DKP);           // the channels whose factors cannot be split, their number in n_steep
     __shared__ int n_steep;
-    pdl_trigger();
     const int h = blockIdx.x, seq = blockIdx.y, c = blockIdx.z, tid = threadIdx.x;
     const int n = min(C, a.q_len[seq] - c * C), r0 = a.q_start[seq] + c * C;
     if (n <= 0) return;
@@ -373,6 +372,7 @@ delta_intra_kernel(DeltaArgs a) {
 #pragma unroll
         for (int t = 0; t < C; ++t) dst[t * step] = x[t];
     }
+    pdl_trigger();
 }
 
 // ------------------------------------------------------------------ chunk after chunk
@@ -396,6 +396,7 @@ __device__ __forceinline__ void delta_copy(float* dst, const float* src, int tid
 // bound by the reads of shared memory); the warps' partial tiles meet in shared memory, where the thread that owns four numbers
 // of U or of S adds them up.
 #define DELTA_STATE_THREADS 256
+#define DELTA_ALONE_SMEM (120 * 1024)
 template <int DKP> constexpr int delta_state_smem() {
     return (2 * DELTA_C * (DKP + 4) + (DKP + DELTA_C) * DELTA_DVT + 8 * DELTA_C * DELTA_DVT) * 4;
 }
@@ -654,14 +655,19 @@ static int launch_delta_chunks(const DeltaArgs& a, int n_seqs, cudaStream_t s) {
     static bool configured = false;
     if (!configured) {
         cudaError_t e = cudaFuncSetAttribute(delta_intra_kernel<T, DKP>, cudaFuncAttributeMaxDynamicSharedMemorySize, delta_intra_smem<DKP>());
-        if (e == cudaSuccess) e = cudaFuncSetAttribute(delta_state_kernel<DKP>, cudaFuncAttributeMaxDynamicSharedMemorySize, delta_state_smem<DKP>());
+        if (e == cudaSuccess) e = cudaFuncSetAttribute(delta_state_kernel<DKP>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+                                                         delta_state_smem<DKP>() > DELTA_ALONE_SMEM ? delta_state_smem<DKP>() : DELTA_ALONE_SMEM);
         if (e == cudaSuccess) e = cudaFuncSetAttribute(delta_out_kernel<DKP>, cudaFuncAttributeMaxDynamicSharedMemorySize, delta_out_smem<DKP>());
         if (e != cudaSuccess) { braid_set_error("delta_rule: cannot reserve shared memory: %s", cudaGetErrorString(e)); return (int)e; }
         configured = true;
     }
     const int spans = (a.tiles * DELTA_DVT + DELTA_OUT_COLS - 1) / DELTA_OUT_COLS;
     braid_launch(delta_intra_kernel<T, DKP>, dim3(a.heads, n_seqs, a.max_chunks), dim3(DELTA_INTRA_THREADS), delta_intra_smem<DKP>(), s, a);
-    braid_launch(delta_state_kernel<DKP>, dim3(a.heads, n_seqs, a.tiles), dim3(DELTA_STATE_THREADS), delta_state_smem<DKP>(), s, a);
+    // where one CTA an SM covers the step, each asks for more than half of an SM's shared memory: launched while the kernel before
+    // drains, they would otherwise settle two and more on the SMs that are free first (8 heads of 128 x 256: 287 -> 220 us in all)
+    const bool alone = (long long)a.heads * n_seqs * a.tiles <= 148;
+    const int state_smem = alone && delta_state_smem<DKP>() < DELTA_ALONE_SMEM ? DELTA_ALONE_SMEM : delta_state_smem<DKP>();
+    braid_launch(delta_state_kernel<DKP>, dim3(a.heads, n_seqs, a.tiles), dim3(DELTA_STATE_THREADS), state_smem, s, a);
     braid_launch(delta_out_kernel<DKP>, dim3(a.heads, n_seqs, a.max_chunks * spans), dim3(DELTA_OUT_THREADS), delta_out_smem<DKP>(), s, a);
     BRAID_LAUNCH_CHECK();
 }
