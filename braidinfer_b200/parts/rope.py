@@ -14,8 +14,8 @@ pair index that turns t times over the original length, lo = max(floor(d(fast)),
 rd - 1) and ramp_p = clamp((p - lo) / max(hi - lo, 0.001), 0, 1):
     f'_p = f_p / factor * ramp_p + f_p * (1 - ramp_p),     amplitude = 0.1 ln(factor) + 1 on sine and cosine.
 Fast pairs keep their frequency, slow pairs are divided by the factor, those between are blended.
-With `"kind": "bands"` the scaling is the other common one (Grattafiori and others: "The Llama 3 Herd of Models", 2024,
-whose 3.1 models use it), by wavelength: l_p = 2 pi / f_p, two bounds `high` > `low` on original / l_p, no amplitude:
+With `"kind": "bands"` the scaling is the other common one (Llama 3.1's), by wavelength: l_p = 2 pi / f_p, two bounds
+`high` > `low` on original / l_p, no amplitude:
     f'_p = f_p                                      l_p < original / high
     f'_p = f_p / factor                             l_p > original / low
     f'_p = (1 - s) f_p / factor + s f_p             between, s = (original / l_p - low) / (high - low)
